@@ -28,6 +28,8 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "--use_fast_math",
 ]
+# files that hold 32-bit reference-grade arithmetic: no fast-math substitutions
+PRECISE_SOURCES = {"layer_ops.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function"]
 
 
@@ -40,7 +42,7 @@ def _cuda_home() -> str:
 
 def _sources():
     cu = sorted((CSRC / "kernels").glob("*.cu"))
-    cpp = sorted((CSRC / "host").glob("*.cpp")) + [CSRC / "bindings.cpp"]
+    cpp = sorted((CSRC / "host").glob("*.cpp")) + sorted(CSRC.glob("bindings*.cpp"))
     headers = sorted(list(CSRC.rglob("*.cuh")) + list(CSRC.rglob("*.h")))
     return cu, cpp, headers
 
@@ -104,16 +106,17 @@ def build(verbose: bool = False, force: bool = False) -> Path:
     for src in cu:
         obj = BUILD_DIR / (src.stem + ".cu.o")
         objects.append(obj)
-        key = _hash([src], header_hash + " ".join(NVCC_FLAGS))
+        flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or src.name not in PRECISE_SOURCES]
+        key = _hash([src], header_hash + " ".join(flags))
         if force or not obj.exists() or obj_stamps.get(obj.name) != key:
-            jobs.append((obj, key, [nvcc, *NVCC_FLAGS, *inc_cuda, "-c", str(src), "-o", str(obj)]))
+            jobs.append((obj, key, [nvcc, *flags, *inc_cuda, "-c", str(src), "-o", str(obj)]))
     for src in cpp:
         obj = BUILD_DIR / (src.stem + ".cpp.o")
         objects.append(obj)
         key = _hash([src], header_hash + " ".join(CXX_FLAGS))
         if force or not obj.exists() or obj_stamps.get(obj.name) != key:
             flags = list(CXX_FLAGS)
-            if src.name == "bindings.cpp":
+            if src.name.startswith("bindings"):
                 flags += ["-DTORCH_EXTENSION_NAME=_C", "-DTORCH_API_INCLUDE_EXTENSION_H", "-D_GLIBCXX_USE_CXX11_ABI=1"]
                 incs = inc_all
             else:

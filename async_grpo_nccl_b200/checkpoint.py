@@ -40,7 +40,7 @@ def save_hf_model(path: str, cfg: ModelConfig, layout: ParamLayout, flat: torch.
     shards: List[Dict[str, torch.Tensor]] = [{}]
     size = 0
     for name, t in layout.hf_items(flat):
-        tb = t.detach().to(torch.bfloat16).cpu().contiguous()
+        tb = t.detach().to(torch.bfloat16).cpu().reshape(layout.hf_shape(name, t)).contiguous()
         nbytes = tb.numel() * 2
         if size + nbytes > max_shard_bytes and shards[-1]:
             shards.append({})
@@ -89,13 +89,14 @@ def load_hf_model(path: str, layout: ParamLayout, out: Optional[torch.Tensor] = 
         with safe_open(os.path.join(path, fn), framework="pt", device="cpu") as f:
             for key in f.keys():
                 if key not in dest:
-                    if key == "lm_head.weight" and layout.cfg.tie_word_embeddings:
+                    if key == "lm_head.weight" and getattr(layout.cfg, "tie_word_embeddings", False):
                         continue
                     raise KeyError(f"unexpected tensor {key} in {fn}")
                 t = f.get_tensor(key)
-                if tuple(t.shape) != tuple(dest[key].shape):
-                    raise ValueError(f"shape mismatch for {key}: {tuple(t.shape)} vs {tuple(dest[key].shape)}")
-                dest[key].copy_(t.to(torch.float32))
+                want = layout.hf_shape(key, dest[key])
+                if tuple(t.shape) != want:
+                    raise ValueError(f"shape mismatch for {key}: {tuple(t.shape)} vs {want}")
+                dest[key].copy_(t.to(torch.float32).reshape(dest[key].shape))
                 seen.add(key)
     missing = [k for k in dest if k not in seen]
     if missing:

@@ -8,6 +8,7 @@
 #include <pybind11/stl.h>
 
 #include "host/kv_allocator.h"
+#include "bindings_layers.h"
 #include "host/packer.h"
 #include "launchers.h"
 
@@ -840,8 +841,15 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
       .def_property_readonly("num_free", &agrpo::BlockAllocator::num_free)
       .def_property_readonly("num_blocks", &agrpo::BlockAllocator::num_blocks);
   py::class_<agrpo::Scheduler>(m, "Scheduler")
-      .def(py::init<int, int, int, int, int>(), py::arg("num_blocks"), py::arg("block_size"), py::arg("max_seqs"),
-           py::arg("max_blocks_per_seq"), py::arg("max_prefill_tokens"))
+      .def(py::init<int, int, int, int, int, int>(), py::arg("num_blocks"), py::arg("block_size"), py::arg("max_seqs"),
+           py::arg("max_blocks_per_seq"), py::arg("max_prefill_tokens"), py::arg("window_tokens") = 0)
+      .def("open_seq", [](agrpo::Scheduler& s) { const auto r = s.open_seq(); return py::make_tuple(r.first, r.second); })
+      .def("extend_seq",
+           [](agrpo::Scheduler& s, long long id, int n) {
+             py::list out;
+             for (const auto& u : s.extend_seq(id, n)) out.append(py::make_tuple(u.slot, u.index, u.block));
+             return out;
+           })
       .def("add_group",
            [](agrpo::Scheduler& s, long long group_id, int prompt_len, int n, int max_new_tokens, std::vector<int> forced,
               std::vector<unsigned long long> block_hashes) {
@@ -872,6 +880,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
       .def_property_readonly("num_cached_blocks", &agrpo::Scheduler::num_cached_blocks)
       .def("clear_prefix_cache", &agrpo::Scheduler::clear_prefix_cache);
 
+  bind_layer_ops(m);
   m.def("gemm_bf16", &gemm_bf16, py::arg("a"), py::arg("b"), py::arg("d"), py::arg("a_mn") = false,
         py::arg("b_mn") = false, py::arg("bias") = py::none(), py::arg("alpha") = 1.0, py::arg("accumulate") = false,
         py::arg("status") = py::none(), py::arg("residual") = py::none(), NOGIL);

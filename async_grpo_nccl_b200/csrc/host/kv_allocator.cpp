@@ -84,9 +84,9 @@ void BlockAllocator::clear_cache() {
   n_evictable_ = 0;
 }
 
-Scheduler::Scheduler(int num_blocks, int block_size, int max_seqs, int max_blocks_per_seq, int max_prefill_tokens)
+Scheduler::Scheduler(int num_blocks, int block_size, int max_seqs, int max_blocks_per_seq, int max_prefill_tokens, int window_tokens)
     : alloc_(num_blocks), block_size_(block_size), max_seqs_(max_seqs), max_blocks_per_seq_(max_blocks_per_seq),
-      max_prefill_tokens_(max_prefill_tokens), slot_owner_(max_seqs, -1) {
+      max_prefill_tokens_(max_prefill_tokens), window_tokens_(window_tokens), slot_owner_(max_seqs, -1) {
   for (int s = max_seqs - 1; s >= 0; --s) free_slots_.push_back(s);
 }
 
@@ -201,8 +201,9 @@ DecodePlan Scheduler::plan_decode() {
   for (int slot = 0; slot < max_seqs_; ++slot) {
     if (slot_owner_[slot] < 0) continue;
     auto it = seqs_.find(slot_owner_[slot]);
-    if (it == seqs_.end() || it->second.finished) continue;
+    if (it == seqs_.end() || it->second.finished || it->second.external) continue;
     order.push_back(&it->second);
+    drop_out_of_window(it->second);
   }
   for (SeqState* s : order) {
     if (s->slot < 0) continue;  // preempted earlier in this loop
@@ -237,14 +238,57 @@ DecodePlan Scheduler::plan_decode() {
   return plan;
 }
 
+// The token at position `len` comes next; no layer of any later step reads a key before position len - window + 1.
+void Scheduler::drop_out_of_window(SeqState& s) {
+  if (window_tokens_ <= 0) return;
+  const int gone = (s.len - window_tokens_ + 1) / block_size_;
+  for (; s.first_live < gone && s.first_live < (int)s.blocks.size(); ++s.first_live) {
+    alloc_.release(s.blocks[s.first_live]);
+    s.blocks[s.first_live] = -1;
+  }
+}
+
+std::pair<long long, int> Scheduler::open_seq() {
+  if (free_slots_.empty()) throw std::runtime_error("open_seq: no free slot");
+  SeqState s;
+  s.seq_id = next_seq_id_++;
+  s.external = true;
+  s.slot = free_slots_.back();
+  free_slots_.pop_back();
+  slot_owner_[s.slot] = s.seq_id;
+  const auto out = std::make_pair(s.seq_id, s.slot);
+  seqs_.emplace(s.seq_id, std::move(s));
+  return out;
+}
+
+std::vector<TableUpdate> Scheduler::extend_seq(long long seq_id, int n) {
+  commit_pending_hashes();
+  auto it = seqs_.find(seq_id);
+  if (it == seqs_.end() || !it->second.external || it->second.slot < 0) throw std::runtime_error("extend_seq: unknown sequence");
+  SeqState& s = it->second;
+  if (n <= 0) throw std::runtime_error("extend_seq: no tokens");
+  const int need = (s.len + n + block_size_ - 1) / block_size_;
+  if (need > max_blocks_per_seq_) throw std::runtime_error("extend_seq: sequence would exceed max_blocks_per_seq");
+  drop_out_of_window(s);
+  std::vector<TableUpdate> out;
+  if (need - (int)s.blocks.size() > alloc_.num_free()) throw std::runtime_error("extend_seq: the cache has no room for these tokens");
+  while ((int)s.blocks.size() < need) {
+    s.blocks.push_back(alloc_.alloc());
+    out.push_back({s.slot, (int)s.blocks.size() - 1, s.blocks.back()});
+  }
+  s.len += n;
+  return out;
+}
+
 void Scheduler::release_seq(SeqState& s) {
-  for (int b : s.blocks) alloc_.release(b);
+  for (int b : s.blocks)
+    if (b >= 0) alloc_.release(b);
   s.blocks.clear();
   if (s.slot >= 0) {
     slot_owner_[s.slot] = -1;
     free_slots_.push_back(s.slot);
     s.slot = -1;
-    --num_running_;
+    if (!s.external) --num_running_;
   }
   s.finished = true;
 }

@@ -62,6 +62,8 @@ struct SeqState {
   int max_len = 0;             // prompt_len + max new tokens
   int forced_len = -1;         // total length at which generation is cut (EOS forced), -1 = none
   bool finished = false;
+  bool external = false;       // advanced by extend_seq(), not by plan_decode()
+  int first_live = 0;          // blocks before this index are outside every layer's window and have been given back (-1)
   std::vector<int> blocks;
 };
 
@@ -100,7 +102,9 @@ struct DecodePlan {
 
 class Scheduler {
  public:
-  Scheduler(int num_blocks, int block_size, int max_seqs, int max_blocks_per_seq, int max_prefill_tokens);
+  // window_tokens > 0: no layer looks further back than that many tokens (the current one included), so blocks that
+  // have left the window are returned to the pool while their sequence still runs.
+  Scheduler(int num_blocks, int block_size, int max_seqs, int max_blocks_per_seq, int max_prefill_tokens, int window_tokens = 0);
 
   void add_group(const GroupRequest& req);
   int num_waiting() const { return (int)waiting_.size(); }
@@ -114,6 +118,11 @@ class Scheduler {
   PrefillPlan plan_prefill();
   // Accounts for one more token per running sequence and allocates blocks where a boundary is crossed.
   DecodePlan plan_decode();
+  // A sequence whose tokens the caller supplies (step-wise driving: prompts in portions of any size, replay of a trace).
+  // Returns {sequence id, slot}; extend_seq() makes room for n more tokens and returns the new block-table entries; finish()
+  // gives everything back.
+  std::pair<long long, int> open_seq();
+  std::vector<TableUpdate> extend_seq(long long seq_id, int n);
   // Marks a sequence finished and frees its slot and blocks.
   void finish(long long seq_id);
   // Moves the sequences in the highest slots into the lowest free slots so that the running sequences occupy a dense
@@ -127,9 +136,10 @@ class Scheduler {
 
  private:
   void release_seq(SeqState& s);
+  void drop_out_of_window(SeqState& s);
   void commit_pending_hashes();
   BlockAllocator alloc_;
-  int block_size_, max_seqs_, max_blocks_per_seq_, max_prefill_tokens_;
+  int block_size_, max_seqs_, max_blocks_per_seq_, max_prefill_tokens_, window_tokens_;
   std::deque<GroupRequest> waiting_;
   std::unordered_map<long long, SeqState> seqs_;
   std::vector<long long> slot_owner_;

@@ -70,12 +70,63 @@ class RolloutEngine:
                  eos_token_id: Optional[int] = None, tp: Any = None, prefix_caching: bool = False):
         from ..ops import native
 
-        assert params.is_cuda and params.dtype == torch.bfloat16
-        if block_size != 16 or cfg.head_dim != 128:
-            raise ValueError("the native engine supports block_size 16 and head_dim 128")
+        assert params.is_cuda
+        self._check_model(cfg, params, block_size)
         self.C = native()
         self.cfg, self.layout, self.params = cfg, layout, params
         self.dev = params.device
+        self._init_sharing(tp, prefix_caching)
+        self.prefix_hit_tokens = 0
+        self.prefix_lookup_tokens = 0
+        self.sm_count = torch.cuda.get_device_properties(self.dev).multi_processor_count  # SMs the engine's stream may use
+        self.block_size = block_size
+        self.max_seqs = int(max_seqs)
+        self.max_model_len = int(max_model_len or cfg.max_position_embeddings)
+        self.max_blocks_per_seq = (self.max_model_len + block_size - 1) // block_size
+        self.max_prefill_tokens = int(max_prefill_tokens)
+        self.eos = cfg.eos_token_id if eos_token_id is None else int(eos_token_id)
+        self._init_decoder()
+        self.status = self.dec.status
+        if num_blocks is None:
+            if kv_memory_bytes is None:
+                free, _ = torch.cuda.mem_get_info(self.dev)
+                kv_memory_bytes = int(free * 0.6)
+            num_blocks = max(64, kv_memory_bytes // self._bytes_per_block())
+        self.num_blocks = int(num_blocks)
+        self._alloc_cache()
+        self.sched = self.C.Scheduler(self.num_blocks, block_size, self.max_seqs, self.max_blocks_per_seq,
+                                      self.max_prefill_tokens, self._window_tokens())
+        self._init_slots()
+        self._init_decode_path()
+        # chosen-token log-probabilities (off until a caller asks: one more small tensor op per step)
+        self.record_logprobs = False
+        self.b_lp: Optional[torch.Tensor] = None
+        self.history_lp: Optional[torch.Tensor] = None
+        self.use_cuda_graph = use_cuda_graph
+        self.use_pdl = os.environ.get("AGRPO_DECODE_PDL", "1") != "0"
+        # keep running sequences in a dense prefix of the slots: the decode batch has as many rows as the highest slot
+        self.compact_slots = os.environ.get("AGRPO_COMPACT_SLOTS", "1") != "0"
+        self.n_compactions = 0
+        self._last_rows = self._last_active = 0
+        self.graphs: Dict[Tuple[int, float, int], torch.cuda.CUDAGraph] = {}
+        self.requests: Dict[int, _Request] = {}
+        self.slot_info: Dict[int, Dict[str, Any]] = {}
+        self.pending: List[_Request] = []
+        self.next_group = 0
+        self.temperature: Optional[float] = None
+        self.tokens_generated = 0
+        self.h2d_bytes = 0
+        self.d2h_bytes = 0
+
+    # ------------------------------------------------------------------ what a model class decides (overridden by other designs)
+    def _check_model(self, cfg: Any, params: torch.Tensor, block_size: int) -> None:
+        if params.dtype != torch.bfloat16:
+            raise ValueError("the native engine of the dense decoders runs bf16 parameters")
+        if block_size != 16 or cfg.head_dim != 128:
+            raise ValueError("the native engine supports block_size 16 and head_dim 128")
+
+    def _init_sharing(self, tp: Any, prefix_caching: bool) -> None:
+        cfg = self.cfg
         # Tensor parallelism (vllm_worker.py:219-232, tensor_parallel_size): ``tp`` is a parallel.symm.TensorParallelComm.
         # This rank then holds Hq / tp query heads and Hkv / tp kv heads (projection columns, KV cache) and F / tp MLP
         # columns; the o and down projections produce partial sums that are all-reduced over peer memory. Embedding,
@@ -94,31 +145,31 @@ class RolloutEngine:
         # reuses them and only its remaining tokens go through the GEMMs. Forgotten at every weight update. A
         # tensor-parallel member caches only its own kv heads while the prefill needs all of them, so it stays off there.
         self.prefix_caching = bool(prefix_caching) and self.tp is None
-        self.prefix_hit_tokens = 0
-        self.prefix_lookup_tokens = 0
-        self.sm_count = torch.cuda.get_device_properties(self.dev).multi_processor_count  # SMs the engine's stream may use
-        self.dec = NativeDecoder(cfg, layout, params)
-        self.status = self.dec.status
-        self.block_size = block_size
-        self.max_seqs = int(max_seqs)
-        self.max_model_len = int(max_model_len or cfg.max_position_embeddings)
-        self.max_blocks_per_seq = (self.max_model_len + block_size - 1) // block_size
-        self.eos = cfg.eos_token_id if eos_token_id is None else int(eos_token_id)
-        per_block = cfg.num_hidden_layers * 2 * self.Hkv_l * block_size * cfg.head_dim * 2
-        if num_blocks is None:
-            if kv_memory_bytes is None:
-                free, _ = torch.cuda.mem_get_info(self.dev)
-                kv_memory_bytes = int(free * 0.6)
-            num_blocks = max(64, kv_memory_bytes // per_block)
-        self.num_blocks = int(num_blocks)
-        self.cache = torch.zeros(cfg.num_hidden_layers, 2, self.num_blocks, self.Hkv_l, block_size,
+
+    def _init_decoder(self) -> None:
+        self.dec = NativeDecoder(self.cfg, self.layout, self.params)
+        self.dec.ensure_rope(min(self.max_model_len, self.cfg.max_position_embeddings))
+
+    def _bytes_per_block(self) -> int:
+        return self.cfg.num_hidden_layers * 2 * self.Hkv_l * self.block_size * self.cfg.head_dim * 2
+
+    def _alloc_cache(self) -> None:
+        cfg = self.cfg
+        self.cache = torch.zeros(cfg.num_hidden_layers, 2, self.num_blocks, self.Hkv_l, self.block_size,
                                  cfg.head_dim, dtype=torch.bfloat16, device=self.dev)
-        self.sched = self.C.Scheduler(self.num_blocks, block_size, self.max_seqs, self.max_blocks_per_seq,
-                                      int(max_prefill_tokens))
-        self.dec.ensure_rope(min(self.max_model_len, cfg.max_position_embeddings))
-        S, H = self.max_seqs, cfg.hidden_size
+
+    def _window_tokens(self) -> int:
+        """How far back any layer looks (0 = to the start): blocks beyond it go back to the pool."""
+        return 0
+
+    def _slot_tensors(self) -> List[torch.Tensor]:
+        """Further per-slot device state (first dimension = slot) that moves with a sequence when slots are compacted."""
+        return []
+
+    def _init_slots(self) -> None:
+        """Per-slot state that every design has: tables, lengths, token history, host mirrors, staging."""
+        cfg, S = self.cfg, self.max_seqs
         i32 = dict(dtype=torch.int32, device=self.dev)
-        bf = dict(dtype=torch.bfloat16, device=self.dev)
         self.block_tables = torch.zeros(S, self.max_blocks_per_seq, **i32)
         self.seq_lens = torch.zeros(S, **i32)
         self.positions = torch.zeros(S, **i32)
@@ -129,23 +180,7 @@ class RolloutEngine:
         self.row_ids = torch.arange(S, dtype=torch.int64, device=self.dev)
         self.hist_cap = self.max_model_len
         self.history = torch.zeros(S, self.hist_cap, **i32)
-        # decode activations (persistent: no allocation inside a step, required for graph capture); the persistent
-        # layer kernel loads them in row tiles of 32 / 64 / 128 / 256, so the buffers hold at least the tile that covers S
-        SA = next((t for t in (32, 64, 128, 256) if t >= S), S)
-        self.b_x = torch.zeros(SA, H, **bf)
-        self.b_x1 = torch.zeros(SA, H, **bf)
-        self.b_h = torch.empty(S, H, **bf)
-        self.b_qkv = torch.zeros(SA, self.Q_l, **bf)
-        self.b_attn = torch.zeros(SA, self.qd_l, **bf)
-        self.b_gu = torch.empty(S, 2 * self.F_l, **bf)
-        self.b_act = torch.zeros(SA, self.F_l, **bf)
         self.b_tokens = torch.zeros(S, **i32)
-        self.max_splits = 8
-        self.b_part_o = torch.empty(S * cfg.num_key_value_heads * self.max_splits * 8 * cfg.head_dim, dtype=torch.float32,
-                                    device=self.dev)
-        self.b_part_ml = torch.empty(S * cfg.num_key_value_heads * self.max_splits * 16, dtype=torch.float32, device=self.dev)
-        # arrival counters of the split-KV merge (the last split CTA merges; counters re-arm themselves)
-        self.b_tickets = torch.zeros(S * cfg.num_key_value_heads, dtype=torch.int32, device=self.dev)
         groups = int(self.C.lm_sample_num_groups(cfg.vocab_size, S))
         g_small = max(groups, int(self.C.lm_sample_num_groups(cfg.vocab_size, 1)))
         self.b_sample_f = torch.empty(4 * g_small * S, dtype=torch.float32, device=self.dev)
@@ -172,6 +207,28 @@ class RolloutEngine:
         # host-side time accounting of the step loop (seconds): where a step's wall time goes on the CPU
         self.t_plan = self.t_prep = self.t_launch = self.t_post = self.t_prefill = self.t_wait = 0.0
         self.n_decode_steps = self.n_prefill_steps = 0
+
+    def _init_decode_path(self) -> None:
+        cfg = self.cfg
+        S, H = self.max_seqs, cfg.hidden_size
+        i32 = dict(dtype=torch.int32, device=self.dev)
+        bf = dict(dtype=torch.bfloat16, device=self.dev)
+        # decode activations (persistent: no allocation inside a step, required for graph capture); the persistent
+        # layer kernel loads them in row tiles of 32 / 64 / 128 / 256, so the buffers hold at least the tile that covers S
+        SA = next((t for t in (32, 64, 128, 256) if t >= S), S)
+        self.b_x = torch.zeros(SA, H, **bf)
+        self.b_x1 = torch.zeros(SA, H, **bf)
+        self.b_h = torch.empty(S, H, **bf)
+        self.b_qkv = torch.zeros(SA, self.Q_l, **bf)
+        self.b_attn = torch.zeros(SA, self.qd_l, **bf)
+        self.b_gu = torch.empty(S, 2 * self.F_l, **bf)
+        self.b_act = torch.zeros(SA, self.F_l, **bf)
+        self.max_splits = 8
+        self.b_part_o = torch.empty(S * cfg.num_key_value_heads * self.max_splits * 8 * cfg.head_dim, dtype=torch.float32,
+                                    device=self.dev)
+        self.b_part_ml = torch.empty(S * cfg.num_key_value_heads * self.max_splits * 16, dtype=torch.float32, device=self.dev)
+        # arrival counters of the split-KV merge (the last split CTA merges; counters re-arm themselves)
+        self.b_tickets = torch.zeros(S * cfg.num_key_value_heads, dtype=torch.int32, device=self.dev)
         # ---- fused decode path (batches of up to 256 rows) ----
         # RMSNorm weights are folded into the columns of the matrices that consume the normalised rows (private copies
         # of wqkv and wgu, refreshed after every weight sync); the row scale rsqrt(mean(x^2) + eps) is applied in those
@@ -213,25 +270,6 @@ class RolloutEngine:
                 self.b_partials = torch.empty(int(self.C.decode_layers_scratch_bytes(self.mega_rows, H, Q, cfg.q_dim, F)) // 4,
                                               dtype=torch.float32, device=self.dev)
                 self.b_counters = torch.zeros(int(self.C.decode_layers_counter_words()), **i32)
-        # chosen-token log-probabilities (off until a caller asks: one more small tensor op per step)
-        self.record_logprobs = False
-        self.b_lp: Optional[torch.Tensor] = None
-        self.history_lp: Optional[torch.Tensor] = None
-        self.use_cuda_graph = use_cuda_graph
-        self.use_pdl = os.environ.get("AGRPO_DECODE_PDL", "1") != "0"
-        # keep running sequences in a dense prefix of the slots: the decode batch has as many rows as the highest slot
-        self.compact_slots = os.environ.get("AGRPO_COMPACT_SLOTS", "1") != "0"
-        self.n_compactions = 0
-        self._last_rows = self._last_active = 0
-        self.graphs: Dict[Tuple[int, float, int], torch.cuda.CUDAGraph] = {}
-        self.requests: Dict[int, _Request] = {}
-        self.slot_info: Dict[int, Dict[str, Any]] = {}
-        self.pending: List[_Request] = []
-        self.next_group = 0
-        self.temperature: Optional[float] = None
-        self.tokens_generated = 0
-        self.h2d_bytes = 0
-        self.d2h_bytes = 0
 
     # ------------------------------------------------------------------ requests
     def add_request(self, request_id: Any, prompt_ids: Sequence[int], n: int = 1, max_new_tokens: int = 128,
@@ -309,10 +347,9 @@ class RolloutEngine:
         self.C.lm_sample(hidden[:rows], wl, temperature, seeds, self.b_sample_f, self.b_sample_i, tokens, logprobs, self.status)
         self.launches += 2
 
-    def _prefill(self, plan: Dict[str, Any]) -> None:
+    def _prompt_hidden(self, plan: Dict[str, Any], reqs: List[_Request]) -> torch.Tensor:
+        """Runs the prompts of a prefill plan; returns the normalised hidden state of every prompt's last token."""
         cfg, C, dec = self.cfg, self.C, self.dec
-        gids = plan["group_ids"]
-        reqs = [self.requests[g] for g in gids]
         samples = [{"sample_ids": r.prompt, "input_len": len(r.prompt), "output_len": 0, "advantage": 0.0} for r in reqs]
         host_batch = pack_samples(samples, pin=True)
         batch = host_batch.to_device(self.dev)
@@ -336,10 +373,23 @@ class RolloutEngine:
             xl = x.index_select(0, last)
         hn = torch.empty_like(xl)
         C.rmsnorm_fwd(xl, dec.w("final_norm"), hn, None, cfg.rms_norm_eps)
+        return hn
+
+    def _copy_blocks(self, src: torch.Tensor, dst: torch.Tensor) -> None:
+        self.cache[:, :, dst] = self.cache[:, :, src]
+
+    def _share_prompt_state(self, plan: Dict[str, Any], reqs: List[_Request]) -> None:
+        """The n samples of a prompt start from the same state: copies what they cannot share (the partial last block)."""
         if plan["copy_src"]:
             src = torch.tensor(plan["copy_src"], dtype=torch.int64).pin_memory().to(self.dev, non_blocking=True)
             dst = torch.tensor(plan["copy_dst"], dtype=torch.int64).pin_memory().to(self.dev, non_blocking=True)
-            self.cache[:, :, dst] = self.cache[:, :, src]
+            self._copy_blocks(src, dst)
+
+    def _prefill(self, plan: Dict[str, Any]) -> None:
+        dec = self.dec
+        reqs = [self.requests[g] for g in plan["group_ids"]]
+        hn = self._prompt_hidden(plan, reqs)
+        self._share_prompt_state(plan, reqs)
         # one sampling row per child
         rep = torch.tensor([r.n for r in reqs], dtype=torch.int64, device=self.dev)
         hrep = hn.repeat_interleave(rep, dim=0).contiguous()
@@ -581,6 +631,15 @@ class RolloutEngine:
         C.lm_sample(h, wl, temperature, self.step_seeds, self.b_sample_f, self.b_sample_i, self.b_tokens, self.b_lp, st)
         self._feed_back(B)
 
+    def _choose_splits(self, B: int, n_active: int, max_len: int) -> int:
+        """Pieces that the attention of one sequence is cut into."""
+        if self.mega_rows and B <= self.mega_rows:
+            # the persistent layer kernel works on one attention item per CTA at a time: one wave of items
+            want = self.sm_count // max(1, n_active * self.cfg.num_key_value_heads)
+        else:
+            want = (self.sm_count * 3) // max(1, n_active * self.cfg.num_key_value_heads)
+        return int(max(1, min(self.max_splits, want, max(1, max_len // 256))))
+
     def _launch_count_decode(self, splits: int, B: int = 0) -> int:
         if self.mega_rows and 0 < B <= self.mega_rows:
             return 1 + 1 + 3
@@ -593,13 +652,8 @@ class RolloutEngine:
             per_layer = 9
         return 1 + per_layer * self.cfg.num_hidden_layers + 3
 
-    def _decode(self, plan: Dict[str, Any]) -> None:
-        rows = int(plan["batch_rows"])
-        if rows == 0:
-            return
-        t_begin = time.perf_counter()
-        B = min(self.max_seqs, (rows + 31) // 32 * 32)  # one captured graph per row count rounded to a warp of rows
-        active = plan["active_slots"]  # int32 array of slots
+    def _stage_decode(self, active: np.ndarray, upd_slot: np.ndarray, upd_index: np.ndarray, upd_block: np.ndarray) -> None:
+        """Brings the inputs of one decode step to the device: every active slot is one token longer."""
         S = self.max_seqs
         ri = self.step_count % len(self.stage_ring)
         t_w = time.perf_counter()
@@ -608,26 +662,31 @@ class RolloutEngine:
         self.h_lens[active] += 1
         self.step_count += 1
         st = self.stage_np[ri]
-        st[:S] = self.h_lens
-        n_upd = len(plan["upd_slot"])
+        st[:S] = 0  # slots that are not part of this step stay idle
+        st[active] = self.h_lens[active]
+        n_upd = len(upd_slot)
         st[S] = n_upd
         st[S + 1] = (self.step_count * 0x632BE5AB) & 0x7FFFFFFF
         if n_upd:
-            st[S + 4: S + 4 + n_upd] = plan["upd_slot"] * self.max_blocks_per_seq + plan["upd_index"]
-            st[S + 4 + S: S + 4 + S + n_upd] = plan["upd_block"]
+            st[S + 4: S + 4 + n_upd] = upd_slot * self.max_blocks_per_seq + upd_index
+            st[S + 4 + S: S + 4 + S + n_upd] = upd_block
         self.d_stage.copy_(self.stage_ring[ri], non_blocking=True)
         self.stage_events[ri].record()
         self.h2d_bytes += self.d_stage.numel() * 4
         # lengths, positions, seeds and the new block-table entries reach their device buffers in one launch
         self.C.decode_step_inputs(self.d_stage, S, self.seq_lens, self.positions, self.block_tables, self.base_seeds,
                                   self.step_seeds, self.status)
+
+    def _decode(self, plan: Dict[str, Any]) -> None:
+        rows = int(plan["batch_rows"])
+        if rows == 0:
+            return
+        t_begin = time.perf_counter()
+        B = min(self.max_seqs, (rows + 31) // 32 * 32)  # one captured graph per row count rounded to a warp of rows
+        active = plan["active_slots"]  # int32 array of slots
+        self._stage_decode(active, plan["upd_slot"], plan["upd_index"], plan["upd_block"])
         max_len = int(self.h_lens[:B].max())
-        if self.mega_rows and B <= self.mega_rows:
-            # the persistent layer kernel works on one attention item per CTA at a time: one wave of items
-            want = self.sm_count // max(1, len(active) * self.cfg.num_key_value_heads)
-        else:
-            want = (self.sm_count * 3) // max(1, len(active) * self.cfg.num_key_value_heads)
-        splits = int(max(1, min(self.max_splits, want, max(1, max_len // 256))))
+        splits = self._choose_splits(B, len(active), max_len)
         temperature = float(self.temperature or 0.0)
         t_mid = time.perf_counter()
         self.t_prep += t_mid - t_begin
@@ -721,7 +780,7 @@ class RolloutEngine:
         to = np.asarray([m[1] for m in moves], dtype=np.int64)
         idx = torch.from_numpy(np.stack([frm, to])).pin_memory().to(self.dev, non_blocking=True)
         self.h2d_bytes += idx.numel() * 8
-        moved = [self.block_tables, self.last_tokens, self.gen_index, self.base_seeds, self.history]
+        moved = [self.block_tables, self.last_tokens, self.gen_index, self.base_seeds, self.history] + self._slot_tensors()
         if self.record_logprobs:
             moved.append(self.history_lp)
         for t in moved:
@@ -732,7 +791,8 @@ class RolloutEngine:
             a[to] = a[frm]
             a[frm] = empty
         for f, t_ in moves:
-            self.slot_info[t_] = self.slot_info.pop(f)
+            if f in self.slot_info:  # step-wise driven sequences have no request
+                self.slot_info[t_] = self.slot_info.pop(f)
 
     def _free_slot(self, slot: int) -> None:
         self.n_watch -= int(self.h_watch[slot])
@@ -816,9 +876,11 @@ class RolloutEngine:
         because they reference the same buffers. The norm-folded copies of the fused decode path are refreshed
         here, and the caller's stream is drained so that the engine thread's next step sees them."""
         self.sched.clear_prefix_cache()  # cached keys and values belong to the previous weights
-        if self.fused_decode:
-            self.refold_weights()
-            torch.cuda.current_stream(self.dev).synchronize()
+        self._weights_changed()
+        torch.cuda.current_stream(self.dev).synchronize()
+
+    def _weights_changed(self) -> None:
+        self.refold_weights()
 
 
 # =====================================================================================================

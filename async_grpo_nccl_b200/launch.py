@@ -23,9 +23,10 @@ import torch
 from . import checkpoint as ckpt
 from .config import GRPOConfig
 from .experience import ExperienceManager
-from .models.config import ModelConfig, resolve_model_config
+from .models.config import ModelConfig
 from .models.decoder import NativeDecoder, OracleDecoder
 from .models.layout import ParamLayout
+from .models.registry import require_trainable, resolve_model_config
 from .rewards import get_or_create_verifier_pool
 from .roles.logprob import LogProbWorker
 from .roles.rollout import GenerationWorker
@@ -165,6 +166,7 @@ class InProcessRuntime:
         cfg = self.config
         self.mcfg = resolve_model_config(cfg.model_name_or_path, cfg.model_config)
         mcfg = self.mcfg
+        require_trainable(mcfg)
         probe_layout = ParamLayout(mcfg, 1)
         flat32 = initial_weights(cfg, mcfg, probe_layout, self.device)
         if self.native:
@@ -455,6 +457,7 @@ class DistributedRuntime:
             free = [0] * self.world
             free[self.rank] = int(f)
         mcfg0 = resolve_model_config(config.model_name_or_path, config.model_config)
+        require_trainable(mcfg0)
         # parameters in bf16 plus (trainer ranks) fp32 master + moments + gradients of this rank's share: a floor, not a plan
         need = mcfg0.num_parameters() * 2
         preflight_placement(place, self.world, torch.cuda.device_count() if cuda else None,

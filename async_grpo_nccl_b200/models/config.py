@@ -143,13 +143,3 @@ PRESETS: Dict[str, ModelConfig] = {
                                model_type="llama", eos_token_id=128001),
 }
 
-
-def resolve_model_config(model_name_or_path: Optional[str], inline: Optional[Dict[str, Any]]) -> ModelConfig:
-    """Inline dict wins; otherwise a preset name or a directory holding ``config.json``."""
-    if inline:
-        return ModelConfig.from_dict(inline)
-    if model_name_or_path in PRESETS:
-        return PRESETS[model_name_or_path]
-    if model_name_or_path and os.path.isdir(model_name_or_path):
-        return ModelConfig.from_pretrained(model_name_or_path)
-    raise FileNotFoundError(f"cannot resolve model config from {model_name_or_path!r}")

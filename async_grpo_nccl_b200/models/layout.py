@@ -11,7 +11,7 @@ conversion and no per-tensor ``load_weights`` as in the reference (gpu_process_w
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Dict, Iterator, List, Tuple
+from typing import Dict, Iterator, List, Optional, Tuple
 
 import torch
 
@@ -54,28 +54,30 @@ class ParamLayout:
             self.segments[name] = seg
             off = _round_up(off + seg.numel, ALIGN)
 
-        h, f, v = cfg.hidden_size, cfg.intermediate_size, cfg.vocab_size
-        start = off
-        add("embed", (v, h), 0)
-        add("final_norm", (h,), 0)
-        if not cfg.tie_word_embeddings:
-            add("lm_head", (v, h), 0)
-        off = _round_up(off, pad_to)
-        self.unit_ranges.append((start, off))
-        for i in range(cfg.num_hidden_layers):
+        for unit, tensors in enumerate(self._declare()):
             start = off
-            u = i + 1
-            add(f"layers.{i}.ln1", (h,), u)
-            add(f"layers.{i}.wqkv", (cfg.qkv_dim, h), u)
-            if cfg.attention_bias:
-                add(f"layers.{i}.bqkv", (cfg.qkv_dim,), u)
-            add(f"layers.{i}.wo", (h, cfg.q_dim), u)
-            add(f"layers.{i}.ln2", (h,), u)
-            add(f"layers.{i}.wgu", (2 * f, h), u)
-            add(f"layers.{i}.wd", (h, f), u)
+            for name, shape in tensors:
+                add(name, shape, unit)
             off = _round_up(off, pad_to)
             self.unit_ranges.append((start, off))
         self.total = off
+
+    def _declare(self) -> List[List[Tuple[str, Tuple[int, ...]]]]:
+        """(name, shape) of every tensor, unit by unit: unit 0 = embedding group, then one unit per decoder layer."""
+        cfg = self.cfg
+        h, f, v = cfg.hidden_size, cfg.intermediate_size, cfg.vocab_size
+        top = [("embed", (v, h)), ("final_norm", (h,))]
+        if not cfg.tie_word_embeddings:
+            top.append(("lm_head", (v, h)))
+        units = [top]
+        for i in range(cfg.num_hidden_layers):
+            p = f"layers.{i}."
+            unit = [(p + "ln1", (h,)), (p + "wqkv", (cfg.qkv_dim, h))]
+            if cfg.attention_bias:
+                unit.append((p + "bqkv", (cfg.qkv_dim,)))
+            unit += [(p + "wo", (h, cfg.q_dim)), (p + "ln2", (h,)), (p + "wgu", (2 * f, h)), (p + "wd", (h, f))]
+            units.append(unit)
+        return units
 
     # ---- views ----
     def view(self, flat: torch.Tensor, name: str) -> torch.Tensor:
@@ -105,6 +107,16 @@ class ParamLayout:
         return out
 
     # ---- init ----
+    def init_value(self, name: str) -> Optional[float]:
+        """Constant that a random init gives the tensor; None = drawn from N(0, initializer_range)."""
+        leaf = name.split(".")[-1]
+        if leaf in ("ln1", "ln2", "final_norm"):
+            return 1.0
+        return 0.0 if leaf == "bqkv" else None
+
+    def init_finish_(self, flat: torch.Tensor) -> None:
+        """Called at the end of a random init (a layout with padded tensors clears the padding here)."""
+
     def init_random_(self, flat: torch.Tensor, seed: int = 0) -> None:
         """N(0, initializer_range) weights, unit norm scales, zero biases; identical on every device."""
         gen = torch.Generator(device="cpu").manual_seed(seed)
@@ -112,11 +124,9 @@ class ParamLayout:
         std = self.cfg.initializer_range
         for name, seg in self.segments.items():
             dst = self.view(flat, name)
-            leaf = name.split(".")[-1]
-            if leaf in ("ln1", "ln2", "final_norm"):
-                dst.fill_(1.0)
-            elif leaf == "bqkv":
-                dst.zero_()
+            const = self.init_value(name)
+            if const is not None:
+                dst.fill_(const)
             else:
                 # generate in row blocks to bound host memory for large tables
                 rows = seg.shape[0]
@@ -125,6 +135,7 @@ class ParamLayout:
                     r1 = min(rows, r0 + step)
                     blk = torch.randn((r1 - r0,) + tuple(seg.shape[1:]), generator=gen, dtype=torch.float32) * std
                     dst[r0:r1].copy_(blk)
+        self.init_finish_(flat)
 
     def init_random_device_(self, flat: torch.Tensor, seed: int = 0) -> None:
         """Same distribution as ``init_random_`` generated on ``flat``'s device (fast for multi-billion-parameter
@@ -134,15 +145,19 @@ class ParamLayout:
         std = self.cfg.initializer_range
         for name, seg in self.segments.items():
             dst = flat[seg.offset: seg.offset + seg.numel]
-            leaf = name.split(".")[-1]
-            if leaf in ("ln1", "ln2", "final_norm"):
-                dst.fill_(1.0)
-            elif leaf == "bqkv":
-                dst.zero_()
+            const = self.init_value(name)
+            if const is not None:
+                dst.fill_(const)
             else:
                 dst.normal_(0.0, std, generator=gen)
+        self.init_finish_(flat)
 
     # ---- HF checkpoint boundary ----
+    def hf_shape(self, name: str, view: torch.Tensor) -> Tuple[int, ...]:
+        """Shape of the checkpoint tensor ``name`` whose place in the flat buffer is ``view`` (a layout that pads heads
+        hands out views with the heads as a dimension of their own; the checkpoint has them flattened)."""
+        return tuple(view.shape)
+
     def hf_items(self, flat: torch.Tensor) -> Iterator[Tuple[str, torch.Tensor]]:
         """Yield (hf_name, tensor view) pairs in HF naming; fused matrices are split into row ranges."""
         cfg = self.cfg
@@ -177,6 +192,6 @@ class ParamLayout:
         out = []
         meta = torch.empty(self.total, dtype=torch.bfloat16, device="meta")
         for name, t in self.hf_items(meta):
-            out.append((name, tuple(t.shape), "bfloat16"))
+            out.append((name, self.hf_shape(name, t), "bfloat16"))
         del probe
         return out

@@ -1,0 +1,183 @@
+"""Native executor of decoders whose layers are listed one by one: the kernels of one layer, in order.
+
+The executor owns no cache and no loop over steps: the engine hands it the residual stream, the paged keys and the
+convolution rings, and a ``StepBatch`` that says where every token row lives. The same layer code serves whole prompts,
+portions of prompts, mixed batches and decode steps; decode differs only in the kernels that are picked.
+
+A layer is four or five launches around two sublayers:
+  fused q | k | gate projection -> short convolution (+ key write) -> attention with mixed heads and gate ->
+  output projection whose epilogue is [norm of the output, residual add, norm ahead of the feed-forward] ->
+  gate/up projection with SwiGLU -> down projection with the same kind of epilogue.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Any, Dict, List, Optional, Sequence, Tuple
+
+import numpy as np
+import torch
+
+from .dezelorn import DezelornConfig
+from .layout import ParamLayout
+
+LOG2E = 1.4426950408889634
+TILE = 128  # query rows per attention tile
+
+
+@dataclass
+class StepBatch:
+    """Where the token rows of a step live. Decode steps (``rows`` None): row = slot, position = seq_lens - 1."""
+    T: int
+    block_tables: torch.Tensor
+    rows: Optional[torch.Tensor] = None      # [T, 4] int32: slot, position, first row of the segment, 0
+    row_end: Optional[torch.Tensor] = None   # [T] last row of the segment
+    tiles: Optional[torch.Tensor] = None     # [n, 4]: first row, rows, position of the first row, slot
+    seq_lens: Optional[torch.Tensor] = None
+    splits: int = 1
+
+
+def host_batch(segments: Sequence[Tuple[int, int, np.ndarray]]) -> Tuple[np.ndarray, int, int]:
+    """(slot, tokens already there, new tokens) per segment -> one int32 array [ids | row_end | rows | tiles], T, n_tiles."""
+    ids, ends, rows, tiles = [], [], [], []
+    t0 = 0
+    for slot, past, toks in segments:
+        n = len(toks)
+        ids.append(np.asarray(toks, dtype=np.int32))
+        ends.append(np.full(n, t0 + n - 1, np.int32))
+        r = np.zeros((n, 4), np.int32)
+        r[:, 0], r[:, 1], r[:, 2] = slot, past + np.arange(n), t0
+        rows.append(r)
+        tiles += [(t0 + a, min(TILE, n - a), past + a, slot) for a in range(0, n, TILE)]
+        t0 += n
+    tiles.sort(key=lambda t: -t[2])
+    tl = np.asarray(tiles, np.int32)
+    pad = (-2 * t0) % 4  # keeps the row table 16-byte aligned
+    flat = np.concatenate(ids + ends + [np.zeros(pad, np.int32)] + [r.ravel() for r in rows] + [tl.ravel()])
+    return flat, t0, len(tiles)
+
+
+def split_batch(flat: torch.Tensor, T: int, n_tiles: int, block_tables: torch.Tensor) -> Tuple[torch.Tensor, StepBatch]:
+    o = 2 * T + (-2 * T) % 4
+    return flat[:T], StepBatch(T, block_tables, rows=flat[o:o + 4 * T].view(T, 4), row_end=flat[T:2 * T],
+                               tiles=flat[o + 4 * T:o + 4 * T + 4 * n_tiles].view(n_tiles, 4))
+
+
+class ListedDecoder:
+    def __init__(self, cfg: DezelornConfig, layout: ParamLayout, params: torch.Tensor, max_len: int):
+        from ..ops import native
+
+        self.C = native()
+        self.cfg, self.layout, self.params = cfg, layout, params
+        self.dev, self.dtype = params.device, params.dtype
+        self.fp32 = params.dtype == torch.float32
+        self.max_len = int(max_len)
+        self.status = torch.zeros(1, dtype=torch.int32, device=self.dev)
+        self.launches = 0
+        self._w: Dict[str, torch.Tensor] = {n: layout.view(params, n) for n in layout.segments}
+        self._norms: Dict[str, List[torch.Tensor]] = {}
+        self.refresh_tables()
+
+    def w(self, name: str) -> torch.Tensor:
+        return self._w[name]
+
+    def norm(self, name: str) -> List[torch.Tensor]:
+        n = self._norms.get(name)
+        if n is None:
+            n = self._norms[name] = [self._w[f"{name}.{p}"] for p in ("w", "b", "alpha")]
+        return n
+
+    def refresh_tables(self) -> None:
+        """Tables that follow from the configuration and the weights, computed in 64-bit: the distance bias of every head
+        (entry d = r1 ln(1 + r2 d)) and the score factor of a query at each position (scale x temperature), both in
+        log2 units. They keep their storage when the weights change, so captured graphs stay valid."""
+        if not hasattr(self, "bias"):
+            self.bias: List[torch.Tensor] = []
+            self.qscale: List[torch.Tensor] = []
+            shared: Dict[Tuple[float, float, float], torch.Tensor] = {}
+            for l in self.cfg.layers:
+                m = l.mixer
+                self.bias.append(torch.empty(m.heads, min(m.window, self.max_len), dtype=torch.float32, device=self.dev))
+                key = (m.temp_coef, m.temp_every, m.scale)
+                if key not in shared:
+                    p = torch.arange(self.max_len, dtype=torch.float64)
+                    temp = 1.0 + m.temp_coef * torch.log(torch.floor((p + 1.0) / m.temp_every) + 1.0)
+                    shared[key] = (temp * (m.scale * LOG2E)).float().to(self.dev)
+                self.qscale.append(shared[key])
+        for i, t in enumerate(self.bias):
+            d = torch.arange(t.shape[1], dtype=torch.float64, device=self.dev)
+            r1, r2 = self.w(f"layers.{i}.r1").double(), self.w(f"layers.{i}.r2").double()
+            t.copy_(r1[:, None] * torch.log1p(r2[:, None] * d[None]) * LOG2E)
+
+    def check_status(self) -> None:
+        code = int(self.status.item())
+        if code != 0:
+            self.status.zero_()
+            raise RuntimeError(f"device kernel reported status {code} (bounded wait ran out or bad index)")
+
+    def next_norm(self, i: int) -> str:
+        return f"layers.{i + 1}.norm1" if i + 1 < len(self.cfg.layers) else "final_norm"
+
+    # ---- pieces ----
+    def embed(self, ids: torch.Tensor, x: torch.Tensor, h: torch.Tensor) -> None:
+        self.C.embed_dyt(ids, self.w("embed"), self.cfg.embedding_scale, x, h, self.norm("layers.0.norm1"))
+        self.launches += 1
+
+    def _project(self, h: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+        if self.fp32:
+            self.C.gemm_f32(h, w, out)
+        else:
+            self.C.gemm_bf16(h, w, out, False, False, None, 1.0, False, self.status, None)
+        self.launches += 1
+
+    def _swiglu(self, h: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+        if self.fp32:
+            self.C.gemm_swiglu_f32(h, w, out)
+        else:
+            self.C.gemm_swiglu(h, w, out, None, 0.0, self.status)
+        self.launches += 1
+
+    def _close_sublayer(self, a: torch.Tensor, w: torch.Tensor, x: torch.Tensor, h: torch.Tensor, out_norm: str, next_norm: str) -> None:
+        """x += out_norm(a w^T); h = next_norm(x)."""
+        self.C.gemm_dyt(a, w, x, self.norm(out_norm), self.norm(next_norm), h, self.status)
+        self.launches += 1
+
+    def _attention(self, i: int, u: torch.Tensor, sb: StepBatch, k_cache: torch.Tensor, ring: torch.Tensor, q: torch.Tensor,
+                   out: torch.Tensor) -> None:
+        m, C, p = self.cfg.layers[i].mixer, self.C, f"layers.{i}."
+        gate = u[:, m.qk_dim:]
+        C.short_conv(u, self.w(p + "conv"), ring, sb.rows, sb.row_end, sb.seq_lens, sb.block_tables, q, k_cache, self.status)
+        C.window_attn(q, k_cache, sb.rows, sb.seq_lens, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate,
+                      m.window, out, self.status)
+        self.launches += 3
+
+    def layer(self, i: int, x: torch.Tensor, h: torch.Tensor, sb: StepBatch, k_cache: torch.Tensor, ring: torch.Tensor,
+              buf: Dict[str, torch.Tensor]) -> None:
+        """``x`` fp32 residual stream and ``h`` = norm1(x), both updated in place (``h`` to the next layer's norm)."""
+        l, p, T = self.cfg.layers[i], f"layers.{i}.", sb.T
+        m = l.mixer
+        u = buf["u"][:T * m.u_dim].view(T, m.u_dim)
+        q = buf["q"][:T * m.q_dim].view(T, m.q_dim)
+        a = buf["a"][:T * m.q_dim].view(T, m.q_dim)
+        self._project(h, self.w(p + "wqkg"), u)
+        self._attention(i, u, sb, k_cache, ring, q, a)
+        self._close_sublayer(a, self.w(p + "wo"), x, h, p + "norm1b", p + "norm2" if l.ff is not None else self.next_norm(i))
+        if l.ff is not None:
+            act = buf["act"][:T * l.ff_p].view(T, l.ff_p)
+            self._swiglu(h, self.w(p + "wgu"), act)
+            self._close_sublayer(act, self.w(p + "wd"), x, h, p + "norm2b", self.next_norm(i))
+
+    def buffers(self, T: int) -> Dict[str, torch.Tensor]:
+        ls = self.cfg.layers
+        dims = {"u": max(l.mixer.u_dim for l in ls), "q": max(l.mixer.q_dim for l in ls), "a": max(l.mixer.q_dim for l in ls),
+                "act": max(l.ff_p for l in ls)}
+        return {k: torch.empty(T * d, dtype=self.dtype, device=self.dev) for k, d in dims.items()}
+
+    def logits(self, h: torch.Tensor) -> torch.Tensor:
+        wl = self.w("lm_head")
+        out = torch.empty(h.shape[0], wl.shape[0], dtype=torch.float32, device=self.dev)
+        if self.fp32:
+            self.C.gemm_f32(h, wl, out)
+        else:
+            self.C.gemm_bf16(h, wl, out, False, False, None, 1.0, False, self.status, None)
+        self.launches += 1
+        return out
