@@ -137,6 +137,47 @@ void window_attn(const Tensor& q, const Tensor& k_cache, const OptTensor& rows, 
   agrpo::launch_window_attn(k_cache.scalar_type() == torch::kFloat32, a, cur_stream());
 }
 
+// Tensor-core form for prompts; false (nothing launched) when the shape is not served.
+bool talk_attn_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& tiles, const Tensor& block_tables, const Tensor& bias,
+                       const Tensor& qscale, const OptTensor& talk, const OptTensor& gate, int64_t window, Tensor& acc, Tensor& out,
+                       const OptTensor& status) {
+  if (k_cache.scalar_type() != torch::kBFloat16 || k_cache.size(2) != 16) return false;
+  check_i32(tiles, "tiles");
+  TORCH_CHECK(tiles.dim() == 2 && tiles.size(1) == 4 && tiles.is_contiguous() && aligned16(tiles), "talk_attn_prefill: tiles [n, 4]");
+  const agrpo::WindowAttnArgs a = attn_args(q, k_cache, OptTensor(), OptTensor(), block_tables, bias, qscale, talk, gate, window, out, status);
+  same_type(acc, false, "acc");
+  TORCH_CHECK(acc.is_contiguous() && acc.numel() >= (int64_t)a.T * a.H * a.G * a.D && aligned16(acc), "talk_attn_prefill: acc [T, H, G, D]");
+  const c10::cuda::CUDAGuard guard(k_cache.device());
+  return agrpo::launch_talk_attn_prefill(a, tiles.data_ptr<int>(), (int)tiles.size(0), acc.data_ptr(), cur_stream());
+}
+
+// Decode step of a mixer after its fused projection u = [q | k | gate]: convolution, attention, mixing, gate, state update.
+void talk_attn_decode(const Tensor& u, const Tensor& conv_w, Tensor& ring, Tensor& k_cache, const Tensor& seq_lens, const Tensor& block_tables,
+                      const Tensor& bias, const Tensor& qscale, const OptTensor& talk, const OptTensor& gate, int64_t window, Tensor& out,
+                      int64_t splits, Tensor& part_o, Tensor& part_ml, Tensor& tickets, const OptTensor& status) {
+  TORCH_CHECK(k_cache.scalar_type() == torch::kBFloat16, "talk_attn_decode: bf16");
+  agrpo::TalkDecodeArgs d{};
+  d.at = attn_args(OptTensor(), k_cache, OptTensor(), seq_lens, block_tables, bias, qscale, talk, gate, window, out, status);
+  const int64_t C = (int64_t)(d.at.H + d.at.G) * d.at.D, B = d.at.T;
+  same_type(u, false, "u"); same_type(conv_w, false, "conv_w"); same_type(ring, false, "ring"); rows2d(u, "u");
+  check_f32(part_o, "part_o"); check_f32(part_ml, "part_ml"); check_i32(tickets, "tickets");
+  TORCH_CHECK(u.size(0) >= B && u.size(1) >= C && u.stride(0) % 8 == 0 && aligned16(u), "talk_attn_decode: u");
+  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == C && conv_w.is_contiguous(), "talk_attn_decode: conv_w [q + k channels, taps]");
+  TORCH_CHECK(ring.dim() == 3 && ring.size(0) >= B && ring.size(1) == conv_w.size(1) && ring.size(2) == C && ring.stride(2) == 1 &&
+              ring.stride(1) == C && ring.stride(0) % 8 == 0 && aligned16(ring), "talk_attn_decode: ring [slots, taps, channels]");
+  TORCH_CHECK(splits >= 1 && splits <= 8, "talk_attn_decode: 1 to 8 splits");
+  TORCH_CHECK(splits == 1 || (part_o.numel() >= B * splits * d.at.H * d.at.G * d.at.D && part_ml.numel() >= B * splits * d.at.H * 2 &&
+              tickets.numel() >= B), "talk_attn_decode: scratch");
+  d.u = u.data_ptr(); d.ldu = u.stride(0);
+  d.conv_w = conv_w.data_ptr(); d.taps = (int)conv_w.size(1);
+  d.ring = ring.data_ptr(); d.ring_len = (int)ring.size(1); d.ring_pitch = ring.stride(0);
+  d.k_cache = k_cache.data_ptr();
+  d.splits = (int)splits;
+  d.part_o = part_o.data_ptr<float>(); d.part_ml = part_ml.data_ptr<float>(); d.tickets = tickets.data_ptr<int>();
+  const c10::cuda::CUDAGuard guard(k_cache.device());
+  agrpo::launch_talk_attn_decode(d, cur_stream());
+}
+
 // D = A . B^T + the sublayer tail; fp32 operands run the true-fp32 kernel
 void gemm_dyt(const Tensor& a, const Tensor& b, Tensor& x, const std::vector<Tensor>& n1, const std::vector<Tensor>& n2, Tensor& h,
               const OptTensor& status, int64_t num_sms) {
@@ -196,6 +237,12 @@ void bind_layer_ops(pybind11::module_& m) {
         py::arg("block_tables"), py::arg("q_out"), py::arg("k_cache"), py::arg("status"), NoGil());
   m.def("window_attn", &window_attn, py::arg("q"), py::arg("k_cache"), py::arg("rows"), py::arg("seq_lens"), py::arg("block_tables"),
         py::arg("bias"), py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("out"), py::arg("status"), NoGil());
+  m.def("talk_attn_prefill", &talk_attn_prefill, py::arg("q"), py::arg("k_cache"), py::arg("tiles"), py::arg("block_tables"), py::arg("bias"),
+        py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("acc"), py::arg("out"), py::arg("status"), NoGil());
+  m.def("talk_attn_decode", &talk_attn_decode, py::arg("u"), py::arg("conv_w"), py::arg("ring"), py::arg("k_cache"), py::arg("seq_lens"),
+        py::arg("block_tables"), py::arg("bias"), py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("out"),
+        py::arg("splits"), py::arg("part_o"), py::arg("part_ml"), py::arg("tickets"), py::arg("status"), NoGil());
+  m.def("talk_decode_supported", &agrpo::talk_decode_supported);
   m.def("gemm_dyt", &gemm_dyt, py::arg("a"), py::arg("b"), py::arg("x"), py::arg("n1"), py::arg("n2"), py::arg("h"), py::arg("status"),
         py::arg("num_sms") = 0, NoGil());
   m.def("gemm_f32", &gemm_f32, NoGil());

@@ -43,6 +43,10 @@ struct DytResidualEpilogue {
 void launch_gemm_dyt_bf16(const void* a, long long lda, const void* b, long long ldb, int M, int N, int K, float* x, long long ldx, void* h,
                           long long ldh, const DytArgs& n1, const DytArgs& n2, int* status, int num_sms, cudaStream_t s) {
   if (M == 0 || N == 0) return;
+  const DytTail tail{x, ldx, h, ldh, n1, n2};
+  if (M <= 256 && launch_gemm_skinny(a, lda, b, ldb, nullptr, 0, M, N, K, nullptr, nullptr, 0, status, num_sms, s, nullptr, nullptr, nullptr, 0.f,
+                                     nullptr, &tail))
+    return;
   const int tiles_m = (M + kGemmBM - 1) / kGemmBM;
   const int cands[3] = {256, 128, 64};
   int BN = 32;

@@ -21,6 +21,8 @@
 #include "../common/ptx.cuh"
 #include "../common/tensormap.h"
 #include "../launchers.h"
+#include "../launchers_layers.h"
+#include "layer_ops.cuh"
 
 namespace agrpo {
 
@@ -47,9 +49,19 @@ struct SkRope {
   int Hq, Hkv, block_size, num_cache_blocks;
 };
 
+// Optional sublayer tail instead of a plain store: x += norm1(result) on the fp32 residual, h = norm2(x).
+struct SkTail {
+  float* x;              // nullptr = off
+  long long ldx;
+  __nv_bfloat16* h;
+  long long ldh;
+  DytNorm<__nv_bfloat16> n1, n2;
+};
+
 struct SkParams {
   int M, N, K;
   SkRope rope;
+  SkTail tail;
   __nv_bfloat16* D;
   long long ldd;
   const __nv_bfloat16* bias;
@@ -416,6 +428,11 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
           if (row < p.M && col < p.N) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) acc[i] *= rs;
+            if (p.tail.x != nullptr) {  // N is a multiple of 8 in this mode
+              dyt_residual8(acc, p.tail.x + (long long)row * p.tail.ldx + col, p.tail.h + (long long)row * p.tail.ldh + col, p.tail.n1,
+                            p.tail.n2, col, ldf(p.tail.n1.alpha), ldf(p.tail.n2.alpha));
+              continue;
+            }
             if (p.bias != nullptr) {
 #pragma unroll
               for (int i = 0; i < 8; ++i)
@@ -497,7 +514,8 @@ int gemm_skinny_splits(int M, int N, int K, int num_sms) {
 // Returns false when the shape is not one this kernel serves (the caller then uses the general GEMM).
 bool launch_gemm_skinny(const void* a, long long lda, const void* b, long long ldb, void* d, long long ldd, int M, int N, int K,
                         const void* bias, const void* residual, long long ldr, int* status, int num_sms, cudaStream_t stream,
-                        long long* trace, const long long* ss_in, long long* ss_out, float eps, const DecodeRopeArgs* rope) {
+                        long long* trace, const long long* ss_in, long long* ss_out, float eps, const DecodeRopeArgs* rope,
+                        const DytTail* tail) {
   const int S = gemm_skinny_splits(M, N, K, num_sms);
   if (S == 0) return false;
   if (rope != nullptr) {
@@ -519,6 +537,16 @@ bool launch_gemm_skinny(const void* a, long long lda, const void* b, long long l
   p.residual = reinterpret_cast<const __nv_bfloat16*>(residual);
   p.ldr = ldr;
   p.rope = SkRope{};
+  p.tail = SkTail{};
+  if (tail != nullptr) {
+    typedef const __nv_bfloat16* P;
+    p.tail.x = tail->x;
+    p.tail.ldx = tail->ldx;
+    p.tail.h = reinterpret_cast<__nv_bfloat16*>(tail->h);
+    p.tail.ldh = tail->ldh;
+    p.tail.n1 = {(P)tail->n1.w, (P)tail->n1.b, (P)tail->n1.alpha};
+    p.tail.n2 = {(P)tail->n2.w, (P)tail->n2.b, (P)tail->n2.alpha};
+  }
   if (rope != nullptr) {
     p.rope.enabled = 1;
     p.rope.cos_t = rope->cos_t; p.rope.sin_t = rope->sin_t; p.rope.max_pos = rope->max_pos;

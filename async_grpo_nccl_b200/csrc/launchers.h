@@ -150,7 +150,8 @@ struct DecodeRopeArgs {
 bool launch_gemm_skinny(const void* a, long long lda, const void* b, long long ldb, void* d, long long ldd, int M, int N, int K,
                         const void* bias, const void* residual, long long ldr, int* status, int num_sms, cudaStream_t stream,
                         long long* trace = nullptr, const long long* ss_in = nullptr, long long* ss_out = nullptr, float eps = 0.f,
-                        const DecodeRopeArgs* rope = nullptr);
+                        const DecodeRopeArgs* rope = nullptr,
+                        const struct DytTail* tail = nullptr);
 int gemm_skinny_splits(int M, int N, int K, int num_sms);
 
 // ---- bandwidth-bound decoder ops (elementwise.cu); bf16 activations, H and F multiples of 8 ----

@@ -11,6 +11,15 @@ struct DytArgs {  // tanh(alpha x) * w + b
   const void* alpha;
 };
 
+// Tail of a sublayer, fused into the GEMM that produces its output: x += n1(output) (fp32 residual), h = n2(x).
+struct DytTail {
+  float* x;
+  long long ldx;
+  void* h;
+  long long ldh;
+  DytArgs n1, n2;
+};
+
 // x[t] = table[ids[t]] * scale (fp32), h[t] = norm(x[t])
 void launch_embed_dyt(bool fp32, const int* ids, const void* table, float scale, float* x, void* h, const DytArgs& norm, int T, int W, int V,
                       cudaStream_t s);

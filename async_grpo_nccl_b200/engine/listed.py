@@ -64,7 +64,13 @@ class ListedEngine(RolloutEngine):
         S, W = self.max_seqs, self.cfg.hidden_size
         self.b_x = torch.zeros(S, W, dtype=torch.float32, device=self.dev)
         self.b_h = torch.zeros(S, W, dtype=self.dtype, device=self.dev)
-        self.b_buf = self.dec.buffers(S)
+        self.b_buf = {k: t.zero_() for k, t in self.dec.buffers(S).items()}  # idle rows hold numbers, not garbage
+        self.max_splits = 8
+        ms = [l.mixer for l in self.cfg.layers]
+        f32 = dict(dtype=torch.float32, device=self.dev)
+        self.b_scratch = (torch.empty(S * self.max_splits * max(m.heads * m.k_dim for m in ms), **f32),
+                          torch.empty(S * self.max_splits * max(m.heads for m in ms) * 2, **f32),
+                          torch.zeros(S, dtype=torch.int32, device=self.dev))
         self.b_logits = torch.empty(S, self.cfg.vocab_size, dtype=torch.float32, device=self.dev) if self.dec.fp32 else None
 
     def _weights_changed(self) -> None:
@@ -150,7 +156,7 @@ class ListedEngine(RolloutEngine):
         self._feed_back(B)
 
     def _decode_layers(self, B: int, splits: int) -> None:
-        sb = StepBatch(B, self.block_tables, seq_lens=self.seq_lens, splits=splits)
+        sb = StepBatch(B, self.block_tables, seq_lens=self.seq_lens, splits=splits, scratch=self.b_scratch)
         self.C.set_pdl(self.use_pdl)  # this thread only: prologues overlap the tail of the kernel before
         try:
             self._layers(self.last_tokens[:B], self.b_x[:B], self.b_h[:B], sb, self.b_buf)
@@ -158,10 +164,15 @@ class ListedEngine(RolloutEngine):
             self.C.set_pdl(False)
 
     def _choose_splits(self, B: int, n_active: int, max_len: int) -> int:
-        return 1
+        """Two CTAs per SM where there are few sequences, each with at least two tiles of 64 keys."""
+        want = (self.sm_count * 2) // max(1, n_active)
+        return int(max(1, min(self.max_splits, want, min(max_len, self.cfg.max_window) // 128)))
 
     def _launch_count_decode(self, splits: int, B: int = 0) -> int:
-        return 1 + sum(5 if l.ff is None else 7 for l in self.cfg.layers) + 2
+        n = 1 + 2
+        for i, l in enumerate(self.cfg.layers):
+            n += (3 if self.dec.tensor_core_decode(i) else 5) + (0 if l.ff is None else 2)
+        return n
 
     # ------------------------------------------------------------------ step-wise driving
     def open_sequence(self) -> int:

@@ -34,6 +34,7 @@ class StepBatch:
     tiles: Optional[torch.Tensor] = None     # [n, 4]: first row, rows, position of the first row, slot
     seq_lens: Optional[torch.Tensor] = None
     splits: int = 1
+    scratch: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None  # decode: partial products, (max, sum), tickets
 
 
 def host_batch(segments: Sequence[Tuple[int, int, np.ndarray]]) -> Tuple[np.ndarray, int, int]:
@@ -114,6 +115,10 @@ class ListedDecoder:
             self.status.zero_()
             raise RuntimeError(f"device kernel reported status {code} (bounded wait ran out or bad index)")
 
+    def tensor_core_decode(self, i: int) -> bool:
+        m = self.cfg.layers[i].mixer
+        return not self.fp32 and self.C.talk_decode_supported(m.heads, m.kv_heads, m.dim_p)
+
     def next_norm(self, i: int) -> str:
         return f"layers.{i + 1}.norm1" if i + 1 < len(self.cfg.layers) else "final_norm"
 
@@ -145,7 +150,18 @@ class ListedDecoder:
                    out: torch.Tensor) -> None:
         m, C, p = self.cfg.layers[i].mixer, self.C, f"layers.{i}."
         gate = u[:, m.qk_dim:]
+        if sb.rows is None and sb.scratch is not None and self.tensor_core_decode(i):
+            C.talk_attn_decode(u, self.w(p + "conv"), ring, k_cache, sb.seq_lens, sb.block_tables, self.bias[i], self.qscale[i],
+                               self.w(p + "talk"), gate, m.window, out, sb.splits, *sb.scratch, self.status)
+            self.launches += 1
+            return
         C.short_conv(u, self.w(p + "conv"), ring, sb.rows, sb.row_end, sb.seq_lens, sb.block_tables, q, k_cache, self.status)
+        if sb.rows is not None and not self.fp32:
+            acc = torch.empty(sb.T * m.heads * m.k_dim, dtype=self.dtype, device=self.dev)
+            if C.talk_attn_prefill(q, k_cache, sb.tiles, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate, m.window,
+                                   acc, out, self.status):
+                self.launches += 4
+                return
         C.window_attn(q, k_cache, sb.rows, sb.seq_lens, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate,
                       m.window, out, self.status)
         self.launches += 3

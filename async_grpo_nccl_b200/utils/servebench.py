@@ -1,0 +1,247 @@
+"""Serving throughput of a listed-layer design beside the dense model of equal size, and the kernels behind it.
+
+    python bench.py --serving dezelorn-1.5b:qwen2.5-1.5b,dezelorn-7b:qwen2.5-7b
+
+Random weights, synthetic prompts. Prefill: prompts of ``--serving-prompt`` tokens through the engine's own prompt step;
+decode: the engine's captured decode step. Times are CUDA events on the launching stream after warm-up; kernel times are
+medians with the L2 flushed (a buffer larger than L2 is written) between iterations. One JSON line per record.
+"""
+from __future__ import annotations
+
+import json
+import os
+from typing import Any, Callable, Dict, List, Tuple
+
+import numpy as np
+import torch
+
+from .microbench import flush_l2, timeit
+
+
+def peaks() -> Dict[str, Any]:
+    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    for p in (os.environ.get("AGRPO_PEAKS_FILE"), os.path.join(root, "MEASURED_PEAKS.json")):
+        if p and os.path.exists(p):
+            with open(p) as f:
+                d = json.load(f)
+            return {"hbm_gbs": float(d["hbm_gbs"]), "bf16_tflops": float(d["bf16_tflops"]), "source": "measured"}
+    return {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+
+
+def out(rec: Dict[str, Any]) -> None:
+    print(json.dumps(rec), flush=True)
+
+
+def make_engine(model: str, max_seqs: int, max_len: int, n_layers: int, blocks: int, **kw: Any) -> Any:
+    """Engine on the first ``n_layers`` layers of a preset (a stack of equal layers: time per layer does not depend on how many)."""
+    from dataclasses import replace
+
+    from ..models.registry import architecture_of, build_engine, make_layout, resolve_model_config
+
+    cfg = resolve_model_config(model)
+    if architecture_of(cfg).name == "dense":
+        cfg = replace(cfg, num_hidden_layers=n_layers)
+    else:
+        cfg = replace(cfg, layers=cfg.layers[:n_layers])
+    layout = make_layout(cfg)
+    params = torch.empty(layout.total, dtype=torch.bfloat16, device="cuda")
+    layout.init_random_device_(params, 0)
+    return cfg, build_engine(cfg, layout, params, max_seqs=max_seqs, max_model_len=max_len, num_blocks=blocks, use_cuda_graph=True,
+                             max_prefill_tokens=1 << 20, **kw)
+
+
+def bench_prefill(model: str, prompt: int, n_prompts: int, n_layers: int, iters: int = 5) -> Dict[str, Any]:
+    max_len = prompt + 32
+    cfg, eng = make_engine(model, 32, max_len, n_layers, n_prompts * (prompt // 16 + 4) + 64)
+    rng = np.random.default_rng(0)
+    times = []
+    for it in range(iters + 3):
+        for i in range(n_prompts):
+            eng.add_request((it, i), rng.integers(0, cfg.vocab_size, prompt).astype(np.int32), n=1, max_new_tokens=1, temperature=0.0,
+                            ignore_eos=True)
+        eng._admit_pending()
+        plan = eng.sched.plan_prefill()
+        assert len(plan["group_ids"]) == n_prompts
+        reqs = [eng.requests[g] for g in plan["group_ids"]]
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        eng._prompt_hidden(plan, reqs)
+        e1.record()
+        torch.cuda.synchronize()
+        if it >= 3:
+            times.append(e0.elapsed_time(e1))
+        for s in plan["seq_ids"]:
+            eng.sched.finish(s)
+    eng.check_status()
+    ms = sorted(times)[len(times) // 2]
+    return {"bench": "prefill", "model": model, "layers": n_layers, "prompts": n_prompts, "prompt_len": prompt, "ms": round(ms, 3),
+            "tokens_per_s": round(prompt * n_prompts / ms * 1e3), "us_per_layer": round(ms * 1e3 / n_layers, 1)}
+
+
+def bench_decode(model: str, batch: int, context: int, n_layers: int, steps: int = 40) -> Dict[str, Any]:
+    max_len = context + steps + 64
+    cfg, eng = make_engine(model, max(32, batch), max_len, n_layers, batch * (max_len // 16 + 2) + 256)
+    rng = np.random.default_rng(0)
+    for i in range(batch):
+        eng.add_request(i, rng.integers(0, cfg.vocab_size, context).astype(np.int32), n=1, max_new_tokens=steps + 16, temperature=1.0, seed=i,
+                        forced_new_tokens=[steps + 16])
+    while eng.sched.num_waiting > 0 or eng.pending:
+        eng.step()
+    for _ in range(4):
+        eng.step()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(steps):
+        eng.step()
+    e1.record()
+    torch.cuda.synchronize()
+    eng.check_status()
+    ms = e0.elapsed_time(e1) / steps
+    return {"bench": "decode", "model": model, "layers": n_layers, "batch": batch, "context": context, "ms_per_step": round(ms, 4),
+            "tokens_per_s": round(batch / ms * 1e3)}
+
+
+def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> List[Tuple[str, str, Callable[[], Any], float, float]]:
+    """(phase / role, side, launch, FLOPs, bytes) of like kernels of one layer: ``new`` a listed-layer configuration, ``old`` the
+    dense one. FLOPs count what the operation needs, not what a kernel spends (scores and one product per pair)."""
+    from ..ops import native
+    from .microbench import _tiles
+    from ..models.listed import host_batch, split_batch
+
+    C = native()
+    bf, dev = torch.bfloat16, "cuda"
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    m = new.layers[0].mixer
+    W, F, H, G, D = new.hidden_size, new.layers[0].ff_p, m.heads, m.kv_heads, m.dim_p
+    R = lambda *s: torch.randn(*s, device=dev).to(bf)
+    Wr = lambda *s: (torch.randn(*s, device=dev) * 0.02).to(bf)
+    cases: List[Tuple[str, str, Callable[[], Any], float, float]] = []
+
+    def add(role: str, side: str, fn: Callable[[], Any], flops: float, nbytes: float) -> None:
+        cases.append((role, side, fn, flops, nbytes))
+
+    n_seq = T // prompt
+    wqkg, wqkv, wo, wgu, wd = Wr(m.u_dim, W), Wr(old.qkv_dim, W), Wr(W, H * D), Wr(2 * F, W), Wr(W, F)
+    nrm = [torch.ones(W, device=dev, dtype=bf), torch.zeros(W, device=dev, dtype=bf), torch.full((1,), 0.5, device=dev, dtype=bf)]
+    ln = torch.ones(W, device=dev, dtype=bf)
+    maxlen = max(prompt, ctx) + 64
+    bias = torch.rand(H, min(m.window, maxlen), device=dev)
+    qscale = torch.full((maxlen,), 0.1, device=dev)
+    talk = (torch.eye(H, device=dev) + 0.02 * torch.randn(H, H, device=dev)).to(bf)
+    conv = R(m.qk_dim, m.conv)
+
+    # ---------------- prompts ----------------
+    h, x, ho = R(T, W), torch.randn(T, W, device=dev), torch.empty(T, W, device=dev, dtype=bf)
+    xb, xb2 = R(T, W), torch.empty(T, W, device=dev, dtype=bf)
+    u, qkv = R(T, m.u_dim), R(T, old.qkv_dim)
+    a, act, gu = R(T, H * D), torch.empty(T, F, device=dev, dtype=bf), torch.empty(T, 2 * F, device=dev, dtype=bf)
+    q = R(T, H * D)
+    nb = (prompt + 15) // 16
+    cache = R(n_seq * nb, G, 16, D)
+    tables = torch.randperm(n_seq * nb, device=dev).int().view(n_seq, nb).contiguous()
+    ring = torch.zeros(max(n_seq, B), m.conv, m.qk_dim, device=dev, dtype=bf)
+    flat, T2, nt = host_batch([(i, 0, np.zeros(prompt, np.int32)) for i in range(n_seq)])
+    _, sb = split_batch(torch.from_numpy(flat).to(dev), T2, nt, tables)
+    acc = torch.empty(T * H * G * D, device=dev, dtype=bf)
+    lse = torch.empty(H, T, device=dev)
+    tiles = _tiles([prompt] * n_seq)
+    pairs = n_seq * sum(min(i + 1, m.window) for i in range(prompt))
+    pairs_old = n_seq * prompt * (prompt + 1) / 2
+    gm = lambda M, N, K: (2.0 * M * N * K, 2.0 * (M * K + N * K + M * N))
+    add("prompt projection", "new", lambda: C.gemm_bf16(h, wqkg, u, False, False, None, 1.0, False, st, None), *gm(T, m.u_dim, W))
+    add("prompt projection", "old", lambda: C.gemm_bf16(h, wqkv, qkv, False, False, None, 1.0, False, st, None), *gm(T, old.qkv_dim, W))
+    add("prompt position op", "new", lambda: C.short_conv(u, conv, ring, sb.rows, sb.row_end, None, tables, q, cache, st), 0.0, 4.0 * T * m.qk_dim)
+    pos = torch.arange(T, device=dev, dtype=torch.int32) % prompt
+    cos = torch.rand(maxlen, D // 2, device=dev)
+    slots = torch.arange(T, device=dev, dtype=torch.int32)
+    kc, vc = torch.zeros(n_seq * nb, G, 16, D, device=dev, dtype=bf), torch.zeros(n_seq * nb, G, 16, D, device=dev, dtype=bf)
+
+    def rope():
+        C.rope_inplace(qkv, pos, cos, cos, H + G, D, False)
+        C.kv_cache_write(qkv, slots, kc, vc, H, G, D, st, 0)
+    add("prompt position op", "old", rope, 0.0, 4.0 * T * (H + G) * D + 8.0 * T * G * D)
+    add("prompt attention", "new", lambda: C.talk_attn_prefill(q, cache, sb.tiles, tables, bias, qscale, talk, u[:, m.qk_dim:], m.window, acc, a, st),
+        4.0 * pairs * H * D, 0.0)
+    add("prompt attention", "old", lambda: C.attn_varlen_fwd(qkv, a, lse, tiles, H, G, D, 0.1, st), 4.0 * pairs_old * H * D, 0.0)
+    add("prompt out projection + tail", "new", lambda: C.gemm_dyt(a, wo, x, nrm, nrm, ho, st), *gm(T, W, H * D))
+
+    def wo_old():
+        C.gemm_bf16(a, wo, xb2, False, False, None, 1.0, False, st, xb)
+        C.rmsnorm_fwd(xb2, ln, ho, None, 1e-6)
+    add("prompt out projection + tail", "old", wo_old, *gm(T, W, H * D))
+    add("prompt gate/up", "new", lambda: C.gemm_swiglu(ho, wgu, act, None, 0.0, st), *gm(T, 2 * F, W))
+
+    def gu_old():
+        C.gemm_bf16(ho, wgu, gu, False, False, None, 1.0, False, st, None)
+        C.swiglu_fwd(gu, act)
+    add("prompt gate/up", "old", gu_old, *gm(T, 2 * F, W))
+    add("prompt down + tail", "new", lambda: C.gemm_dyt(act, wd, x, nrm, nrm, ho, st), *gm(T, W, F))
+
+    def wd_old():
+        C.gemm_bf16(act, wd, xb2, False, False, None, 1.0, False, st, xb)
+        C.rmsnorm_fwd(xb2, ln, ho, None, 1e-6)
+    add("prompt down + tail", "old", wd_old, *gm(T, W, F))
+
+    # ---------------- decode ----------------
+    nbd = (ctx + 15) // 16 + 1
+    dcache, dk, dv = R(B * nbd, G, 16, D), R(B * nbd, G, 16, D), R(B * nbd, G, 16, D)
+    dtab = torch.randperm(B * nbd, device=dev).int().view(B, nbd).contiguous()
+    lens = torch.full((B,), ctx, device=dev, dtype=torch.int32)
+    hb, ub, qb = R(B, W), R(B, m.u_dim), R(B, old.qkv_dim)
+    ab, actb, xbd, hob = R(B, H * D), R(B, F), torch.randn(B, W, device=dev), torch.empty(B, W, device=dev, dtype=bf)
+    part_o, part_ml = torch.empty(B * 8 * H * G * D, device=dev), torch.empty(B * 8 * H * G * 16, device=dev)
+    tick = torch.zeros(B * G, device=dev, dtype=torch.int32)
+    n_sm = torch.cuda.get_device_properties(0).multi_processor_count
+    seen = min(ctx, m.window)
+    sp_new = max(1, min(8, 2 * n_sm // B, seen // 128))
+    sp_old = max(1, min(8, 3 * n_sm // (B * G), ctx // 256))
+    wb = lambda N, K, extra=0: 2.0 * N * K + 2.0 * B * (N + K) + extra
+    ss = torch.full((B,), W << 30, device=dev, dtype=torch.int64)
+    add("decode projection", "new", lambda: C.gemm_bf16(hb, wqkg, ub, False, False, None, 1.0, False, st, None), 0.0, wb(m.u_dim, W))
+    add("decode projection", "old", lambda: C.gemm_decode(hb, wqkv, qb, None, None, ss, None, 1e-6, st), 0.0, wb(old.qkv_dim, W))
+    add("decode attention", "new", lambda: C.talk_attn_decode(ub, conv, ring[:B], dcache, lens, dtab, bias, qscale, talk, ub[:, m.qk_dim:],
+                                                              m.window, ab, sp_new, part_o, part_ml, tick, st), 0.0, 2.0 * B * seen * G * D)
+    add("decode attention", "old", lambda: C.paged_decode_attn(qb, dk, dv, dtab, lens, ab, H, G, D, 0.1, sp_old, part_o, part_ml, st, tick),
+        0.0, 4.0 * B * ctx * G * D)
+    add("decode out projection + tail", "new", lambda: C.gemm_dyt(ab, wo, xbd, nrm, nrm, hob, st), 0.0, wb(W, H * D, 12 * B * W))
+    so = torch.zeros(B, device=dev, dtype=torch.int64)
+    xs = R(B, W)
+    add("decode out projection + tail", "old", lambda: C.gemm_decode(ab, wo, hob, None, xs, None, so, 1e-6, st), 0.0, wb(W, H * D, 4 * B * W))
+    add("decode gate/up", "new", lambda: C.gemm_swiglu(hb, wgu, actb, None, 0.0, st), 0.0, wb(2 * F, W))
+    add("decode gate/up", "old", lambda: C.gemm_swiglu(hb, wgu, actb, ss, 1e-6, st), 0.0, wb(2 * F, W))
+    add("decode down + tail", "new", lambda: C.gemm_dyt(actb, wd, xbd, nrm, nrm, hob, st), 0.0, wb(W, F, 12 * B * W))
+    add("decode down + tail", "old", lambda: C.gemm_decode(actb, wd, hob, None, xs, None, so, 1e-6, st), 0.0, wb(W, F, 4 * B * W))
+    return cases
+
+
+def bench_kernels(new_name: str, old_name: str, T: int, prompt: int, B: int, ctx: int) -> None:
+    from ..models.registry import PRESETS
+
+    pk = peaks()
+    res: Dict[str, Dict[str, Dict[str, float]]] = {}
+    for role, side, fn, flops, nbytes in kernel_cases(PRESETS[new_name], PRESETS[old_name], T, prompt, B, ctx):
+        ms = timeit(fn, iters=10, flush=True)
+        bound = max(flops / (pk["bf16_tflops"] * 1e9), nbytes / (pk["hbm_gbs"] * 1e6))  # ms
+        res.setdefault(role, {})[side] = {"us": round(ms * 1e3, 1), "of_roofline": round(bound / ms, 3)}
+    for role, r in res.items():
+        out({"bench": "kernel", "pair": f"{new_name}:{old_name}", "shape": f"T={T} prompt={prompt}" if role.startswith("prompt") else f"B={B} ctx={ctx}",
+             "role": role, "new": r["new"], "old": r["old"], "distance_ratio": round(r["old"]["of_roofline"] / r["new"]["of_roofline"], 2),
+             "peaks": pk["source"]})
+
+
+def run(pairs: str, prompt: int = 4096, n_layers: int = 8, kernels: bool = True) -> None:
+    for pair in pairs.split(","):
+        new, _, old = pair.partition(":")
+        for model in (new, old):
+            out(bench_prefill(model, prompt, max(1, 16384 // prompt), n_layers))
+            torch.cuda.empty_cache()
+        for batch, ctx in ((16, 2048), (64, 2048), (256, 1024)):
+            for model in (new, old):
+                out(bench_decode(model, batch, ctx, n_layers))
+                torch.cuda.empty_cache()
+        if kernels:
+            for B, ctx in ((16, 4096), (128, 2048)):
+                bench_kernels(new, old, 16384, prompt, B, ctx)
+                torch.cuda.empty_cache()

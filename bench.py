@@ -62,6 +62,11 @@ def parse_args():
                     help="consecutive rollout ranks that form one tensor-parallel engine replica (1 = every rank a replica)")
     ap.add_argument("--placement", default=None, help='JSON role placement overriding the default, e.g. '
                     '\'{"trainer": [0, 1], "logprob": [0], "rollout": [1]}\'')
+    ap.add_argument("--serving", default=None, metavar="NEW:OLD[,NEW:OLD...]",
+                    help="instead of the headline workload: prefill and decode throughput of the listed-layer preset NEW beside the dense "
+                         "preset OLD of equal size, and their like kernels against the roofline, e.g. dezelorn-1.5b:qwen2.5-1.5b")
+    ap.add_argument("--serving-prompt", type=int, default=4096)
+    ap.add_argument("--serving-layers", type=int, default=8, help="layers of each preset that are built")
     # reference arm only (its own defaults: orchestrator.py:137, 158 of the reference)
     ap.add_argument("--ref-max-num-seqs", type=int, default=512, help="vLLM max_num_seqs of the reference arm (its default)")
     ap.add_argument("--ref-loss-chunksize", type=int, default=None, help="loss_chunksize of the reference arm (its default: none)")
@@ -151,6 +156,14 @@ def main() -> None:
     args = parse_args()
     if args.impl == "reference":
         reference_arm(args)
+        return
+    if args.serving:
+        from async_grpo_nccl_b200.utils.servebench import run
+
+        sampler = ClockSampler()
+        sampler.start()
+        run(args.serving, args.serving_prompt, args.serving_layers)
+        print(json.dumps({"bench": "clocks", **sampler.stop()}))
         return
     import torch
 
