@@ -79,14 +79,15 @@ agrpo::ShortConvArgs conv_args(const Tensor& u, const Tensor& w, Tensor& ring, c
   return a;
 }
 
-void short_conv(const Tensor& u, const Tensor& w, Tensor& ring, const OptTensor& rows, const OptTensor& row_end, const OptTensor& seq_lens,
+void short_conv(const Tensor& u, const Tensor& w, Tensor& ring, const OptTensor& rows, const OptTensor& ring_rows, const OptTensor& seq_lens,
                 const Tensor& block_tables, Tensor& q_out, Tensor& k_cache, const OptTensor& status) {
   const agrpo::ShortConvArgs a = conv_args(u, w, ring, rows, seq_lens, block_tables, q_out, k_cache, status);
   const bool f = u.scalar_type() == torch::kFloat32;
-  if (given(rows)) { TORCH_CHECK(given(row_end), "short_conv: row_end with rows"); check_i32(*row_end, "row_end"); TORCH_CHECK(row_end->numel() >= a.T, "row_end [T]"); }
+  if (given(rows)) { TORCH_CHECK(given(ring_rows) && ring_rows->is_contiguous(), "short_conv: ring_rows with rows"); check_i32(*ring_rows, "ring_rows"); }
   const c10::cuda::CUDAGuard guard(u.device());
   agrpo::launch_short_conv(f, a, cur_stream());
-  agrpo::launch_short_conv_ring(f, a, given(rows) ? row_end->data_ptr<int>() : nullptr, cur_stream());
+  agrpo::launch_short_conv_ring(f, a, given(rows) ? ring_rows->data_ptr<int>() : nullptr,
+                                given(rows) ? (int)ring_rows->numel() : 0, cur_stream());
 }
 
 agrpo::WindowAttnArgs attn_args(const OptTensor& q, const Tensor& k_cache, const OptTensor& rows, const OptTensor& seq_lens,
@@ -233,7 +234,7 @@ void bind_layer_ops(pybind11::module_& m) {
   namespace py = pybind11;
   using NoGil = py::call_guard<py::gil_scoped_release>;
   m.def("embed_dyt", &embed_dyt, NoGil());
-  m.def("short_conv", &short_conv, py::arg("u"), py::arg("w"), py::arg("ring"), py::arg("rows"), py::arg("row_end"), py::arg("seq_lens"),
+  m.def("short_conv", &short_conv, py::arg("u"), py::arg("w"), py::arg("ring"), py::arg("rows"), py::arg("ring_rows"), py::arg("seq_lens"),
         py::arg("block_tables"), py::arg("q_out"), py::arg("k_cache"), py::arg("status"), NoGil());
   m.def("window_attn", &window_attn, py::arg("q"), py::arg("k_cache"), py::arg("rows"), py::arg("seq_lens"), py::arg("block_tables"),
         py::arg("bias"), py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("out"), py::arg("status"), NoGil());

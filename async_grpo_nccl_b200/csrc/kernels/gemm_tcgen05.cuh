@@ -360,6 +360,15 @@ struct GatherJob {
   }
 };
 
+// Optional hook epi.tile_begin(row, col0, M, N): called for every tile before the wait for its accumulator, so that an
+// epilogue can start reading what it will need (a residual row) while the main loop still runs.
+template <class Epi>
+__device__ __forceinline__ auto epi_tile_begin(Epi& e, int row, int col0, int M, int N, int) -> decltype(e.tile_begin(row, col0, M, N)) {
+  e.tile_begin(row, col0, M, N);
+}
+template <class Epi>
+__device__ __forceinline__ void epi_tile_begin(Epi&, int, int, int, int, long) {}
+
 // Work-item order.
 //  group_n == 1: bands of 16 row-tiles, column-tile fastest across a band, so that the CTAs running at
 //                the same time share A and B tiles through L2.
@@ -560,6 +569,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       for (int t = 0; t < count; ++t, ++local) {
         const int buf = local & 1;
         const uint32_t acc_phase = (local >> 1) & 1;
+        epi_tile_begin(epi, row, (tn0 + t) * BN, p.M, p.N, 0);
         if (!mbar_wait(&tfull_bar[buf], acc_phase)) {
           report_status(p.status, kStatusWaitTmemFullTimeout);
           ok = false;

@@ -44,16 +44,51 @@ __global__ void embed_dyt_kernel(const int* __restrict__ ids, const T* __restric
 }
 
 // ------------------------------------------------------------------------------------------------
-// Short convolution. Thread = 8 channels of one token row.
+// Short convolution. Thread = 8 channels of kConvRows consecutive token rows. Inside a segment the rows it needs are loaded
+// up front and stay in registers; a tile at a segment's start, or with rows of several segments, goes row by row and takes
+// older values from the ring.
+constexpr int kConvRows = 8;
+
 template <typename T>
-__global__ void short_conv_kernel(ShortConvArgs p) {
-  pdl_wait();
-  pdl_launch();
-  const int C = p.q_cols + p.k_cols;
-  const int t = blockIdx.y;
-  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
-  if (c >= C) return;
-  const RowMap map{reinterpret_cast<const int4*>(p.rows), p.seq_lens};
+struct ConvVec;
+template <>
+struct ConvVec<bf16> {
+  uint4 v;
+  __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ float get(int i) const {
+    const uint32_t w = i < 2 ? v.x : (i < 4 ? v.y : (i < 6 ? v.z : v.w));
+    return __uint_as_float((i & 1) ? (w & 0xffff0000u) : (w << 16));
+  }
+};
+template <>
+struct ConvVec<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) {
+    a = *reinterpret_cast<const float4*>(p);
+    b = *reinterpret_cast<const float4*>(p + 4);
+  }
+  __device__ __forceinline__ float get(int i) const {
+    return i == 0 ? a.x : i == 1 ? a.y : i == 2 ? a.z : i == 3 ? a.w : i == 4 ? b.x : i == 5 ? b.y : i == 6 ? b.z : b.w;
+  }
+};
+
+template <typename T>
+__device__ __forceinline__ void conv_store(const ShortConvArgs& p, int t, const int4& r, int c, const float (&acc)[8]) {
+  if (c < p.q_cols) {
+    st8(reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_cols + c, acc);
+    return;
+  }
+  const int blk = p.block_tables[(size_t)r.x * p.max_blocks + r.y / p.block_size];
+  if (blk < 0 || blk >= p.num_cache_blocks) {
+    report_status(p.status, kStatusBadIndex);
+    return;
+  }
+  const int kc = c - p.q_cols, g = kc / p.D, d = kc % p.D, G = p.k_cols / p.D;
+  st8(reinterpret_cast<T*>(p.k_cache) + (((size_t)blk * G + g) * p.block_size + r.y % p.block_size) * p.D + d, acc);
+}
+
+template <typename T>
+__device__ __forceinline__ void conv_row(const ShortConvArgs& p, const RowMap& map, int t, int c, int C) {
   const int4 r = map.get(t);
   if (r.y < 0) return;
   const T* u = reinterpret_cast<const T*>(p.u);
@@ -73,29 +108,67 @@ __global__ void short_conv_kernel(ShortConvArgs p) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i] = fmaf(ldf(w + i * p.taps + tap), v[i], acc[i]);
   }
-  if (c < p.q_cols) {
-    st8(reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_cols + c, acc);
-    return;
-  }
-  const int blk = p.block_tables[(size_t)r.x * p.max_blocks + r.y / p.block_size];
-  if (blk < 0 || blk >= p.num_cache_blocks) {
-    report_status(p.status, kStatusBadIndex);
-    return;
-  }
-  const int kc = c - p.q_cols, g = kc / p.D, d = kc % p.D, G = p.k_cols / p.D;
-  st8(reinterpret_cast<T*>(p.k_cache) + (((size_t)blk * G + g) * p.block_size + r.y % p.block_size) * p.D + d, acc);
+  conv_store<T>(p, t, r, c, acc);
 }
 
-template <typename T>
-__global__ void short_conv_ring_kernel(ShortConvArgs p, const int* __restrict__ row_end) {
+// TAPS = 0: any number of taps, row by row
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) short_conv_kernel(ShortConvArgs p) {
   pdl_wait();
   pdl_launch();
   const int C = p.q_cols + p.k_cols;
-  const int t = blockIdx.y;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+  if (c >= C) return;
+  const RowMap map{reinterpret_cast<const int4*>(p.rows), p.seq_lens};
+  const int t0 = blockIdx.x * kConvRows;
+  const int n = p.T - t0 < kConvRows ? p.T - t0 : kConvRows;
+  if constexpr (TAPS > 0) {
+    if (p.rows != nullptr && n == kConvRows) {
+      const int4 first = map.get(t0), last = map.get(t0 + kConvRows - 1);
+      if (first.z == last.z && t0 - (TAPS - 1) >= first.z) {
+        const T* u = reinterpret_cast<const T*>(p.u) + c;
+        ConvVec<T> v[kConvRows + TAPS - 1];
+#pragma unroll
+        for (int i = 0; i < kConvRows + TAPS - 1; ++i) v[i].load(u + (size_t)(t0 - (TAPS - 1) + i) * p.ldu);
+        float w[8 * TAPS];
+        const T* wp = reinterpret_cast<const T*>(p.w) + (size_t)c * TAPS;
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) {
+          float x[8];
+          ld8(wp + i * 8, x);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) w[i * 8 + k] = x[k];
+        }
+#pragma unroll
+        for (int r = 0; r < kConvRows; ++r) {
+          float acc[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            acc[i] = 0.f;
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k) acc[i] = fmaf(w[i * TAPS + k], v[r + k].get(i), acc[i]);
+          }
+          conv_store<T>(p, t0 + r, make_int4(first.x, first.y + r, first.z, 0), c, acc);
+        }
+        return;
+      }
+    }
+  }
+  for (int r = 0; r < n; ++r) conv_row<T>(p, map, t0 + r, c, C);
+}
+
+// ring_rows: the rows whose values later steps need (the last ring_len of each segment); decode: every row
+template <typename T>
+__global__ void short_conv_ring_kernel(ShortConvArgs p, const int* __restrict__ ring_rows) {
+  pdl_wait();
+  pdl_launch();
+  const int C = p.q_cols + p.k_cols;
+  const int t = ring_rows != nullptr ? ring_rows[blockIdx.x] : blockIdx.x;
+  if (t < 0 || t >= p.T) return;
   const RowMap map{reinterpret_cast<const int4*>(p.rows), p.seq_lens};
   const int4 r = map.get(t);
-  if (r.y < 0 || (row_end != nullptr && row_end[t] - t >= p.ring_len)) return;
-  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (r.y < 0) return;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
   if (c >= C) return;
   float v[8];
   ld8(reinterpret_cast<const T*>(p.u) + (size_t)t * p.ldu + c, v);
@@ -425,18 +498,28 @@ void launch_embed_dyt(bool fp32, const int* ids, const void* table, float scale,
   }
 }
 
+namespace {
+template <typename T>
+void short_conv_t(const ShortConvArgs& a, cudaStream_t s) {
+  const dim3 grid((a.T + kConvRows - 1) / kConvRows, ((a.q_cols + a.k_cols) / 8 + 127) / 128), block(128);
+  auto kernel = a.taps == 1 ? short_conv_kernel<T, 1> : a.taps == 2 ? short_conv_kernel<T, 2> : a.taps == 3 ? short_conv_kernel<T, 3>
+                : a.taps == 4 ? short_conv_kernel<T, 4> : short_conv_kernel<T, 0>;
+  launch_kernel(kernel, grid, block, 0, s, "short_conv", a);
+}
+}  // namespace
+
 void launch_short_conv(bool fp32, const ShortConvArgs& a, cudaStream_t s) {
   if (a.T == 0) return;
-  const dim3 grid(((a.q_cols + a.k_cols) / 8 + 127) / 128, a.T), block(128);
-  if (fp32) launch_kernel(short_conv_kernel<float>, grid, block, 0, s, "short_conv", a);
-  else launch_kernel(short_conv_kernel<bf16>, grid, block, 0, s, "short_conv", a);
+  if (fp32) short_conv_t<float>(a, s);
+  else short_conv_t<bf16>(a, s);
 }
 
-void launch_short_conv_ring(bool fp32, const ShortConvArgs& a, const int* row_end, cudaStream_t s) {
-  if (a.T == 0 || a.taps <= 1) return;
-  const dim3 grid(((a.q_cols + a.k_cols) / 8 + 127) / 128, a.T), block(128);
-  if (fp32) launch_kernel(short_conv_ring_kernel<float>, grid, block, 0, s, "short_conv_ring", a, row_end);
-  else launch_kernel(short_conv_ring_kernel<bf16>, grid, block, 0, s, "short_conv_ring", a, row_end);
+void launch_short_conv_ring(bool fp32, const ShortConvArgs& a, const int* ring_rows, int n_ring_rows, cudaStream_t s) {
+  const int n = ring_rows != nullptr ? n_ring_rows : a.T;
+  if (n == 0 || a.taps <= 1) return;
+  const dim3 grid(n, ((a.q_cols + a.k_cols) / 8 + 127) / 128), block(128);
+  if (fp32) launch_kernel(short_conv_ring_kernel<float>, grid, block, 0, s, "short_conv_ring", a, ring_rows);
+  else launch_kernel(short_conv_ring_kernel<bf16>, grid, block, 0, s, "short_conv_ring", a, ring_rows);
 }
 
 void launch_window_attn(bool fp32, const WindowAttnArgs& a, cudaStream_t s) {

@@ -22,6 +22,10 @@ __device__ __forceinline__ float tanh_f32(float z) {
   return copysignf(__fdividef(1.f - e, 1.f + e), z);
 }
 
+// The same function for the bf16 epilogues: absolute error about 1e-7 everywhere (the difference cancels near zero), a third of
+// the instructions.
+__device__ __forceinline__ float tanh_abs_f32(float z) { return fmaf(-2.f, __fdividef(1.f, 1.f + __expf(2.f * z)), 1.f); }
+
 __device__ __forceinline__ float sigmoid_f32(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 
 // Dynamic Tanh norm: y = tanh(alpha * x) * w + b, elementwise.
@@ -78,8 +82,8 @@ __device__ __forceinline__ void dyt_residual8(const float (&acc)[8], float* x, T
   ld8(n2.b + col, b2);
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
-    xv[i] += fmaf(tanh_f32(a1 * acc[i]), w1[i], b1[i]);
-    hv[i] = fmaf(tanh_f32(a2 * xv[i]), w2[i], b2[i]);
+    xv[i] += fmaf(tanh_abs_f32(a1 * acc[i]), w1[i], b1[i]);
+    hv[i] = fmaf(tanh_abs_f32(a2 * xv[i]), w2[i], b2[i]);
   }
   st8(x, xv);
   st8(h, hv);

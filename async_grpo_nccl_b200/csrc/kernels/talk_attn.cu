@@ -487,24 +487,39 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
   const int* table = p.block_tables + (size_t)b * p.max_blocks;
   const bf16* cache = reinterpret_cast<const bf16*>(p.k_cache);
 
+  // Pages of the next tile to load, one per lane (a tile of 64 keys touches at most five): looked up one tile ahead, so that
+  // no copy waits for its table entry.
+  int page = 0;
+  auto fetch_pages = [&](int t) {
+    const int bi = (lo + t * kDT) / 16 + lane;
+    if (t < t_end && lane < 5 && bi <= pos / 16) {
+      page = table[bi];
+      if (page < 0 || page >= p.num_cache_blocks) {
+        report_status(p.status, kStatusBadIndex);
+        page = 0;
+      }
+    }
+  };
   auto load_tile = [&](int t, int stage) {
     constexpr int kRowChunks = D / 8;
     uint8_t* dst = sKV + stage * stage_bytes;
-    for (int i = tid; i < kDT * G * kRowChunks; i += kDThreads) {
+    const int jt = lo + t * kDT, b0 = jt / 16;
+    const int n = kDT * G * kRowChunks;                      // a multiple of the CTA's threads: warps stay whole
+#pragma unroll 4
+    for (int i = tid; i < n; i += kDThreads) {
       const int ch = i % kRowChunks, row = i / kRowChunks;   // row = m * 64 + key
-      const int m = row / kDT, key = row % kDT;
-      int j = lo + t * kDT + key;
-      if (j == pos) continue;                                // comes from sKnew
-      if (j > pos) j = pos > 0 ? pos - 1 : 0;                // masked; any key that exists
-      int blk = table[j / 16];
-      if (blk < 0 || blk >= p.num_cache_blocks) {
-        report_status(p.status, kStatusBadIndex);
-        blk = 0;
-      }
-      cp_async16(sw_chunk<D>(dst, row, ch), cache + (((size_t)blk * G + m) * 16 + j % 16) * D + ch * 8);
+      const int m = row / kDT;
+      int j = jt + row % kDT;
+      const bool on = j < pos;                               // the newest key comes from sKnew, later ones are masked
+      const int blk = __shfl_sync(0xffffffffu, page, on ? j / 16 - b0 : 0);
+      j = on ? j : 0;
+      if (on) cp_async16(sw_chunk<D>(dst, row, ch), cache + (((size_t)blk * G + m) * 16 + j % 16) * D + ch * 8);
+      else if (row % kDT != pos - jt) *reinterpret_cast<uint4*>(sw_chunk<D>(dst, row, ch)) = make_uint4(0u, 0u, 0u, 0u);
     }
+    fetch_pages(t + 1);
   };
   // loads first: they do not depend on the new token
+  fetch_pages(t_begin);
   for (int i = 0; i < n_stages - 1; ++i) {
     if (t_begin + i < t_end) load_tile(t_begin + i, i);
     cp_async_commit();
@@ -581,7 +596,16 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
       cp_async_commit();
     }
     // ---- scores of keys [8 warp, 8 warp + 8) for all heads ----
-    float s[MT][4];
+    float s[MT][4], bv[MT][4];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {  // distance biases, on their way while the MMAs run
+        const int h = mt * 16 + r0 + (e >> 1) * 8;
+        const int d = pos - (j0 + warp * 8 + cq + (e & 1));
+        const bool on = h < H && d >= 0 && d < p.window && d < p.bias_len;
+        bv[mt][e] = on ? __ldg(p.bias + (size_t)h * p.bias_len + d) : INFINITY;
+      }
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       s[mt][0] = s[mt][1] = s[mt][2] = s[mt][3] = 0.f;
@@ -603,13 +627,7 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
       }
       // scale, distance bias, mask; row maxima over this warp's keys
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int h = h_lo + r0 + (e >> 1) * 8;
-        const int d = pos - (j0 + warp * 8 + cq + (e & 1));
-        const bool on = h < H && d >= 0 && d < p.window && d < p.bias_len;
-        const float bv = __ldg(p.bias + (on ? (size_t)h * p.bias_len + d : 0));
-        s[mt][e] = on ? fmaf(s[mt][e], qs, -bv) : -INFINITY;
-      }
+      for (int e = 0; e < 4; ++e) s[mt][e] = fmaf(s[mt][e], qs, -bv[mt][e]);  // masked: minus infinity
 #pragma unroll
       for (int q = 0; q < 2; ++q) {
         float mx = fmaxf(s[mt][2 * q], s[mt][2 * q + 1]);

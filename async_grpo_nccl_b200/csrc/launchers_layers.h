@@ -46,8 +46,9 @@ struct ShortConvArgs {
   int* status;
 };
 void launch_short_conv(bool fp32, const ShortConvArgs& a, cudaStream_t s);
-// Writes the values that later steps need (the last ring_len of each segment) into the ring; row_end[t] = last row of t's segment.
-void launch_short_conv_ring(bool fp32, const ShortConvArgs& a, const int* row_end, cudaStream_t s);
+// Writes the values that later steps need into the ring: ring_rows lists the last ring_len rows of each segment
+// (nullptr: decode rows, every row). A launch of its own: the convolution of a segment's first rows reads the ring.
+void launch_short_conv_ring(bool fp32, const ShortConvArgs& a, const int* ring_rows, int n_ring_rows, cudaStream_t s);
 
 // Sliding-window attention over the paged keys (which are also the values), softmax weights mixed across heads by
 // talk [H, H], output multiplied by sigmoid(gate). Any head size that is a multiple of 8.

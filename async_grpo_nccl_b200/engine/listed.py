@@ -104,10 +104,11 @@ class ListedEngine(RolloutEngine):
     def _forward(self, segments: Sequence[Tuple[int, int, np.ndarray]]) -> torch.Tensor:
         """One step over segments (slot, tokens already cached, new tokens): keys and rings are updated, the final normed
         hidden states of all rows come back."""
-        flat, T, n_tiles = host_batch(segments)
+        flat, where = host_batch(segments, [l.mixer.conv for l in self.cfg.layers])
         dev_flat = torch.from_numpy(flat).pin_memory().to(self.dev, non_blocking=True)
         self.h2d_bytes += flat.nbytes
-        ids, sb = split_batch(dev_flat, T, n_tiles, self.block_tables)
+        ids, sb = split_batch(dev_flat, where, self.block_tables)
+        T = sb.T
         x = torch.empty(T, self.cfg.hidden_size, dtype=torch.float32, device=self.dev)
         h = torch.empty(T, self.cfg.hidden_size, dtype=self.dtype, device=self.dev)
         self._layers(ids, x, h, sb, self.dec.buffers(T))

@@ -30,37 +30,44 @@ class StepBatch:
     T: int
     block_tables: torch.Tensor
     rows: Optional[torch.Tensor] = None      # [T, 4] int32: slot, position, first row of the segment, 0
-    row_end: Optional[torch.Tensor] = None   # [T] last row of the segment
+    ring_rows: Optional[Dict[int, torch.Tensor]] = None  # taps -> the last `taps` rows of each segment
     tiles: Optional[torch.Tensor] = None     # [n, 4]: first row, rows, position of the first row, slot
     seq_lens: Optional[torch.Tensor] = None
     splits: int = 1
     scratch: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None  # decode: partial products, (max, sum), tickets
 
 
-def host_batch(segments: Sequence[Tuple[int, int, np.ndarray]]) -> Tuple[np.ndarray, int, int]:
-    """(slot, tokens already there, new tokens) per segment -> one int32 array [ids | row_end | rows | tiles], T, n_tiles."""
-    ids, ends, rows, tiles = [], [], [], []
+def host_batch(segments: Sequence[Tuple[int, int, np.ndarray]], taps: Sequence[int]) -> Tuple[np.ndarray, Dict[str, Tuple[int, int]]]:
+    """(slot, tokens already there, new tokens) per segment -> one int32 array with the step's tables and where each of them
+    is in it: token ids, rows, attention tiles and, for every length in ``taps``, the rows that the convolution rings keep."""
+    ids, rows, tiles = [], [], []
+    keep: Dict[int, List[np.ndarray]] = {k: [] for k in sorted(set(taps))}
     t0 = 0
     for slot, past, toks in segments:
         n = len(toks)
         ids.append(np.asarray(toks, dtype=np.int32))
-        ends.append(np.full(n, t0 + n - 1, np.int32))
         r = np.zeros((n, 4), np.int32)
         r[:, 0], r[:, 1], r[:, 2] = slot, past + np.arange(n), t0
         rows.append(r)
         tiles += [(t0 + a, min(TILE, n - a), past + a, slot) for a in range(0, n, TILE)]
+        for k, v in keep.items():
+            v.append(np.arange(t0 + max(0, n - k), t0 + n, dtype=np.int32))
         t0 += n
     tiles.sort(key=lambda t: -t[2])
-    tl = np.asarray(tiles, np.int32)
-    pad = (-2 * t0) % 4  # keeps the row table 16-byte aligned
-    flat = np.concatenate(ids + ends + [np.zeros(pad, np.int32)] + [r.ravel() for r in rows] + [tl.ravel()])
-    return flat, t0, len(tiles)
+    parts = {"rows": np.concatenate(rows).ravel(), "tiles": np.asarray(tiles, np.int32).ravel(), "ids": np.concatenate(ids),
+             **{f"ring{k}": np.concatenate(v) for k, v in keep.items()}}   # the two tables of int4 come first: 16-byte aligned
+    where, o = {}, 0
+    for k, v in parts.items():
+        where[k] = (o, len(v))
+        o += len(v)
+    return np.concatenate(list(parts.values())), where
 
 
-def split_batch(flat: torch.Tensor, T: int, n_tiles: int, block_tables: torch.Tensor) -> Tuple[torch.Tensor, StepBatch]:
-    o = 2 * T + (-2 * T) % 4
-    return flat[:T], StepBatch(T, block_tables, rows=flat[o:o + 4 * T].view(T, 4), row_end=flat[T:2 * T],
-                               tiles=flat[o + 4 * T:o + 4 * T + 4 * n_tiles].view(n_tiles, 4))
+def split_batch(flat: torch.Tensor, where: Dict[str, Tuple[int, int]], block_tables: torch.Tensor) -> Tuple[torch.Tensor, StepBatch]:
+    part = {k: flat[o:o + n] for k, (o, n) in where.items()}
+    T = where["ids"][1]
+    return part["ids"], StepBatch(T, block_tables, rows=part["rows"].view(T, 4), tiles=part["tiles"].view(-1, 4),
+                                  ring_rows={int(k[4:]): v for k, v in part.items() if k.startswith("ring")})
 
 
 class ListedDecoder:
@@ -155,7 +162,7 @@ class ListedDecoder:
                                self.w(p + "talk"), gate, m.window, out, sb.splits, *sb.scratch, self.status)
             self.launches += 1
             return
-        C.short_conv(u, self.w(p + "conv"), ring, sb.rows, sb.row_end, sb.seq_lens, sb.block_tables, q, k_cache, self.status)
+        C.short_conv(u, self.w(p + "conv"), ring, sb.rows, sb.ring_rows[m.conv] if sb.rows is not None else None, sb.seq_lens, sb.block_tables, q, k_cache, self.status)
         if sb.rows is not None and not self.fp32:
             acc = torch.empty(sb.T * m.heads * m.k_dim, dtype=self.dtype, device=self.dev)
             if C.talk_attn_prefill(q, k_cache, sb.tiles, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate, m.window,

@@ -142,8 +142,8 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
     cache = R(n_seq * nb, G, 16, D)
     tables = torch.randperm(n_seq * nb, device=dev).int().view(n_seq, nb).contiguous()
     ring = torch.zeros(max(n_seq, B), m.conv, m.qk_dim, device=dev, dtype=bf)
-    flat, T2, nt = host_batch([(i, 0, np.zeros(prompt, np.int32)) for i in range(n_seq)])
-    _, sb = split_batch(torch.from_numpy(flat).to(dev), T2, nt, tables)
+    flat, where = host_batch([(i, 0, np.zeros(prompt, np.int32)) for i in range(n_seq)], [m.conv])
+    _, sb = split_batch(torch.from_numpy(flat).to(dev), where, tables)
     acc = torch.empty(T * H * G * D, device=dev, dtype=bf)
     lse = torch.empty(H, T, device=dev)
     tiles = _tiles([prompt] * n_seq)
@@ -152,7 +152,7 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
     gm = lambda M, N, K: (2.0 * M * N * K, 2.0 * (M * K + N * K + M * N))
     add("prompt projection", "new", lambda: C.gemm_bf16(h, wqkg, u, False, False, None, 1.0, False, st, None), *gm(T, m.u_dim, W))
     add("prompt projection", "old", lambda: C.gemm_bf16(h, wqkv, qkv, False, False, None, 1.0, False, st, None), *gm(T, old.qkv_dim, W))
-    add("prompt position op", "new", lambda: C.short_conv(u, conv, ring, sb.rows, sb.row_end, None, tables, q, cache, st), 0.0, 4.0 * T * m.qk_dim)
+    add("prompt position op", "new", lambda: C.short_conv(u, conv, ring, sb.rows, sb.ring_rows[m.conv], None, tables, q, cache, st), 0.0, 4.0 * T * m.qk_dim)
     pos = torch.arange(T, device=dev, dtype=torch.int32) % prompt
     cos = torch.rand(maxlen, D // 2, device=dev)
     slots = torch.arange(T, device=dev, dtype=torch.int32)
