@@ -58,8 +58,8 @@ agrpo::ShortConvArgs conv_args(const Tensor& u, const Tensor& w, Tensor& ring, c
   a.k_cols = (int)(k_cache.size(1) * k_cache.size(3));
   a.q_cols = (int)q_out.size(1);
   const int64_t C = a.q_cols + a.k_cols, T = u.size(0);
-  TORCH_CHECK(w.dim() == 2 && w.size(0) == C && w.is_contiguous(), "short_conv: w [q + k channels, taps]");
-  TORCH_CHECK(ring.dim() == 3 && ring.size(2) == C && ring.size(1) >= w.size(1) && ring.stride(2) == 1 &&
+  TORCH_CHECK(w.dim() == 2 && w.size(1) == C && w.is_contiguous() && aligned16(w), "short_conv: w [taps, q + k channels]");
+  TORCH_CHECK(ring.dim() == 3 && ring.size(2) == C && ring.size(1) >= w.size(0) && ring.stride(2) == 1 &&
               ring.stride(1) == C && ring.stride(0) % 8 == 0 && aligned16(ring),
               "short_conv: ring [slots, >= taps, channels]");
   TORCH_CHECK(u.size(1) >= C && u.stride(0) % 8 == 0 && aligned16(u) && q_out.is_contiguous() && q_out.size(0) >= T && aligned16(q_out), "short_conv: u / q_out");
@@ -68,7 +68,7 @@ agrpo::ShortConvArgs conv_args(const Tensor& u, const Tensor& w, Tensor& ring, c
   else { TORCH_CHECK(given(seq_lens), "short_conv: rows or seq_lens"); check_i32(*seq_lens, "seq_lens");
          TORCH_CHECK(seq_lens->numel() >= T && block_tables.size(0) >= T && ring.size(0) >= T, "short_conv: decode rows"); }
   a.u = u.data_ptr(); a.ldu = u.stride(0);
-  a.w = w.data_ptr(); a.taps = (int)w.size(1);
+  a.w = w.data_ptr(); a.taps = (int)w.size(0);
   a.ring = ring.data_ptr(); a.ring_len = (int)ring.size(1); a.ring_pitch = ring.stride(0);
   a.rows = iptr(rows); a.seq_lens = iptr(seq_lens);
   a.block_tables = block_tables.data_ptr<int>(); a.max_blocks = (int)block_tables.size(1);
@@ -163,14 +163,14 @@ void talk_attn_decode(const Tensor& u, const Tensor& conv_w, Tensor& ring, Tenso
   same_type(u, false, "u"); same_type(conv_w, false, "conv_w"); same_type(ring, false, "ring"); rows2d(u, "u");
   check_f32(part_o, "part_o"); check_f32(part_ml, "part_ml"); check_i32(tickets, "tickets");
   TORCH_CHECK(u.size(0) >= B && u.size(1) >= C && u.stride(0) % 8 == 0 && aligned16(u), "talk_attn_decode: u");
-  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == C && conv_w.is_contiguous(), "talk_attn_decode: conv_w [q + k channels, taps]");
-  TORCH_CHECK(ring.dim() == 3 && ring.size(0) >= B && ring.size(1) == conv_w.size(1) && ring.size(2) == C && ring.stride(2) == 1 &&
+  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(1) == C && conv_w.is_contiguous() && aligned16(conv_w), "talk_attn_decode: conv_w [taps, q + k channels]");
+  TORCH_CHECK(ring.dim() == 3 && ring.size(0) >= B && ring.size(1) == conv_w.size(0) && ring.size(2) == C && ring.stride(2) == 1 &&
               ring.stride(1) == C && ring.stride(0) % 8 == 0 && aligned16(ring), "talk_attn_decode: ring [slots, taps, channels]");
   TORCH_CHECK(splits >= 1 && splits <= 8, "talk_attn_decode: 1 to 8 splits");
   TORCH_CHECK(splits == 1 || (part_o.numel() >= B * splits * d.at.H * d.at.G * d.at.D && part_ml.numel() >= B * splits * d.at.H * 2 &&
               tickets.numel() >= B), "talk_attn_decode: scratch");
   d.u = u.data_ptr(); d.ldu = u.stride(0);
-  d.conv_w = conv_w.data_ptr(); d.taps = (int)conv_w.size(1);
+  d.conv_w = conv_w.data_ptr(); d.taps = (int)conv_w.size(0);
   d.ring = ring.data_ptr(); d.ring_len = (int)ring.size(1); d.ring_pitch = ring.stride(0);
   d.k_cache = k_cache.data_ptr();
   d.splits = (int)splits;

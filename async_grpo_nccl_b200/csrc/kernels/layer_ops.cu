@@ -93,7 +93,7 @@ __device__ __forceinline__ void conv_row(const ShortConvArgs& p, const RowMap& m
   if (r.y < 0) return;
   const T* u = reinterpret_cast<const T*>(p.u);
   const T* ring = reinterpret_cast<const T*>(p.ring);
-  const T* w = reinterpret_cast<const T*>(p.w) + (size_t)c * p.taps;
+  const T* w = reinterpret_cast<const T*>(p.w) + c;
   float acc[8];
 #pragma unroll
   for (int i = 0; i < 8; ++i) acc[i] = 0.f;
@@ -102,11 +102,11 @@ __device__ __forceinline__ void conv_row(const ShortConvArgs& p, const RowMap& m
     const int row = t - back;
     const T* src = row >= r.z ? u + (size_t)row * p.ldu + c
                               : ring + (size_t)r.x * p.ring_pitch + (size_t)((r.y - back) % p.ring_len) * C + c;
-    float v[8];
+    float v[8], x[8];
     ld8(src, v);
-    const int tap = p.taps - 1 - back;
+    ld8(w + (size_t)(p.taps - 1 - back) * C, x);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i] = fmaf(ldf(w + i * p.taps + tap), v[i], acc[i]);
+    for (int i = 0; i < 8; ++i) acc[i] = fmaf(x[i], v[i], acc[i]);
   }
   conv_store<T>(p, t, r, c, acc);
 }
@@ -130,15 +130,9 @@ __global__ void __launch_bounds__(128) short_conv_kernel(ShortConvArgs p) {
         ConvVec<T> v[kConvRows + TAPS - 1];
 #pragma unroll
         for (int i = 0; i < kConvRows + TAPS - 1; ++i) v[i].load(u + (size_t)(t0 - (TAPS - 1) + i) * p.ldu);
-        float w[8 * TAPS];
-        const T* wp = reinterpret_cast<const T*>(p.w) + (size_t)c * TAPS;
+        float w[TAPS][8];
 #pragma unroll
-        for (int i = 0; i < TAPS; ++i) {
-          float x[8];
-          ld8(wp + i * 8, x);
-#pragma unroll
-          for (int k = 0; k < 8; ++k) w[i * 8 + k] = x[k];
-        }
+        for (int k = 0; k < TAPS; ++k) ld8(reinterpret_cast<const T*>(p.w) + (size_t)k * C + c, w[k]);
 #pragma unroll
         for (int r = 0; r < kConvRows; ++r) {
           float acc[8];
@@ -146,7 +140,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(ShortConvArgs p) {
           for (int i = 0; i < 8; ++i) {
             acc[i] = 0.f;
 #pragma unroll
-            for (int k = 0; k < TAPS; ++k) acc[i] = fmaf(w[i * TAPS + k], v[r + k].get(i), acc[i]);
+            for (int k = 0; k < TAPS; ++k) acc[i] = fmaf(w[k][i], v[r + k].get(i), acc[i]);
           }
           conv_store<T>(p, t0 + r, make_int4(first.x, first.y + r, first.z, 0), c, acc);
         }

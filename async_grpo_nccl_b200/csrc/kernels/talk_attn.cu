@@ -27,12 +27,15 @@ typedef __nv_bfloat16 bf16;
 // ================================================================================================
 // Prompts: one CTA = 128 query rows of one head g, value heads [m0, m0 + mc). S (two buffers, so that the scores of tile
 // j + 1 are computed while the softmax of tile j runs) and the mc accumulators fill tensor memory. Warp 0 loads key tiles
-// page by page, warp 1 issues MMAs, warps 2-9 run the softmax: two threads per query row, 64 keys each. The key tile of
-// a head serves as K-major operand of Q K^T and as MN-major operand of P V.
+// page by page, warp 1 issues MMAs, warps 2-17 run the softmax: four threads per query row, 32 keys each (with fewer warps
+// the softmax is bound by latency and the tensor cores wait for it). The key tile of a head serves as K-major operand of
+// Q K^T and as MN-major operand of P V.
 // ================================================================================================
 constexpr int kPM = 128;
 constexpr int kPN = 128;
-constexpr int kPThreads = 320;
+constexpr int kPParts = 4;                            // threads per query row
+constexpr int kPKeys = kPN / kPParts;                // keys per thread and tile
+constexpr int kPThreads = 64 + kPParts * kPM;
 constexpr int kRingBytes = 192 * 1024;
 
 struct TalkPrefillParams {
@@ -50,7 +53,7 @@ struct TalkPrefillParams {
   int* status;
 };
 
-__device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+__device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 512;" ::: "memory"); }
 
 template <int D>
 __global__ void __launch_bounds__(kPThreads, 1)
@@ -62,7 +65,8 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   extern __shared__ __align__(1024) uint8_t tp_smem[];
   uint8_t* sQ = tp_smem;
   uint8_t* sK = tp_smem + kTile;
-  float* smax = reinterpret_cast<float*>(sK + kRingBytes);   // [2 parities][2 halves][128]
+  float* smax = reinterpret_cast<float*>(sK + kRingBytes);   // 2 KB: row maxima [2 parities][4 parts][128] as bf16, at the end sums
+  bf16* smax16 = reinterpret_cast<bf16*>(smax);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smax + 512);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;      // [3]
@@ -96,7 +100,7 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
     mbar_init(&s_full[0], 1);
     mbar_init(&s_full[1], 1);
-    mbar_init(p_ready, 8);
+    mbar_init(p_ready, 4 * kPParts);
     mbar_init(o_done, 1);
     fence_mbar_init();
   }
@@ -216,53 +220,54 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
     }
   } else {
-    // ---------------- softmax: thread = (query row, half of the tile's keys) ----------------
-    const int quarter = warp & 3, half = (warp - 2) >> 2;
+    // ---------------- softmax: thread = (query row, quarter of the tile's keys) ----------------
+    const int quarter = warp & 3, part = (warp - 2) >> 2;
     const int r = quarter * 32 + lane;
     const int qi = pos0 + r;
     const uint32_t lane_off = static_cast<uint32_t>(quarter * 32) << 16;
     const float qs = p.qscale[qi < p.qscale_len ? qi : p.qscale_len - 1];
     const float* bias = p.bias + (size_t)head * p.bias_len;
-    const int o_cols = mc * D / 2;            // accumulator columns that this half rescales and stores
+    const int o_cols = mc * D / kPParts;      // accumulator columns that this thread rescales and stores
+    const uint32_t tO = tmem_O + lane_off + part * o_cols;
     float m = -INFINITY, l = 0.f;
     bool ok = true;                           // after a failure the barriers are still met, nothing else is waited for
     for (int j = 0; j < n_kv; ++j) {
+      const int tk = j0 + j * kPN;            // first key of the tile
+      const int d0 = qi - (tk + part * kPKeys);  // distance of this thread's first key
+      const bool inside = tk + kPN - 1 <= pos0 && pos0 + kPM - 1 - tk < p.window && pos0 + kPM - 1 - tk < p.bias_len;
+      float v[kPKeys];                        // distance biases, on their way while the scores are computed
+      if (inside) {
+#pragma unroll
+        for (int i = 0; i < kPKeys; ++i) v[i] = __ldg(bias + d0 - i);
+      } else {
+#pragma unroll
+        for (int i = 0; i < kPKeys; ++i) {
+          const int d = d0 - i;
+          v[i] = d >= 0 && d < p.window && d < p.bias_len ? __ldg(bias + d) : INFINITY;
+        }
+      }
       if (ok && !mbar_wait(&s_full[j & 1], (j >> 1) & 1)) {
         report_status(p.status, kStatusWaitTmemFullTimeout);
         ok = false;
       }
       tc_fence_after();
       const uint32_t tS = tmem + (j & 1) * 128 + lane_off;
-      const int tk = j0 + j * kPN;            // first key of the tile
-      const int d0 = qi - (tk + half * 64);   // distance of this thread's first key
-      uint32_t s0[32], s1[32];
-      tmem_ld_32x32(tS + half * 64, s0);
-      tmem_ld_32x32(tS + half * 64 + 32, s1);
+      uint32_t s0[32];
+      tmem_ld_32x32(tS + part * kPKeys, s0);
       tc_wait_ld();
-      float v[64];
-      float mx = -INFINITY;
-      const bool inside = tk + kPN - 1 <= pos0 && pos0 + kPM - 1 - tk < p.window && pos0 + kPM - 1 - tk < p.bias_len;
-      if (inside) {
 #pragma unroll
-        for (int i = 0; i < 64; ++i) {
-          v[i] = fmaf(__uint_as_float(i < 32 ? s0[i & 31] : s1[i & 31]), qs, -__ldg(bias + d0 - i));
-          mx = fmaxf(mx, v[i]);
-        }
-      } else {
+      for (int i = 0; i < kPKeys; ++i) v[i] = fmaf(__uint_as_float(s0[i]), qs, -v[i]);  // masked keys: minus infinity
+      float mx4[4] = {v[0], v[1], v[2], v[3]};
 #pragma unroll
-        for (int i = 0; i < 64; ++i) {
-          const int d = d0 - i;
-          const bool on = d >= 0 && d < p.window && d < p.bias_len;
-          const float b = __ldg(bias + (on ? d : 0));
-          v[i] = on ? fmaf(__uint_as_float(i < 32 ? s0[i & 31] : s1[i & 31]), qs, -b) : -INFINITY;
-          mx = fmaxf(mx, v[i]);
-        }
-      }
-      smax[((j & 1) * 2 + half) * 128 + r] = mx;
+      for (int i = 4; i < kPKeys; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], v[i]);
+      // the maximum is only a reference point: exchanged in bf16, the same rounded value for all threads of a row
+      smax16[((j & 1) * kPParts + part) * 128 + r] = __float2bfloat16(fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])));
       tc_fence_before();
-      softmax_bar();                          // both halves have read their scores: the weights may overwrite them
+      softmax_bar();                          // everybody has read the scores: the weights may overwrite them
       tc_fence_after();
-      mx = fmaxf(mx, smax[((j & 1) * 2 + (half ^ 1)) * 128 + r]);
+      float mx = -INFINITY;
+#pragma unroll
+      for (int e = 0; e < kPParts; ++e) mx = fmaxf(mx, __bfloat162float(smax16[((j & 1) * kPParts + e) * 128 + r]));
       // keep a stale maximum unless it grew by more than 2^8: the weights stay bounded and O rarely needs rescaling
       float alpha = 1.f;
       if (mx > m + 8.f || m == -INFINITY) {
@@ -277,58 +282,54 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         }
         tc_fence_after();
 #pragma unroll 1
-        for (int c = 0; c < o_cols; c += 32) {
-          const uint32_t a = tmem_O + lane_off + half * o_cols + c;
-          uint32_t o[32];
-          tmem_ld_32x32(a, o);
+        for (int c = 0; c < o_cols; c += 16) {
+          uint32_t o[16];
+          tmem_ld_32x16(tO + c, o);
           tc_wait_ld();
-          uint32_t x0[16], x1[16];
 #pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            x0[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
-            x1[i] = __float_as_uint(__uint_as_float(o[16 + i]) * alpha);
-          }
-          tmem_st_32x16(a, x0);
-          tmem_st_32x16(a + 16, x1);
+          for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+          tmem_st_32x16(tO + c, o);
         }
         l *= alpha;
       }
-      uint32_t w0[16], w1[16];
+      uint32_t w[kPKeys / 2];
+      float l0 = 0.f, l1 = 0.f;
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
+      for (int i = 0; i < kPKeys / 2; ++i) {
         const float a = exp2f(v[2 * i] - base), b = exp2f(v[2 * i + 1] - base);
-        const float c = exp2f(v[32 + 2 * i] - base), d = exp2f(v[32 + 2 * i + 1] - base);
-        l += (a + b) + (c + d);
-        w0[i] = pack_bf16x2(a, b);
-        w1[i] = pack_bf16x2(c, d);
+        l0 += a;
+        l1 += b;
+        w[i] = pack_bf16x2(a, b);
       }
-      tmem_st_32x16(tS + half * 32, w0);
-      tmem_st_32x16(tS + half * 32 + 16, w1);
+      l += l0 + l1;
+      tmem_st_32x16(tS + part * (kPKeys / 2), w);
       tc_wait_st();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(p_ready);
     }
-    // the two halves of a row add up their sums
+    // the threads of a row add up their sums
     softmax_bar();
-    smax[half * 128 + r] = l;
+    smax[part * 128 + r] = l;
     softmax_bar();
-    l += smax[(half ^ 1) * 128 + r];
+    l = 0.f;
+#pragma unroll
+    for (int e = 0; e < kPParts; ++e) l += smax[e * 128 + r];
     if (ok && !mbar_wait(o_done, (n_kv - 1) & 1)) {
       report_status(p.status, kStatusWaitTmemFullTimeout);
       ok = false;
     }
     tc_fence_after();
     const float inv = l > 0.f ? 1.f / l : 0.f;
-    bf16* dst = p.acc + (((size_t)(tile.x + r) * p.H + head) * p.G + m0) * D + half * o_cols;
+    bf16* dst = p.acc + (((size_t)(tile.x + r) * p.H + head) * p.G + m0) * D + part * o_cols;
 #pragma unroll 1
-    for (int c = 0; c < o_cols; c += 32) {
-      uint32_t o[32];
-      tmem_ld_32x32(tmem_O + lane_off + half * o_cols + c, o);
+    for (int c = 0; c < o_cols; c += 16) {
+      uint32_t o[16];
+      tmem_ld_32x16(tO + c, o);
       tc_wait_ld();
       if (ok && r < n_rows) {
 #pragma unroll
-        for (int i = 0; i < 32; i += 8) {
+        for (int i = 0; i < 16; i += 8) {
           uint4 w;
           w.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
           w.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
@@ -424,9 +425,10 @@ void launch_prefill_t(const CUtensorMap& tq, const CUtensorMap& tk, const TalkPr
 
 // ================================================================================================
 // Decode: CTA = (split, sequence), 8 warps, all heads. The prologue convolves the new token's q (every split) and k (the
-// split that owns the newest token, which also writes the key page and the ring). Per tile of 64 keys: warp w scores its 8
-// keys against all heads, the CTA agrees on the row maxima, the weights meet in shared memory, and warp w accumulates its
-// share of the G * D value columns for all heads. The last split of a sequence to finish merges, mixes, gates and stores.
+// split that owns the newest token, which also writes the key page and the ring). Key tiles of 64 tokens arrive by TMA, page
+// by page, from before the new token's projections are complete. Per tile: warp w scores its 8 keys against all heads, the
+// CTA agrees on the row maxima, the weights meet in shared memory, and warp w accumulates its share of the G * D value
+// columns for all heads. The last split of a sequence to finish merges, mixes, gates and stores.
 // ================================================================================================
 constexpr int kDT = 64;         // keys per tile
 constexpr int kDThreads = 256;
@@ -434,101 +436,117 @@ constexpr int kPPitch = kDT + 8;
 
 template <int D, int MT>
 struct DecSmem {
-  static constexpr int kRowBytes = D * 2;
-  static constexpr int kQ = MT * 16 * kRowBytes;
+  static constexpr int kQ = MT * 16 * D * 2;
   static constexpr int kP = MT * 16 * kPPitch * 2;
   static constexpr int kMax = MT * 16 * 8 * 4;
 };
 
-template <int D>
-__device__ __forceinline__ uint8_t* sw_chunk(uint8_t* base, int row, int chunk) {  // 16-byte chunks, conflict-free for ldmatrix
-  return base + row * (D * 2) + ((chunk ^ (row & 7)) << 4);
-}
+// Rows of 64 channels (128 bytes), 16-byte chunk c of row r stored at c ^ (r & 7): the layout of a TMA box with 128-byte swizzle.
+__device__ __forceinline__ uint32_t sw_off(int row, int chunk) { return row * 128 + ((chunk ^ (row & 7)) << 4); }
 
-// eight channels of the convolution of the token at `pos` (its own value in u, older ones in the ring)
+// eight channels of the convolution of the token at `pos` (its own value in u, older ones in the ring); weights [taps, C]
 __device__ __forceinline__ void conv8(const TalkDecodeArgs& a, int b, int pos, int C, int c, float (&acc)[8]) {
-  const bf16* w = reinterpret_cast<const bf16*>(a.conv_w) + (size_t)c * a.taps;
-  const bf16* ring = reinterpret_cast<const bf16*>(a.ring) + (size_t)b * a.ring_pitch;
+  const bf16* w = reinterpret_cast<const bf16*>(a.conv_w) + c;
+  const bf16* ring = reinterpret_cast<const bf16*>(a.ring) + (size_t)b * a.ring_pitch + c;
+  const bf16* u = reinterpret_cast<const bf16*>(a.u) + (size_t)b * a.ldu + c;
 #pragma unroll
   for (int i = 0; i < 8; ++i) acc[i] = 0.f;
-  for (int back = a.taps - 1; back >= 0; --back) {
-    if (pos - back < 0) continue;
-    float v[8];
-    ld8(back == 0 ? reinterpret_cast<const bf16*>(a.u) + (size_t)b * a.ldu + c : ring + (size_t)((pos - back) % a.ring_len) * C + c, v);
+  int slot = pos % a.ring_len;
+#pragma unroll 4
+  for (int back = 0; back < a.taps; ++back) {
+    if (pos - back >= 0) {
+      float v[8], x[8];
+      ld8(back == 0 ? u : ring + (size_t)slot * C, v);
+      ld8(w + (size_t)(a.taps - 1 - back) * C, x);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i] = fmaf(ldf(w + i * a.taps + a.taps - 1 - back), v[i], acc[i]);
+      for (int i = 0; i < 8; ++i) acc[i] = fmaf(x[i], v[i], acc[i]);
+    }
+    slot = slot == 0 ? a.ring_len - 1 : slot - 1;
   }
 }
 
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+
 template <int D, int MT, int NTW>
-__global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecodeArgs a, const int n_stages) {
+__global__ void __launch_bounds__(kDThreads, MT * NTW <= 8 ? 2 : 1)
+talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs a, const int n_stages) {
+  constexpr int kPl = D / 64;                                    // planes of 64 channels
   extern __shared__ __align__(1024) uint8_t td_smem[];
-  __shared__ int s_last;
   const WindowAttnArgs& p = a.at;
   const int H = p.H, G = p.G, grp = H / G, GD = G * D;
   const int stage_bytes = kDT * GD * 2;
-  uint8_t* sKV = td_smem;                                        // [stages][G][64][D], later the fp32 products [H][G * D]
-  uint8_t* sQ = sKV + n_stages * stage_bytes;
+  uint8_t* sKV = td_smem;                                        // [stages][G][planes][64][128 B], later the fp32 products [H][G * D]
+  uint8_t* sQ = sKV + n_stages * stage_bytes;                    // [MT][planes][16][128 B]
   uint8_t* sP = sQ + DecSmem<D, MT>::kQ;
   float* sMax = reinterpret_cast<float*>(sP + DecSmem<D, MT>::kP);   // [MT * 16][8]
   bf16* sKnew = reinterpret_cast<bf16*>(reinterpret_cast<uint8_t*>(sMax) + DecSmem<D, MT>::kMax);  // [G * D]
   float* sTalk = reinterpret_cast<float*>(sKnew + GD);           // [H][H]
+  uint64_t* full = reinterpret_cast<uint64_t*>(sTalk + ((H * H + 1) & ~1));  // [4]
+  int* s_last = reinterpret_cast<int*>(full + 4);
   const int split = blockIdx.x, b = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  pdl_wait();
-  pdl_launch();
+  // Lengths, tables and the keys of earlier tokens were complete before the kernel ahead of this one started.
   const int pos = p.seq_lens[b] - 1;
-  if (pos < 0) return;
+  if (pos < 0) {
+    pdl_wait();
+    pdl_launch();
+    return;
+  }
   const int C = H * D + GD;
   const int lo = pos - p.window + 1 > 0 ? pos - p.window + 1 : 0;
-  const int n_tiles = (pos - lo) / kDT + 1;
+  const int jb = (lo / 16) * 16;
+  const int n_tiles = (pos - jb) / kDT + 1;
   const int t_begin = (int)((long long)n_tiles * split / a.splits), t_end = (int)((long long)n_tiles * (split + 1) / a.splits);
   const bool newest = split == a.splits - 1;
   const int* table = p.block_tables + (size_t)b * p.max_blocks;
-  const bf16* cache = reinterpret_cast<const bf16*>(p.k_cache);
 
-  // Pages of the next tile to load, one per lane (a tile of 64 keys touches at most five): looked up one tile ahead, so that
-  // no copy waits for its table entry.
+  // Warp 0 issues the loads: lane -> page (lane & 3), which it looks up one tile ahead.
   int page = 0;
-  auto fetch_pages = [&](int t) {
-    const int bi = (lo + t * kDT) / 16 + lane;
-    if (t < t_end && lane < 5 && bi <= pos / 16) {
-      page = table[bi];
-      if (page < 0 || page >= p.num_cache_blocks) {
-        report_status(p.status, kStatusBadIndex);
-        page = 0;
-      }
+  auto fetch_page = [&](int t) {
+    if (t >= t_end) return;
+    int bi = (jb + t * kDT) / 16 + (lane & 3);
+    bi = bi > pos / 16 ? pos / 16 : bi;       // past the end: any valid page, masked
+    page = table[bi];
+    if (page < 0 || page >= p.num_cache_blocks) {
+      report_status(p.status, kStatusBadIndex);
+      page = 0;
     }
   };
-  auto load_tile = [&](int t, int stage) {
-    constexpr int kRowChunks = D / 8;
-    uint8_t* dst = sKV + stage * stage_bytes;
-    const int jt = lo + t * kDT, b0 = jt / 16;
-    const int n = kDT * G * kRowChunks;                      // a multiple of the CTA's threads: warps stay whole
-#pragma unroll 4
-    for (int i = tid; i < n; i += kDThreads) {
-      const int ch = i % kRowChunks, row = i / kRowChunks;   // row = m * 64 + key
-      const int m = row / kDT;
-      int j = jt + row % kDT;
-      const bool on = j < pos;                               // the newest key comes from sKnew, later ones are masked
-      const int blk = __shfl_sync(0xffffffffu, page, on ? j / 16 - b0 : 0);
-      j = on ? j : 0;
-      if (on) cp_async16(sw_chunk<D>(dst, row, ch), cache + (((size_t)blk * G + m) * 16 + j % 16) * D + ch * 8);
-      else if (row % kDT != pos - jt) *reinterpret_cast<uint4*>(sw_chunk<D>(dst, row, ch)) = make_uint4(0u, 0u, 0u, 0u);
+  auto load_tile = [&](int t, int stage) {    // warp 0
+    if (lane == 0) mbar_expect_tx(&full[stage], stage_bytes);
+    __syncwarp();
+    for (int i = lane >> 2; i < G * kPl; i += 8) {
+      const int m = i / kPl, pl = i % kPl;
+      tma_load_2d(sKV + stage * stage_bytes + (i * kDT + (lane & 3) * 16) * 128, &tmK, &full[stage], pl * 64, (page * G + m) * 16);
     }
-    fetch_pages(t + 1);
+    fetch_page(t + 1);
   };
-  // loads first: they do not depend on the new token
-  fetch_pages(t_begin);
-  for (int i = 0; i < n_stages - 1; ++i) {
-    if (t_begin + i < t_end) load_tile(t_begin + i, i);
-    cp_async_commit();
+  if (warp == 0) {
+    if (lane == 0) {
+      for (int i = 0; i < 4; ++i) mbar_init(&full[i], 1);
+      fence_mbar_init();
+    }
+    __syncwarp();
+    fetch_page(t_begin);
+    for (int i = 0; i < n_stages - 1; ++i)
+      if (t_begin + i < t_end) load_tile(t_begin + i, i);
   }
+  if (p.talk != nullptr)
+    for (int i = tid; i < H * H; i += kDThreads) sTalk[i] = ldf(reinterpret_cast<const bf16*>(p.talk) + i);
+  pdl_wait();
+  pdl_launch();
   for (int i = tid; i < MT * 16 * (D / 8); i += kDThreads) {
     const int row = i / (D / 8), ch = i % (D / 8);
     float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
     if (row < H) conv8(a, b, pos, C, row * D + ch * 8, v);
-    st8(reinterpret_cast<bf16*>(sw_chunk<D>(sQ, row, ch)), v);
+    st8(reinterpret_cast<bf16*>(sQ + ((row >> 4) * kPl + (ch >> 3)) * 2048 + sw_off(row & 15, ch & 7)), v);
   }
   if (newest) {
     int blk = table[pos / 16];
@@ -549,13 +567,36 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
       for (int i = tid * 8; i < C; i += kDThreads * 8) *reinterpret_cast<uint4*>(ring + i) = *reinterpret_cast<const uint4*>(u + i);
     }
   }
-  if (p.talk != nullptr)
-    for (int i = tid; i < H * H; i += kDThreads) sTalk[i] = ldf(reinterpret_cast<const bf16*>(p.talk) + i);
 
   const float qs = p.qscale[pos < p.qscale_len ? pos : p.qscale_len - 1];
   const int npw = (GD / 8 + 7) / 8;              // 8-wide value-column tiles per warp
   const int nt0 = warp * npw;
   const int r0 = lane >> 2, cq = (lane & 3) * 2;
+  // fragment addresses that do not change from tile to tile (inside a stage)
+  const uint32_t k_off = sw_off(warp * 8 + (lane & 7), lane >> 3);                       // keys: chunks 0-3; chunks 4-7 at ^ 64
+  const uint32_t q_off = smem_u32(sQ) + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, lane >> 4);  // queries: k-step s at ^ (s * 32)
+  const uint32_t p_off = smem_u32(sP) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + (lane >> 4) * 8) * 2;
+  constexpr int kPairs = NTW > 1 ? NTW / 2 : 1;
+  uint32_t v_off[kPairs];                        // value columns: two neighbouring 8-wide tiles per ldmatrix
+#pragma unroll
+  for (int i = 0; i < kPairs; ++i) {
+    const int n1 = nt0 + 2 * i < GD / 8 ? nt0 + 2 * i : GD / 8 - 1;
+    const int n2 = n1 + 1 < GD / 8 ? n1 + 1 : n1;
+    const int nn = (lane >> 4) ? n2 : n1;
+    const int m = nn / (D / 8), ch = nn % (D / 8);
+    v_off[i] = (m * kPl + (ch >> 3)) * (kDT * 128) + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, ch & 7);
+  }
+  const float* bias_row[MT][2];                  // rows past the last head read the last head's biases; they are never stored
+  int key_head[MT][2];
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      int h = mt * 16 + r0 + q * 8;
+      h = h < H ? h : H - 1;
+      bias_row[mt][q] = p.bias + (size_t)h * p.bias_len;
+      key_head[mt][q] = h / grp;
+    }
   float acc[MT][NTW][4];
   float mrow[MT][2], lrow[MT][2];
 #pragma unroll
@@ -567,65 +608,78 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
     mrow[t][0] = mrow[t][1] = -INFINITY;
     lrow[t][0] = lrow[t][1] = 0.f;
   }
-  __syncthreads();  // q, the new key and the mixing matrix are in shared memory
+  __syncthreads();  // barriers, q, the new key and the mixing matrix are in shared memory
   int stage = 0;
+  uint32_t phase = 0;
+  bool ok = true;
   for (int t = t_begin; t < t_end; ++t) {
     if (n_stages == 1) {
       __syncthreads();
-      load_tile(t, 0);
-      cp_async_commit();
-      cp_async_wait<0>();
-    } else if (n_stages == 2) {
-      cp_async_wait<0>();
-    } else {
-      cp_async_wait<1>();
+      if (warp == 0) load_tile(t, 0);
+    }
+    const int j0 = jb + t * kDT;
+    const bool inside = j0 >= lo && j0 + kDT - 1 <= pos && pos - j0 < p.bias_len;
+    float bv[MT][4];                             // distance biases, on their way while the tile arrives
+    {
+      const int d = pos - (j0 + warp * 8 + cq);
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int de = d - (e & 1);
+          if (inside) bv[mt][e] = __ldg(bias_row[mt][e >> 1] + de);
+          else bv[mt][e] = de >= 0 && de < p.window && de < p.bias_len ? __ldg(bias_row[mt][e >> 1] + de) : INFINITY;
+        }
+    }
+    if (ok && !mbar_wait(&full[stage], phase)) {
+      report_status(p.status, kStatusWaitFullTimeout);
+      ok = false;
     }
     uint8_t* kt = sKV + stage * stage_bytes;
-    const int j0 = lo + t * kDT;
+    const uint32_t kts = smem_u32(kt);
     if (newest && t == t_end - 1) {
       const int key = pos - j0;
       for (int i = tid; i < GD / 8; i += kDThreads) {
         const int m = i / (D / 8), ch = i % (D / 8);
-        *reinterpret_cast<uint4*>(sw_chunk<D>(kt, m * kDT + key, ch)) = *reinterpret_cast<const uint4*>(sKnew + i * 8);
+        *reinterpret_cast<uint4*>(kt + (m * kPl + (ch >> 3)) * (kDT * 128) + sw_off(key, ch & 7)) = *reinterpret_cast<const uint4*>(sKnew + i * 8);
       }
-    }
-    __syncthreads();  // the tile is complete; everybody is done with the stage that is loaded next
-    if (n_stages > 1) {
-      const int nxt = t + n_stages - 1;
-      if (nxt < t_end) load_tile(nxt, stage == 0 ? n_stages - 1 : stage - 1);
-      cp_async_commit();
+      __syncthreads();
     }
     // ---- scores of keys [8 warp, 8 warp + 8) for all heads ----
-    float s[MT][4], bv[MT][4];
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {  // distance biases, on their way while the MMAs run
-        const int h = mt * 16 + r0 + (e >> 1) * 8;
-        const int d = pos - (j0 + warp * 8 + cq + (e & 1));
-        const bool on = h < H && d >= 0 && d < p.window && d < p.bias_len;
-        bv[mt][e] = on ? __ldg(p.bias + (size_t)h * p.bias_len + d) : INFINITY;
-      }
+    float s[MT][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       s[mt][0] = s[mt][1] = s[mt][2] = s[mt][3] = 0.f;
-      const int h_lo = mt * 16, h_hi = (mt * 16 + 16 < H ? mt * 16 + 16 : H) - 1;
-      const int ka = (h_lo + r0) / grp, kb = (h_lo + r0 + 8) / grp;   // key heads of this thread's two rows
-      for (int m = h_lo / grp; m <= h_hi / grp && h_hi >= h_lo; ++m) {
-        const bool ua = ka == m, ub = kb == m;
+      if (mt * 16 < H) {
+        const int m_lo = mt * 16 / grp, m_hi = ((mt * 16 + 16 < H ? mt * 16 + 16 : H) - 1) / grp;
+        for (int m = m_lo; m <= m_hi; ++m) {
+          float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int kk = 0; kk < D / 32; ++kk) {
-          uint32_t kf[4];  // two k-steps of 16 for 8 keys
-          ldmatrix_x4(kf, sw_chunk<D>(kt, m * kDT + warp * 8 + (lane & 7), kk * 4 + (lane >> 3)));
-#pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            uint32_t qf[4];
-            ldmatrix_x4(qf, sw_chunk<D>(sQ, h_lo + (lane & 7) + ((lane >> 3) & 1) * 8, (kk * 2 + half) * 2 + (lane >> 4)));
-            mma_16816(s[mt], ua ? qf[0] : 0u, ub ? qf[1] : 0u, ua ? qf[2] : 0u, ub ? qf[3] : 0u, kf[half * 2], kf[half * 2 + 1]);
+          for (int pl = 0; pl < kPl; ++pl) {
+            const uint32_t ka = kts + (m * kPl + pl) * (kDT * 128) + k_off;
+            const uint32_t qa = q_off + (mt * kPl + pl) * 2048;
+            uint32_t k0[4], k1[4], q0[4], q1[4], q2[4], q3[4];
+            ldsm4(k0, ka);
+            ldsm4(q0, qa);
+            ldsm4(q1, qa ^ 32);
+            ldsm4(k1, ka ^ 64);
+            ldsm4(q2, qa ^ 64);
+            ldsm4(q3, qa ^ 96);
+            mma_16816(c0, q0[0], q0[1], q0[2], q0[3], k0[0], k0[1]);
+            mma_16816(c1, q1[0], q1[1], q1[2], q1[3], k0[2], k0[3]);
+            mma_16816(c0, q2[0], q2[1], q2[2], q2[3], k1[0], k1[1]);
+            mma_16816(c1, q3[0], q3[1], q3[2], q3[3], k1[2], k1[3]);
+          }
+          if (key_head[mt][0] == m) {
+            s[mt][0] = c0[0] + c1[0];
+            s[mt][1] = c0[1] + c1[1];
+          }
+          if (key_head[mt][1] == m) {
+            s[mt][2] = c0[2] + c1[2];
+            s[mt][3] = c0[3] + c1[3];
           }
         }
       }
-      // scale, distance bias, mask; row maxima over this warp's keys
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[mt][e] = fmaf(s[mt][e], qs, -bv[mt][e]);  // masked: minus infinity
 #pragma unroll
@@ -633,10 +687,14 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
         float mx = fmaxf(s[mt][2 * q], s[mt][2 * q + 1]);
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        if ((lane & 3) == 0) sMax[(h_lo + r0 + q * 8) * 8 + warp] = mx;
+        if ((lane & 3) == 0) sMax[(mt * 16 + r0 + q * 8) * 8 + warp] = mx;
       }
     }
-    __syncthreads();
+    __syncthreads();  // maxima; everybody is done with the products of the tile before, whose stage is loaded next
+    if (n_stages > 1 && warp == 0) {
+      const int nxt = t + n_stages - 1;
+      if (nxt < t_end) load_tile(nxt, stage == 0 ? n_stages - 1 : stage - 1);
+    }
     // ---- weights ----
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
@@ -668,31 +726,25 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
     for (int kk = 0; kk < kDT / 16; ++kk) {
       uint32_t pf[MT][4];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
-        ldmatrix_x4(pf[mt], sP + ((mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + kk * 16 + (lane >> 4) * 8) * 2);
+      for (int mt = 0; mt < MT; ++mt) ldsm4(pf[mt], p_off + (mt * 16 * kPPitch + kk * 16) * 2);
 #pragma unroll
-      for (int i = 0; i < NTW; i += (NTW > 1 ? 2 : 1)) {
-        if (i < npw && nt0 + i < GD / 8) {
-          // x4: two neighbouring column tiles (the second one may belong to the next warp; it is then not used)
-          const int n1 = nt0 + i;
-          const int n2 = n1 + 1 < GD / 8 ? n1 + 1 : n1;
-          const int nn = (lane >> 4) ? n2 : n1;
-          const int m = nn / (D / 8), ch = nn % (D / 8);
+      for (int i = 0; i < kPairs; ++i) {
+        if (2 * i < npw) {   // columns past the end repeat the last ones; they are never stored
           uint32_t vf[4];
-          ldmatrix_x4_trans(vf, sw_chunk<D>(kt, m * kDT + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, ch));
+          ldsm4_t(vf, kts + v_off[i] + kk * 2048);
 #pragma unroll
           for (int mt = 0; mt < MT; ++mt) {
-            mma_16816(acc[mt][i], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[0], vf[1]);
-            if constexpr (NTW > 1) {
-              if (i + 1 < npw) mma_16816(acc[mt][i + 1], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[2], vf[3]);
-            }
+            mma_16816(acc[mt][2 * i], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[0], vf[1]);
+            if constexpr (NTW > 1) mma_16816(acc[mt][2 * i + 1], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[2], vf[3]);
           }
         }
       }
     }
-    stage = stage + 1 == n_stages ? 0 : stage + 1;
+    if (++stage == n_stages) {
+      stage = 0;
+      phase ^= 1;
+    }
   }
-  cp_async_wait<0>();
   __syncthreads();
   // ---- row sums over the warps ----
 #pragma unroll
@@ -730,11 +782,11 @@ __global__ void __launch_bounds__(kDThreads) talk_decode_kernel(const TalkDecode
     __syncthreads();
     if (tid == 0) {
       const int ticket = atomicAdd(a.tickets + b, 1);
-      s_last = ticket == a.splits - 1;
-      if (s_last) a.tickets[b] = 0;
+      *s_last = ticket == a.splits - 1;
+      if (*s_last) a.tickets[b] = 0;
     }
     __syncthreads();
-    if (!s_last) return;
+    if (!*s_last) return;
     __threadfence();
     float* wgt = sMax;  // [H][splits] merge weights, splits <= 8
     for (int h = tid; h < H; h += kDThreads) {
@@ -805,13 +857,13 @@ DecPlan plan_decode_kernel(int H, int G, int D) {
   while (ntw < npw) ntw *= 2;
   if (ntw > 16 || mt * ntw > 32) return d;
   const size_t stage = (size_t)kDT * G * D * 2;
-  const size_t fixed = (size_t)mt * 16 * D * 2 + (size_t)mt * 16 * kPPitch * 2 + (size_t)mt * 16 * 32 + (size_t)G * D * 2 + (size_t)H * H * 4;
+  const size_t fixed = (size_t)mt * 16 * D * 2 + (size_t)mt * 16 * kPPitch * 2 + (size_t)mt * 16 * 32 + (size_t)G * D * 2 + (size_t)(H * H + 1) * 4 + 64;
   const size_t prod = (size_t)H * G * D * 4;
-  int st = 3;
-  while (st > 1 && st * stage + fixed > (size_t)110 * 1024) --st;  // two CTAs per SM while that leaves two stages
-  if (st < 2) {
-    st = 2;
-    if (st * stage + fixed > (size_t)224 * 1024) st = 1;
+  int st = 4;
+  while (st > 1 && st * stage + fixed > (size_t)112 * 1024) --st;
+  if (st < 2 || mt * ntw > 8) {  // one CTA per SM: as many stages as fit
+    st = 4;
+    while (st > 1 && st * stage + fixed > (size_t)224 * 1024) --st;
   }
   if (st * stage < prod) return d;
   if (st * stage + fixed > (size_t)224 * 1024) return d;
@@ -824,7 +876,8 @@ void launch_decode_t(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) 
   auto kernel = talk_decode_kernel<D, MT, NTW>;
   AGRPO_SET_MAX_DYN_SMEM(kernel, 226 * 1024, "talk_decode smem attr");
   AGRPO_PREFER_SMEM(kernel);
-  launch_kernel(kernel, dim3(a.splits, a.at.T), dim3(kDThreads), d.smem, s, "talk_decode", a, d.stages);
+  const CUtensorMap tk = make_tmap_2d(a.k_cache, D, (uint64_t)a.at.num_cache_blocks * a.at.G * 16, D, 64, 16);
+  launch_kernel(kernel, dim3(a.splits, a.at.T), dim3(kDThreads), d.smem, s, "talk_decode", tk, a, d.stages);
 }
 template <int D, int MT>
 void launch_decode_n(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) {

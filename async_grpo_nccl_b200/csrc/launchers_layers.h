@@ -24,7 +24,7 @@ struct DytTail {
 void launch_embed_dyt(bool fp32, const int* ids, const void* table, float scale, float* x, void* h, const DytArgs& norm, int T, int W, int V,
                       cudaStream_t s);
 
-// Causal short convolution of the first `q_cols + k_cols` columns of u [T, ldu] (weights [q_cols + k_cols, taps]). The q
+// Causal short convolution of the first `q_cols + k_cols` columns of u [T, ldu] (weights [taps, q_cols + k_cols], the current token's last). The q
 // part goes to q_out [T, q_cols], the k part to its place in the paged cache [blocks, G, block_size, D]. Values of tokens
 // before the segment come from the sequence's ring [slots, ring_len, q_cols + k_cols] (position p at p % ring_len; slots are
 // ring_pitch elements apart).

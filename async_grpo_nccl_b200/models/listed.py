@@ -95,12 +95,14 @@ class ListedDecoder:
         return n
 
     def refresh_tables(self) -> None:
-        """Tables that follow from the configuration and the weights, computed in 64-bit: the distance bias of every head
-        (entry d = r1 ln(1 + r2 d)) and the score factor of a query at each position (scale x temperature), both in
-        log2 units. They keep their storage when the weights change, so captured graphs stay valid."""
+        """Tables that follow from the configuration and the weights: the distance bias of every head (entry d =
+        r1 ln(1 + r2 d)) and the score factor of a query at each position (scale x temperature), both computed in 64-bit
+        and in log2 units, and the convolution weights with the channels contiguous. They keep their storage when the weights change, so captured graphs stay valid."""
         if not hasattr(self, "bias"):
             self.bias: List[torch.Tensor] = []
             self.qscale: List[torch.Tensor] = []
+            self.conv: List[torch.Tensor] = [torch.empty(l.mixer.conv, l.mixer.qk_dim, dtype=self.dtype, device=self.dev)
+                                             for l in self.cfg.layers]
             shared: Dict[Tuple[float, float, float], torch.Tensor] = {}
             for l in self.cfg.layers:
                 m = l.mixer
@@ -112,6 +114,7 @@ class ListedDecoder:
                     shared[key] = (temp * (m.scale * LOG2E)).float().to(self.dev)
                 self.qscale.append(shared[key])
         for i, t in enumerate(self.bias):
+            self.conv[i].copy_(self.w(f"layers.{i}.conv").t())
             d = torch.arange(t.shape[1], dtype=torch.float64, device=self.dev)
             r1, r2 = self.w(f"layers.{i}.r1").double(), self.w(f"layers.{i}.r2").double()
             t.copy_(r1[:, None] * torch.log1p(r2[:, None] * d[None]) * LOG2E)
@@ -158,11 +161,11 @@ class ListedDecoder:
         m, C, p = self.cfg.layers[i].mixer, self.C, f"layers.{i}."
         gate = u[:, m.qk_dim:]
         if sb.rows is None and sb.scratch is not None and self.tensor_core_decode(i):
-            C.talk_attn_decode(u, self.w(p + "conv"), ring, k_cache, sb.seq_lens, sb.block_tables, self.bias[i], self.qscale[i],
+            C.talk_attn_decode(u, self.conv[i], ring, k_cache, sb.seq_lens, sb.block_tables, self.bias[i], self.qscale[i],
                                self.w(p + "talk"), gate, m.window, out, sb.splits, *sb.scratch, self.status)
             self.launches += 1
             return
-        C.short_conv(u, self.w(p + "conv"), ring, sb.rows, sb.ring_rows[m.conv] if sb.rows is not None else None, sb.seq_lens, sb.block_tables, q, k_cache, self.status)
+        C.short_conv(u, self.conv[i], ring, sb.rows, sb.ring_rows[m.conv] if sb.rows is not None else None, sb.seq_lens, sb.block_tables, q, k_cache, self.status)
         if sb.rows is not None and not self.fp32:
             acc = torch.empty(sb.T * m.heads * m.k_dim, dtype=self.dtype, device=self.dev)
             if C.talk_attn_prefill(q, k_cache, sb.tiles, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate, m.window,

@@ -130,7 +130,7 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
     bias = torch.rand(H, min(m.window, maxlen), device=dev)
     qscale = torch.full((maxlen,), 0.1, device=dev)
     talk = (torch.eye(H, device=dev) + 0.02 * torch.randn(H, H, device=dev)).to(bf)
-    conv = R(m.qk_dim, m.conv)
+    conv = R(m.conv, m.qk_dim)
 
     # ---------------- prompts ----------------
     h, x, ho = R(T, W), torch.randn(T, W, device=dev), torch.empty(T, W, device=dev, dtype=bf)

@@ -267,7 +267,7 @@ class AttnCase:
         u = torch.cat([self.uq.flatten(1), self.uk.flatten(1), self.gate], 1).to(self.dt).to(dev)
         cache = torch.full((self.nblk, self.G, 16, self.D), 3.0, device=dev, dtype=self.dt)  # stale values everywhere
         ring = torch.full((3, self.taps, (self.H + self.G) * self.D), -2.0, device=dev, dtype=self.dt)
-        return u, cache, ring, self.conv.to(self.dt).to(dev), self.talk.to(self.dt).to(dev), self.tables.to(dev)
+        return u, cache, ring, self.conv.t().contiguous().to(self.dt).to(dev), self.talk.to(self.dt).to(dev), self.tables.to(dev)
 
     def oracle(self):
         """Output [n, H * D] (q and k rounded as the kernels store them)."""
