@@ -27,15 +27,15 @@ typedef __nv_bfloat16 bf16;
 // ================================================================================================
 // Prompts: one CTA = 128 query rows of one head g, value heads [m0, m0 + mc). S (two buffers, so that the scores of tile
 // j + 1 are computed while the softmax of tile j runs) and the mc accumulators fill tensor memory. Warp 0 loads key tiles
-// page by page, warp 1 issues MMAs, warps 2-17 run the softmax: four threads per query row, 32 keys each (with fewer warps
-// the softmax is bound by latency and the tensor cores wait for it). The key tile of a head serves as K-major operand of
-// Q K^T and as MN-major operand of P V.
+// page by page, warp 1 issues MMAs, warps 2-17 run the softmax in two groups that take alternating tiles (one group's loads
+// and maxima overlap the other's exponentials); in a group two threads share a query row, 64 keys each. The reference maximum
+// of a row is handed from tile to tile through shared memory, so that all weights of a row are on one scale. The key tile of a
+// head serves as K-major operand of Q K^T and as MN-major operand of P V.
 // ================================================================================================
 constexpr int kPM = 128;
 constexpr int kPN = 128;
-constexpr int kPParts = 4;                            // threads per query row
-constexpr int kPKeys = kPN / kPParts;                // keys per thread and tile
-constexpr int kPThreads = 64 + kPParts * kPM;
+constexpr int kPKeys = 64;                            // keys per thread and tile
+constexpr int kPThreads = 64 + 4 * kPM;
 constexpr int kRingBytes = 192 * 1024;
 
 struct TalkPrefillParams {
@@ -53,7 +53,8 @@ struct TalkPrefillParams {
   int* status;
 };
 
-__device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 512;" ::: "memory"); }
+__device__ __forceinline__ void softmax_group_bar(int group) { asm volatile("bar.sync %0, 256;" ::"r"(group + 1) : "memory"); }
+__device__ __forceinline__ void softmax_all_bar() { asm volatile("bar.sync 3, 512;" ::: "memory"); }
 
 template <int D>
 __global__ void __launch_bounds__(kPThreads, 1)
@@ -65,16 +66,18 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   extern __shared__ __align__(1024) uint8_t tp_smem[];
   uint8_t* sQ = tp_smem;
   uint8_t* sK = tp_smem + kTile;
-  float* smax = reinterpret_cast<float*>(sK + kRingBytes);   // 2 KB: row maxima [2 parities][4 parts][128] as bf16, at the end sums
+  float* smax = reinterpret_cast<float*>(sK + kRingBytes);   // 2 KB: row maxima [2 groups][2 turns][2 halves][128] as bf16, at the end sums
   bf16* smax16 = reinterpret_cast<bf16*>(smax);
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smax + 512);
+  bf16* sref = reinterpret_cast<bf16*>(smax + 512);          // [2][128] reference maximum after the latest even / odd tile
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sref + 256);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;      // [3]
   uint64_t* k_empty = bars + 4;     // [3]
   uint64_t* s_full = bars + 7;      // [2]
-  uint64_t* p_ready = bars + 9;
-  uint64_t* o_done = bars + 10;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 11);
+  uint64_t* p_ready = bars + 9;     // [2]
+  uint64_t* ref_set = bars + 11;    // [2]
+  uint64_t* o_done = bars + 13;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.x;
@@ -100,7 +103,10 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
     mbar_init(&s_full[0], 1);
     mbar_init(&s_full[1], 1);
-    mbar_init(p_ready, 4 * kPParts);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&p_ready[i], 8);
+      mbar_init(&ref_set[i], 8);
+    }
     mbar_init(o_done, 1);
     fence_mbar_init();
   }
@@ -198,7 +204,7 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           tc_fence_after();
           scores(j + 1, nstage);
         }
-        if (!mbar_wait(p_ready, j & 1)) {
+        if (!mbar_wait(&p_ready[j & 1], (j >> 1) & 1)) {
           report_status(p.status, kStatusWaitTmemFullTimeout);
           break;
         }
@@ -220,20 +226,21 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
     }
   } else {
-    // ---------------- softmax: thread = (query row, quarter of the tile's keys) ----------------
-    const int quarter = warp & 3, part = (warp - 2) >> 2;
+    // ---------------- softmax: thread = (query row, half of the keys of every second tile) ----------------
+    const int group = (warp - 2) >> 3, half = ((warp - 2) >> 2) & 1, quarter = warp & 3;
+    const int part = group * 2 + half;
     const int r = quarter * 32 + lane;
     const int qi = pos0 + r;
     const uint32_t lane_off = static_cast<uint32_t>(quarter * 32) << 16;
     const float qs = p.qscale[qi < p.qscale_len ? qi : p.qscale_len - 1];
     const float* bias = p.bias + (size_t)head * p.bias_len;
-    const int o_cols = mc * D / kPParts;      // accumulator columns that this thread rescales and stores
-    const uint32_t tO = tmem_O + lane_off + part * o_cols;
-    float m = -INFINITY, l = 0.f;
+    const int h_cols = mc * D / 2;            // accumulator columns that this thread rescales
+    const uint32_t tS = tmem + group * 128 + lane_off;
+    float m = -INFINITY, l = 0.f;             // reference maximum of this group's latest tile, sum of its weights on that scale
     bool ok = true;                           // after a failure the barriers are still met, nothing else is waited for
-    for (int j = 0; j < n_kv; ++j) {
+    for (int j = group; j < n_kv; j += 2) {
       const int tk = j0 + j * kPN;            // first key of the tile
-      const int d0 = qi - (tk + part * kPKeys);  // distance of this thread's first key
+      const int d0 = qi - (tk + half * kPKeys);  // distance of this thread's first key
       const bool inside = tk + kPN - 1 <= pos0 && pos0 + kPM - 1 - tk < p.window && pos0 + kPM - 1 - tk < p.bias_len;
       float v[kPKeys];                        // distance biases, on their way while the scores are computed
       if (inside) {
@@ -246,35 +253,44 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           v[i] = d >= 0 && d < p.window && d < p.bias_len ? __ldg(bias + d) : INFINITY;
         }
       }
-      if (ok && !mbar_wait(&s_full[j & 1], (j >> 1) & 1)) {
+      if (ok && !mbar_wait(&s_full[group], (j >> 1) & 1)) {
         report_status(p.status, kStatusWaitTmemFullTimeout);
         ok = false;
       }
       tc_fence_after();
-      const uint32_t tS = tmem + (j & 1) * 128 + lane_off;
-      uint32_t s0[32];
-      tmem_ld_32x32(tS + part * kPKeys, s0);
-      tc_wait_ld();
+      float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-      for (int i = 0; i < kPKeys; ++i) v[i] = fmaf(__uint_as_float(s0[i]), qs, -v[i]);  // masked keys: minus infinity
-      float mx4[4] = {v[0], v[1], v[2], v[3]};
+      for (int c = 0; c < kPKeys; c += 16) {
+        uint32_t s0[16];
+        tmem_ld_32x16(tS + half * kPKeys + c, s0);
+        tc_wait_ld();
 #pragma unroll
-      for (int i = 4; i < kPKeys; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], v[i]);
-      // the maximum is only a reference point: exchanged in bf16, the same rounded value for all threads of a row
-      smax16[((j & 1) * kPParts + part) * 128 + r] = __float2bfloat16(fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])));
-      tc_fence_before();
-      softmax_bar();                          // everybody has read the scores: the weights may overwrite them
-      tc_fence_after();
-      float mx = -INFINITY;
-#pragma unroll
-      for (int e = 0; e < kPParts; ++e) mx = fmaxf(mx, __bfloat162float(smax16[((j & 1) * kPParts + e) * 128 + r]));
-      // keep a stale maximum unless it grew by more than 2^8: the weights stay bounded and O rarely needs rescaling
-      float alpha = 1.f;
-      if (mx > m + 8.f || m == -INFINITY) {
-        if (m != -INFINITY) alpha = exp2f(m - mx);  // nothing has been accumulated before the first visible key
-        m = mx;
+        for (int i = 0; i < 16; ++i) {
+          v[c + i] = fmaf(__uint_as_float(s0[i]), qs, -v[c + i]);  // masked keys: minus infinity
+          mx4[i & 3] = fmaxf(mx4[i & 3], v[c + i]);
+        }
       }
-      const float base = m == -INFINITY ? 0.f : m;
+      // the maximum is only a reference point: kept in bf16, the same rounded value for all threads of a row
+      bf16* mine = smax16 + (group * 2 + ((j >> 1) & 1)) * 256;
+      mine[half * 128 + r] = __float2bfloat16(fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])));
+      tc_fence_before();
+      softmax_group_bar(group);               // both halves have read their scores: the weights may overwrite them
+      tc_fence_after();
+      const float mx = fmaxf(__bfloat162float(mine[r]), __bfloat162float(mine[128 + r]));
+      float m_prev = -INFINITY;               // scale of what is accumulated so far
+      if (j > 0) {
+        if (ok && !mbar_wait(&ref_set[group ^ 1], ((j - 1) >> 1) & 1)) {
+          report_status(p.status, kStatusWaitTmemFullTimeout);
+          ok = false;
+        }
+        m_prev = __bfloat162float(sref[(group ^ 1) * 128 + r]);
+      }
+      // keep a stale maximum unless it grew by more than 2^8: the weights stay bounded and O rarely needs rescaling
+      const float m_new = (mx > m_prev + 8.f || m_prev == -INFINITY) ? mx : m_prev;
+      if (half == 0) sref[group * 128 + r] = __float2bfloat16(m_new);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&ref_set[group]);
+      const float alpha = m_prev == -INFINITY ? 1.f : exp2f(m_prev - m_new);  // nothing is accumulated before the first visible key
       if (__any_sync(0xffffffffu, alpha != 1.f)) {
         if (ok && !mbar_wait(o_done, (j - 1) & 1)) {
           report_status(p.status, kStatusWaitTmemFullTimeout);
@@ -282,50 +298,62 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         }
         tc_fence_after();
 #pragma unroll 1
-        for (int c = 0; c < o_cols; c += 16) {
+        for (int c = 0; c < h_cols; c += 16) {
+          const uint32_t ta = tmem_O + lane_off + half * h_cols + c;
           uint32_t o[16];
-          tmem_ld_32x16(tO + c, o);
+          tmem_ld_32x16(ta, o);
           tc_wait_ld();
 #pragma unroll
           for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
-          tmem_st_32x16(tO + c, o);
+          tmem_st_32x16(ta, o);
         }
-        l *= alpha;
       }
-      uint32_t w[kPKeys / 2];
+      if (m != m_new) l *= m == -INFINITY ? 0.f : exp2f(m - m_new);
+      m = m_new;
+      const float base = m == -INFINITY ? 0.f : m;
       float l0 = 0.f, l1 = 0.f;
 #pragma unroll
-      for (int i = 0; i < kPKeys / 2; ++i) {
-        const float a = exp2f(v[2 * i] - base), b = exp2f(v[2 * i + 1] - base);
-        l0 += a;
-        l1 += b;
-        w[i] = pack_bf16x2(a, b);
+      for (int c = 0; c < kPKeys; c += 32) {
+        uint32_t w[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float a = exp2f(v[c + 2 * i] - base), b = exp2f(v[c + 2 * i + 1] - base);
+          l0 += a;
+          l1 += b;
+          w[i] = pack_bf16x2(a, b);
+        }
+        tmem_st_32x16(tS + half * (kPKeys / 2) + c / 2, w);
       }
       l += l0 + l1;
-      tmem_st_32x16(tS + part * (kPKeys / 2), w);
       tc_wait_st();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_ready);
+      if (lane == 0) mbar_arrive(&p_ready[group]);
     }
-    // the threads of a row add up their sums
-    softmax_bar();
+    // the four threads of a row add up their sums on the scale of the last tile
+    const int last = (n_kv - 1) & 1;
+    if (ok && !mbar_wait(&ref_set[last], ((n_kv - 1) >> 1) & 1)) {
+      report_status(p.status, kStatusWaitTmemFullTimeout);
+      ok = false;
+    }
+    const float m_end = __bfloat162float(sref[last * 128 + r]);
+    if (m != m_end) l *= m == -INFINITY ? 0.f : exp2f(m - m_end);
+    softmax_all_bar();
     smax[part * 128 + r] = l;
-    softmax_bar();
-    l = 0.f;
-#pragma unroll
-    for (int e = 0; e < kPParts; ++e) l += smax[e * 128 + r];
+    softmax_all_bar();
+    l = (smax[r] + smax[128 + r]) + (smax[256 + r] + smax[384 + r]);
     if (ok && !mbar_wait(o_done, (n_kv - 1) & 1)) {
       report_status(p.status, kStatusWaitTmemFullTimeout);
       ok = false;
     }
     tc_fence_after();
     const float inv = l > 0.f ? 1.f / l : 0.f;
+    const int o_cols = mc * D / 4;
     bf16* dst = p.acc + (((size_t)(tile.x + r) * p.H + head) * p.G + m0) * D + part * o_cols;
 #pragma unroll 1
     for (int c = 0; c < o_cols; c += 16) {
       uint32_t o[16];
-      tmem_ld_32x16(tO + c, o);
+      tmem_ld_32x16(tmem_O + lane_off + part * o_cols + c, o);
       tc_wait_ld();
       if (ok && r < n_rows) {
 #pragma unroll
@@ -417,21 +445,20 @@ talk_mix_gate_kernel(const bf16* __restrict__ acc, const bf16* __restrict__ talk
 
 template <int D>
 void launch_prefill_t(const CUtensorMap& tq, const CUtensorMap& tk, const TalkPrefillParams& p, int n_tiles, int chunks, cudaStream_t s) {
-  constexpr int smem = kPM * D * 2 + kRingBytes + 512 * 4 + 128;
+  constexpr int smem = kPM * D * 2 + kRingBytes + 512 * 4 + 256 * 2 + 128;
   auto kernel = talk_prefill_kernel<D>;
   AGRPO_SET_MAX_DYN_SMEM(kernel, smem, "talk_prefill smem attr");
   launch_kernel(kernel, dim3(p.H, chunks, n_tiles), dim3(kPThreads), smem, s, "talk_prefill", tq, tk, p);
 }
 
 // ================================================================================================
-// Decode: CTA = (split, sequence), 8 warps, all heads. The prologue convolves the new token's q (every split) and k (the
+// Decode: CTA = (split, sequence), all heads: 8 warps per MTW row tiles of 16 heads plus one warp that loads. The prologue convolves the new token's q (every split) and k (the
 // split that owns the newest token, which also writes the key page and the ring). Key tiles of 64 tokens arrive by TMA, page
-// by page, from before the new token's projections are complete. Per tile: warp w scores its 8 keys against all heads, the
-// CTA agrees on the row maxima, the weights meet in shared memory, and warp w accumulates its share of the G * D value
-// columns for all heads. The last split of a sequence to finish merges, mixes, gates and stores.
+// by page, from before the new token's projections are complete. Per tile: a warp scores its 8 keys against its heads, the
+// CTA agrees on the row maxima, the weights meet in shared memory, and the warp accumulates its share of the G * D value
+// columns for its heads. The last split of a sequence to finish merges, mixes, gates and stores.
 // ================================================================================================
 constexpr int kDT = 64;         // keys per tile
-constexpr int kDThreads = 256;
 constexpr int kPPitch = kDT + 8;
 
 template <int D, int MT>
@@ -474,10 +501,17 @@ __device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-template <int D, int MT, int NTW>
-__global__ void __launch_bounds__(kDThreads, MT * NTW <= 8 ? 2 : 1)
+template <int N>
+__device__ __forceinline__ void compute_bar() { asm volatile("bar.sync 1, %0;" ::"n"(N) : "memory"); }
+
+// MW groups of 8 warps, MTW row tiles of 16 heads per warp, up to NTW 8-wide value-column tiles per warp
+template <int D, int MW, int MTW, int NTW>
+__global__ void __launch_bounds__(MW * 256 + 32, (MW == 1 && NTW <= 4) ? 2 : 1)
 talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs a, const int n_stages) {
+  constexpr int MT = MW * MTW;
+  constexpr int kDThreads = MW * 256;                            // computing threads
   constexpr int kPl = D / 64;                                    // planes of 64 channels
+  constexpr bool kQReg = MTW == 1 && NTW <= (MW == 1 ? 8 : 4);                   // query fragments stay in registers
   extern __shared__ __align__(1024) uint8_t td_smem[];
   const WindowAttnArgs& p = a.at;
   const int H = p.H, G = p.G, grp = H / G, GD = G * D;
@@ -489,7 +523,8 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
   bf16* sKnew = reinterpret_cast<bf16*>(reinterpret_cast<uint8_t*>(sMax) + DecSmem<D, MT>::kMax);  // [G * D]
   float* sTalk = reinterpret_cast<float*>(sKnew + GD);           // [H][H]
   uint64_t* full = reinterpret_cast<uint64_t*>(sTalk + ((H * H + 1) & ~1));  // [4]
-  int* s_last = reinterpret_cast<int*>(full + 4);
+  uint64_t* empty = full + 4;                                    // [4]
+  int* s_last = reinterpret_cast<int*>(empty + 4);
   const int split = blockIdx.x, b = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   // Lengths, tables and the keys of earlier tokens were complete before the kernel ahead of this one started.
@@ -507,36 +542,51 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
   const bool newest = split == a.splits - 1;
   const int* table = p.block_tables + (size_t)b * p.max_blocks;
 
-  // Warp 0 issues the loads: lane -> page (lane & 3), which it looks up one tile ahead.
-  int page = 0;
-  auto fetch_page = [&](int t) {
-    if (t >= t_end) return;
-    int bi = (jb + t * kDT) / 16 + (lane & 3);
-    bi = bi > pos / 16 ? pos / 16 : bi;       // past the end: any valid page, masked
-    page = table[bi];
-    if (page < 0 || page >= p.num_cache_blocks) {
-      report_status(p.status, kStatusBadIndex);
-      page = 0;
+  if (tid == 0) {
+    for (int i = 0; i < 4; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], MW * 8);
     }
-  };
-  auto load_tile = [&](int t, int stage) {    // warp 0
-    if (lane == 0) mbar_expect_tx(&full[stage], stage_bytes);
-    __syncwarp();
-    for (int i = lane >> 2; i < G * kPl; i += 8) {
-      const int m = i / kPl, pl = i % kPl;
-      tma_load_2d(sKV + stage * stage_bytes + (i * kDT + (lane & 3) * 16) * 128, &tmK, &full[stage], pl * 64, (page * G + m) * 16);
+    fence_mbar_init();
+  }
+  __syncthreads();
+  if (warp == MW * 8) {
+    // ---- the loading warp: lane -> page (lane & 3) of a tile, looked up one tile ahead ----
+    int stage = 0;
+    uint32_t phase = 1;
+    auto page_of = [&](int t) {
+      const int bi = (jb + t * kDT) / 16 + (lane & 3);
+      return table[bi > pos / 16 ? pos / 16 : bi];  // past the end: any valid page, masked
+    };
+    int next = t_begin < t_end ? page_of(t_begin) : 0;
+    for (int t = t_begin; t < t_end; ++t) {
+      int page = next;
+      if (t + 1 < t_end) next = page_of(t + 1);
+      if (page < 0 || page >= p.num_cache_blocks) {
+        report_status(p.status, kStatusBadIndex);
+        page = 0;
+      }
+      int good = 1;
+      if (lane == 0) {
+        if (!mbar_wait(&empty[stage], phase)) {
+          report_status(p.status, kStatusWaitEmptyTimeout);
+          good = 0;
+        } else {
+          mbar_expect_tx(&full[stage], stage_bytes);
+        }
+      }
+      good = __shfl_sync(0xffffffffu, good, 0);
+      if (!good) break;
+      uint8_t* dst = sKV + stage * stage_bytes + (lane & 3) * (16 * 128);
+      for (int i = lane >> 2; i < G * kPl; i += 8)
+        tma_load_2d(dst + i * (kDT * 128), &tmK, &full[stage], (i % kPl) * 64, (page * G + i / kPl) * 16);
+      if (++stage == n_stages) {
+        stage = 0;
+        phase ^= 1;
+      }
     }
-    fetch_page(t + 1);
-  };
-  if (warp == 0) {
-    if (lane == 0) {
-      for (int i = 0; i < 4; ++i) mbar_init(&full[i], 1);
-      fence_mbar_init();
-    }
-    __syncwarp();
-    fetch_page(t_begin);
-    for (int i = 0; i < n_stages - 1; ++i)
-      if (t_begin + i < t_end) load_tile(t_begin + i, i);
+    pdl_wait();
+    return;
   }
   if (p.talk != nullptr)
     for (int i = tid; i < H * H; i += kDThreads) sTalk[i] = ldf(reinterpret_cast<const bf16*>(p.talk) + i);
@@ -570,12 +620,13 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
 
   const float qs = p.qscale[pos < p.qscale_len ? pos : p.qscale_len - 1];
   const int npw = (GD / 8 + 7) / 8;              // 8-wide value-column tiles per warp
-  const int nt0 = warp * npw;
+  const int cw = warp & 7, mt0 = (warp >> 3) * MTW;  // warp within its group, first row tile
+  const int nt0 = cw * npw;
   const int r0 = lane >> 2, cq = (lane & 3) * 2;
   // fragment addresses that do not change from tile to tile (inside a stage)
-  const uint32_t k_off = sw_off(warp * 8 + (lane & 7), lane >> 3);                       // keys: chunks 0-3; chunks 4-7 at ^ 64
-  const uint32_t q_off = smem_u32(sQ) + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, lane >> 4);  // queries: k-step s at ^ (s * 32)
-  const uint32_t p_off = smem_u32(sP) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + (lane >> 4) * 8) * 2;
+  const uint32_t k_off = sw_off(cw * 8 + (lane & 7), lane >> 3);                       // keys: chunks 0-3; chunks 4-7 at ^ 64
+  const uint32_t q_off = smem_u32(sQ) + mt0 * kPl * 2048 + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, lane >> 4);  // queries: k-step s at ^ (s * 32)
+  const uint32_t p_off = smem_u32(sP) + ((mt0 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + (lane >> 4) * 8) * 2;
   constexpr int kPairs = NTW > 1 ? NTW / 2 : 1;
   uint32_t v_off[kPairs];                        // value columns: two neighbouring 8-wide tiles per ldmatrix
 #pragma unroll
@@ -586,21 +637,28 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
     const int m = nn / (D / 8), ch = nn % (D / 8);
     v_off[i] = (m * kPl + (ch >> 3)) * (kDT * 128) + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, ch & 7);
   }
-  const float* bias_row[MT][2];                  // rows past the last head read the last head's biases; they are never stored
-  int key_head[MT][2];
+  const float* bias_row[MTW][2];                  // rows past the last head read the last head's biases; they are never stored
+  int key_head[MTW][2];
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
+  for (int mt = 0; mt < MTW; ++mt)
 #pragma unroll
     for (int q = 0; q < 2; ++q) {
-      int h = mt * 16 + r0 + q * 8;
+      int h = (mt0 + mt) * 16 + r0 + q * 8;
       h = h < H ? h : H - 1;
       bias_row[mt][q] = p.bias + (size_t)h * p.bias_len;
       key_head[mt][q] = h / grp;
     }
-  float acc[MT][NTW][4];
-  float mrow[MT][2], lrow[MT][2];
+  int m_lo[MTW], m_hi[MTW];                      // key heads that a row tile reads
 #pragma unroll
-  for (int t = 0; t < MT; ++t) {
+  for (int mt = 0; mt < MTW; ++mt) {
+    const int h0 = (mt0 + mt) * 16, h1 = (h0 + 16 < H ? h0 + 16 : H) - 1;
+    m_lo[mt] = h0 / grp;
+    m_hi[mt] = h0 < H ? h1 / grp : -1;
+  }
+  float acc[MTW][NTW][4];
+  float mrow[MTW][2], lrow[MTW][2];
+#pragma unroll
+  for (int t = 0; t < MTW; ++t) {
 #pragma unroll
     for (int i = 0; i < NTW; ++i)
 #pragma unroll
@@ -608,22 +666,23 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
     mrow[t][0] = mrow[t][1] = -INFINITY;
     lrow[t][0] = lrow[t][1] = 0.f;
   }
-  __syncthreads();  // barriers, q, the new key and the mixing matrix are in shared memory
+  compute_bar<kDThreads>();  // q, the new key and the mixing matrix are in shared memory
+  uint32_t qf[kQReg ? D / 16 : 1][4];
+  if constexpr (kQReg) {
+#pragma unroll
+    for (int k = 0; k < D / 16; ++k) ldsm4(qf[k], (q_off + (k >> 2) * 2048) ^ ((k & 3) * 32));
+  }
   int stage = 0;
   uint32_t phase = 0;
   bool ok = true;
   for (int t = t_begin; t < t_end; ++t) {
-    if (n_stages == 1) {
-      __syncthreads();
-      if (warp == 0) load_tile(t, 0);
-    }
     const int j0 = jb + t * kDT;
     const bool inside = j0 >= lo && j0 + kDT - 1 <= pos && pos - j0 < p.bias_len;
-    float bv[MT][4];                             // distance biases, on their way while the tile arrives
+    float bv[MTW][4];                             // distance biases, on their way while the tile arrives
     {
-      const int d = pos - (j0 + warp * 8 + cq);
+      const int d = pos - (j0 + cw * 8 + cq);
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
+      for (int mt = 0; mt < MTW; ++mt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int de = d - (e & 1);
@@ -643,26 +702,31 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
         const int m = i / (D / 8), ch = i % (D / 8);
         *reinterpret_cast<uint4*>(kt + (m * kPl + (ch >> 3)) * (kDT * 128) + sw_off(key, ch & 7)) = *reinterpret_cast<const uint4*>(sKnew + i * 8);
       }
-      __syncthreads();
+      compute_bar<kDThreads>();
     }
     // ---- scores of keys [8 warp, 8 warp + 8) for all heads ----
-    float s[MT][4];
+    float s[MTW][4];
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
+    for (int mt = 0; mt < MTW; ++mt) {
       s[mt][0] = s[mt][1] = s[mt][2] = s[mt][3] = 0.f;
-      if (mt * 16 < H) {
-        const int m_lo = mt * 16 / grp, m_hi = ((mt * 16 + 16 < H ? mt * 16 + 16 : H) - 1) / grp;
-        for (int m = m_lo; m <= m_hi; ++m) {
-          float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int m = m_lo[mt]; m <= m_hi[mt]; ++m) {
+        float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-          for (int pl = 0; pl < kPl; ++pl) {
-            const uint32_t ka = kts + (m * kPl + pl) * (kDT * 128) + k_off;
+        for (int pl = 0; pl < kPl; ++pl) {
+          const uint32_t ka = kts + (m * kPl + pl) * (kDT * 128) + k_off;
+          uint32_t k0[4], k1[4];
+          ldsm4(k0, ka);
+          ldsm4(k1, ka ^ 64);
+          if constexpr (kQReg) {
+            mma_16816(c0, qf[pl * 4][0], qf[pl * 4][1], qf[pl * 4][2], qf[pl * 4][3], k0[0], k0[1]);
+            mma_16816(c1, qf[pl * 4 + 1][0], qf[pl * 4 + 1][1], qf[pl * 4 + 1][2], qf[pl * 4 + 1][3], k0[2], k0[3]);
+            mma_16816(c0, qf[pl * 4 + 2][0], qf[pl * 4 + 2][1], qf[pl * 4 + 2][2], qf[pl * 4 + 2][3], k1[0], k1[1]);
+            mma_16816(c1, qf[pl * 4 + 3][0], qf[pl * 4 + 3][1], qf[pl * 4 + 3][2], qf[pl * 4 + 3][3], k1[2], k1[3]);
+          } else {
             const uint32_t qa = q_off + (mt * kPl + pl) * 2048;
-            uint32_t k0[4], k1[4], q0[4], q1[4], q2[4], q3[4];
-            ldsm4(k0, ka);
+            uint32_t q0[4], q1[4], q2[4], q3[4];
             ldsm4(q0, qa);
             ldsm4(q1, qa ^ 32);
-            ldsm4(k1, ka ^ 64);
             ldsm4(q2, qa ^ 64);
             ldsm4(q3, qa ^ 96);
             mma_16816(c0, q0[0], q0[1], q0[2], q0[3], k0[0], k0[1]);
@@ -670,14 +734,14 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
             mma_16816(c0, q2[0], q2[1], q2[2], q2[3], k1[0], k1[1]);
             mma_16816(c1, q3[0], q3[1], q3[2], q3[3], k1[2], k1[3]);
           }
-          if (key_head[mt][0] == m) {
-            s[mt][0] = c0[0] + c1[0];
-            s[mt][1] = c0[1] + c1[1];
-          }
-          if (key_head[mt][1] == m) {
-            s[mt][2] = c0[2] + c1[2];
-            s[mt][3] = c0[3] + c1[3];
-          }
+        }
+        if (key_head[mt][0] == m) {
+          s[mt][0] = c0[0] + c1[0];
+          s[mt][1] = c0[1] + c1[1];
+        }
+        if (key_head[mt][1] == m) {
+          s[mt][2] = c0[2] + c1[2];
+          s[mt][3] = c0[3] + c1[3];
         }
       }
 #pragma unroll
@@ -687,21 +751,17 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
         float mx = fmaxf(s[mt][2 * q], s[mt][2 * q + 1]);
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        if ((lane & 3) == 0) sMax[(mt * 16 + r0 + q * 8) * 8 + warp] = mx;
+        if ((lane & 3) == 0) sMax[((mt0 + mt) * 16 + r0 + q * 8) * 8 + cw] = mx;
       }
     }
-    __syncthreads();  // maxima; everybody is done with the products of the tile before, whose stage is loaded next
-    if (n_stages > 1 && warp == 0) {
-      const int nxt = t + n_stages - 1;
-      if (nxt < t_end) load_tile(nxt, stage == 0 ? n_stages - 1 : stage - 1);
-    }
+    compute_bar<kDThreads>();
     // ---- weights ----
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
+    for (int mt = 0; mt < MTW; ++mt) {
       float al[2];
 #pragma unroll
       for (int q = 0; q < 2; ++q) {
-        const int row = mt * 16 + r0 + q * 8;
+        const int row = (mt0 + mt) * 16 + r0 + q * 8;
         const float4 x = *reinterpret_cast<const float4*>(sMax + row * 8), y = *reinterpret_cast<const float4*>(sMax + row * 8 + 4);
         const float mx = fmaxf(fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w)), fmaxf(fmaxf(y.x, y.y), fmaxf(y.z, y.w)));
         const float mn = fmaxf(mrow[mt][q], mx);
@@ -710,7 +770,7 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
         const float base = mn == -INFINITY ? 0.f : mn;
         const float p0 = exp2f(s[mt][2 * q] - base), p1 = exp2f(s[mt][2 * q + 1] - base);
         lrow[mt][q] = lrow[mt][q] * al[q] + p0 + p1;
-        *reinterpret_cast<uint32_t*>(sP + (row * kPPitch + warp * 8 + cq) * 2) = pack_bf16x2(p0, p1);
+        *reinterpret_cast<uint32_t*>(sP + (row * kPPitch + cw * 8 + cq) * 2) = pack_bf16x2(p0, p1);
       }
 #pragma unroll
       for (int i = 0; i < NTW; ++i) {
@@ -720,50 +780,52 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
         acc[mt][i][3] *= al[1];
       }
     }
-    __syncthreads();
-    // ---- products: all heads x this warp's value columns ----
+    compute_bar<kDThreads>();
+    // ---- products: this warp's heads x its value columns ----
 #pragma unroll
     for (int kk = 0; kk < kDT / 16; ++kk) {
-      uint32_t pf[MT][4];
+      uint32_t pf[MTW][4];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) ldsm4(pf[mt], p_off + (mt * 16 * kPPitch + kk * 16) * 2);
+      for (int mt = 0; mt < MTW; ++mt) ldsm4(pf[mt], p_off + (mt * 16 * kPPitch + kk * 16) * 2);
 #pragma unroll
       for (int i = 0; i < kPairs; ++i) {
         if (2 * i < npw) {   // columns past the end repeat the last ones; they are never stored
           uint32_t vf[4];
           ldsm4_t(vf, kts + v_off[i] + kk * 2048);
 #pragma unroll
-          for (int mt = 0; mt < MT; ++mt) {
+          for (int mt = 0; mt < MTW; ++mt) {
             mma_16816(acc[mt][2 * i], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[0], vf[1]);
             if constexpr (NTW > 1) mma_16816(acc[mt][2 * i + 1], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[2], vf[3]);
           }
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[stage]);
     if (++stage == n_stages) {
       stage = 0;
       phase ^= 1;
     }
   }
-  __syncthreads();
+  compute_bar<kDThreads>();
   // ---- row sums over the warps ----
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
+  for (int mt = 0; mt < MTW; ++mt)
 #pragma unroll
     for (int q = 0; q < 2; ++q) {
       float l = lrow[mt][q];
       l += __shfl_xor_sync(0xffffffffu, l, 1);
       l += __shfl_xor_sync(0xffffffffu, l, 2);
-      if ((lane & 3) == 0) sMax[(mt * 16 + r0 + q * 8) * 8 + warp] = l;
+      if ((lane & 3) == 0) sMax[((mt0 + mt) * 16 + r0 + q * 8) * 8 + cw] = l;
     }
-  __syncthreads();
+  compute_bar<kDThreads>();
   float* prod = reinterpret_cast<float*>(sKV);   // [H][G * D]
   const size_t part = ((size_t)b * a.splits + split) * H;
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
+  for (int mt = 0; mt < MTW; ++mt)
 #pragma unroll
     for (int q = 0; q < 2; ++q) {
-      const int h = mt * 16 + r0 + q * 8;
+      const int h = (mt0 + mt) * 16 + r0 + q * 8;
       if (h >= H) continue;
       float l = 0.f;
 #pragma unroll
@@ -774,18 +836,18 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
       for (int i = 0; i < NTW; ++i)
         if (i < npw && nt0 + i < GD / 8)
           *reinterpret_cast<float2*>(dst + (nt0 + i) * 8 + cq) = make_float2(acc[mt][i][2 * q] * inv, acc[mt][i][2 * q + 1] * inv);
-      if (a.splits > 1 && warp == 0 && (lane & 3) == 0)
+      if (a.splits > 1 && cw == 0 && (lane & 3) == 0)
         *reinterpret_cast<float2*>(a.part_ml + (part + h) * 2) = make_float2(mrow[mt][q], l);
     }
   if (a.splits > 1) {
     __threadfence();
-    __syncthreads();
+    compute_bar<kDThreads>();
     if (tid == 0) {
       const int ticket = atomicAdd(a.tickets + b, 1);
       *s_last = ticket == a.splits - 1;
       if (*s_last) a.tickets[b] = 0;
     }
-    __syncthreads();
+    compute_bar<kDThreads>();
     if (!*s_last) return;
     __threadfence();
     float* wgt = sMax;  // [H][splits] merge weights, splits <= 8
@@ -801,7 +863,7 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
       }
       for (int s = 0; s < a.splits; ++s) wgt[h * 8 + s] *= L > 0.f ? 1.f / L : 0.f;
     }
-    __syncthreads();
+    compute_bar<kDThreads>();
     for (int i = tid; i < H * GD / 4; i += kDThreads) {
       const int h = i / (GD / 4);
       float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -816,7 +878,7 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
       reinterpret_cast<float4*>(prod)[i] = o;
     }
   }
-  __syncthreads();
+  compute_bar<kDThreads>();
   // ---- mix across heads, gate, store ----
   const bf16* gate = p.gate != nullptr ? reinterpret_cast<const bf16*>(p.gate) + (size_t)b * p.ldg : nullptr;
   bf16* out = reinterpret_cast<bf16*>(p.out) + (size_t)b * p.ldo;
@@ -844,51 +906,52 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
 }
 
 struct DecPlan {
-  int mt, ntw, stages;
+  int mw, mtw, ntw, stages;
   size_t smem;
 };
-// picks the template and the number of stages; mt = 0: not served
+// picks the template and the number of stages; mw = 0: not served
 DecPlan plan_decode_kernel(int H, int G, int D) {
-  DecPlan d{0, 0, 0, 0};
+  DecPlan d{0, 0, 0, 0, 0};
   if ((D != 64 && D != 128) || H > 64 || H % G != 0) return d;
-  const int mt = H <= 16 ? 1 : (H <= 32 ? 2 : 4);
+  const int mw = H <= 16 ? 1 : 2, mtw = H <= 32 ? 1 : 2, mt = mw * mtw;
   const int npw = (G * D / 8 + 7) / 8;
-  int ntw = 1;
+  int ntw = 2;
   while (ntw < npw) ntw *= 2;
-  if (ntw > 16 || mt * ntw > 32) return d;
+  if (ntw > 16 || mtw * ntw > 16) return d;
   const size_t stage = (size_t)kDT * G * D * 2;
-  const size_t fixed = (size_t)mt * 16 * D * 2 + (size_t)mt * 16 * kPPitch * 2 + (size_t)mt * 16 * 32 + (size_t)G * D * 2 + (size_t)(H * H + 1) * 4 + 64;
+  const size_t fixed = (size_t)mt * 16 * D * 2 + (size_t)mt * 16 * kPPitch * 2 + (size_t)mt * 16 * 32 + (size_t)G * D * 2 + (size_t)(H * H + 1) * 4 + 96;
   const size_t prod = (size_t)H * G * D * 4;
+  const size_t budget = (size_t)(mw == 1 && ntw <= 4 ? 112 : 224) * 1024;  // two CTAs per SM or one
   int st = 4;
-  while (st > 1 && st * stage + fixed > (size_t)112 * 1024) --st;
-  if (st < 2 || mt * ntw > 8) {  // one CTA per SM: as many stages as fit
-    st = 4;
-    while (st > 1 && st * stage + fixed > (size_t)224 * 1024) --st;
-  }
-  if (st * stage < prod) return d;
-  if (st * stage + fixed > (size_t)224 * 1024) return d;
-  d.mt = mt; d.ntw = ntw; d.stages = st; d.smem = st * stage + fixed;
+  while (st > 1 && st * stage + fixed > budget) --st;
+  if (st * stage < prod || st * stage + fixed > budget) return d;
+  d.mw = mw; d.mtw = mtw; d.ntw = ntw; d.stages = st; d.smem = st * stage + fixed;
   return d;
 }
 
-template <int D, int MT, int NTW>
+template <int D, int MW, int MTW, int NTW>
 void launch_decode_t(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) {
-  auto kernel = talk_decode_kernel<D, MT, NTW>;
+  auto kernel = talk_decode_kernel<D, MW, MTW, NTW>;
   AGRPO_SET_MAX_DYN_SMEM(kernel, 226 * 1024, "talk_decode smem attr");
   AGRPO_PREFER_SMEM(kernel);
   const CUtensorMap tk = make_tmap_2d(a.k_cache, D, (uint64_t)a.at.num_cache_blocks * a.at.G * 16, D, 64, 16);
-  launch_kernel(kernel, dim3(a.splits, a.at.T), dim3(kDThreads), d.smem, s, "talk_decode", tk, a, d.stages);
+  launch_kernel(kernel, dim3(a.splits, a.at.T), dim3(MW * 256 + 32), d.smem, s, "talk_decode", tk, a, d.stages);
 }
-template <int D, int MT>
+template <int D, int MW, int MTW>
 void launch_decode_n(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) {
-  if (d.ntw == 1) return launch_decode_t<D, MT, 1>(a, d, s);
-  if (d.ntw == 2) return launch_decode_t<D, MT, 2>(a, d, s);
-  if (d.ntw == 4) return launch_decode_t<D, MT, 4>(a, d, s);
-  if (d.ntw == 8) return launch_decode_t<D, MT, 8>(a, d, s);
-  if constexpr (MT <= 2) {
-    if (d.ntw == 16) return launch_decode_t<D, MT, 16>(a, d, s);
+  if (d.ntw == 2) return launch_decode_t<D, MW, MTW, 2>(a, d, s);
+  if (d.ntw == 4) return launch_decode_t<D, MW, MTW, 4>(a, d, s);
+  if (d.ntw == 8) return launch_decode_t<D, MW, MTW, 8>(a, d, s);
+  if constexpr (MTW == 1) {
+    if (d.ntw == 16) return launch_decode_t<D, MW, MTW, 16>(a, d, s);
   }
   throw std::runtime_error("talk_decode: shape not served");
+}
+template <int D>
+void launch_decode_d(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) {
+  if (d.mw == 1) launch_decode_n<D, 1, 1>(a, d, s);
+  else if (d.mtw == 1) launch_decode_n<D, 2, 1>(a, d, s);
+  else launch_decode_n<D, 2, 2>(a, d, s);
 }
 
 }  // namespace
@@ -927,21 +990,14 @@ bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_t
   return true;
 }
 
-bool talk_decode_supported(int H, int G, int D) { return plan_decode_kernel(H, G, D).mt > 0; }
+bool talk_decode_supported(int H, int G, int D) { return plan_decode_kernel(H, G, D).mw > 0; }
 
 void launch_talk_attn_decode(const TalkDecodeArgs& a, cudaStream_t s) {
   const DecPlan d = plan_decode_kernel(a.at.H, a.at.G, a.at.D);
-  if (d.mt == 0 || a.at.block_size != 16 || a.splits < 1 || a.splits > 8) throw std::runtime_error("talk_decode: shape not served");
+  if (d.mw == 0 || a.at.block_size != 16 || a.splits < 1 || a.splits > 8) throw std::runtime_error("talk_decode: shape not served");
   if (a.at.T == 0) return;
-  if (a.at.D == 128) {
-    if (d.mt == 1) launch_decode_n<128, 1>(a, d, s);
-    else if (d.mt == 2) launch_decode_n<128, 2>(a, d, s);
-    else launch_decode_n<128, 4>(a, d, s);
-  } else {
-    if (d.mt == 1) launch_decode_n<64, 1>(a, d, s);
-    else if (d.mt == 2) launch_decode_n<64, 2>(a, d, s);
-    else launch_decode_n<64, 4>(a, d, s);
-  }
+  if (a.at.D == 128) launch_decode_d<128>(a, d, s);
+  else launch_decode_d<64>(a, d, s);
 }
 
 }  // namespace agrpo
