@@ -804,6 +804,11 @@ class RolloutEngine:
         self.h_eos_at[slot] = -1
         del self.slot_info[slot]
 
+    # ------------------------------------------------------------------ step-wise driving
+    def open_sequence(self) -> int:
+        """Starts a sequence whose tokens the caller supplies (``extend``, ``close_sequence``)."""
+        raise NotImplementedError(f"{type(self).__name__} has no step-wise interface")
+
     # ------------------------------------------------------------------ stepping
     def step(self) -> List[FinishedSequence]:
         pc = time.perf_counter
