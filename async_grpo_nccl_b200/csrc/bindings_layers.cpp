@@ -139,17 +139,22 @@ void window_attn(const Tensor& q, const Tensor& k_cache, const OptTensor& rows, 
 }
 
 // Tensor-core form for prompts; false (nothing launched) when the shape is not served.
-bool talk_attn_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& tiles, const Tensor& block_tables, const Tensor& bias,
+bool talk_attn_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& tiles, const Tensor& pages, Tensor& keys, const Tensor& block_tables, const Tensor& bias,
                        const Tensor& qscale, const OptTensor& talk, const OptTensor& gate, int64_t window, Tensor& acc, Tensor& out,
                        const OptTensor& status) {
   if (k_cache.scalar_type() != torch::kBFloat16 || k_cache.size(2) != 16) return false;
   check_i32(tiles, "tiles");
   TORCH_CHECK(tiles.dim() == 2 && tiles.size(1) == 4 && tiles.is_contiguous() && aligned16(tiles), "talk_attn_prefill: tiles [n, 4]");
+  check_i32(pages, "pages"); same_type(keys, false, "keys");
+  TORCH_CHECK(pages.dim() == 2 && pages.size(1) == 2 && pages.is_contiguous() && (reinterpret_cast<uintptr_t>(pages.data_ptr()) & 7) == 0, "talk_attn_prefill: pages [n, 2]");
+  TORCH_CHECK(keys.is_contiguous() && aligned16(keys) && keys.numel() >= pages.size(0) * 16 * k_cache.size(1) * k_cache.size(3),
+              "talk_attn_prefill: keys [16 pages, G * D]");
   const agrpo::WindowAttnArgs a = attn_args(q, k_cache, OptTensor(), OptTensor(), block_tables, bias, qscale, talk, gate, window, out, status);
   same_type(acc, false, "acc");
   TORCH_CHECK(acc.is_contiguous() && acc.numel() >= (int64_t)a.T * a.H * a.G * a.D && aligned16(acc), "talk_attn_prefill: acc [T, H, G, D]");
   const c10::cuda::CUDAGuard guard(k_cache.device());
-  return agrpo::launch_talk_attn_prefill(a, tiles.data_ptr<int>(), (int)tiles.size(0), acc.data_ptr(), cur_stream());
+  return agrpo::launch_talk_attn_prefill(a, tiles.data_ptr<int>(), (int)tiles.size(0), pages.data_ptr<int>(), (int)pages.size(0),
+                                         keys.data_ptr(), acc.data_ptr(), cur_stream());
 }
 
 // Decode step of a mixer after its fused projection u = [q | k | gate]: convolution, attention, mixing, gate, state update.
@@ -238,7 +243,7 @@ void bind_layer_ops(pybind11::module_& m) {
         py::arg("block_tables"), py::arg("q_out"), py::arg("k_cache"), py::arg("status"), NoGil());
   m.def("window_attn", &window_attn, py::arg("q"), py::arg("k_cache"), py::arg("rows"), py::arg("seq_lens"), py::arg("block_tables"),
         py::arg("bias"), py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("out"), py::arg("status"), NoGil());
-  m.def("talk_attn_prefill", &talk_attn_prefill, py::arg("q"), py::arg("k_cache"), py::arg("tiles"), py::arg("block_tables"), py::arg("bias"),
+  m.def("talk_attn_prefill", &talk_attn_prefill, py::arg("q"), py::arg("k_cache"), py::arg("tiles"), py::arg("pages"), py::arg("keys"), py::arg("block_tables"), py::arg("bias"),
         py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("acc"), py::arg("out"), py::arg("status"), NoGil());
   m.def("talk_attn_decode", &talk_attn_decode, py::arg("u"), py::arg("conv_w"), py::arg("ring"), py::arg("k_cache"), py::arg("seq_lens"),
         py::arg("block_tables"), py::arg("bias"), py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("out"),

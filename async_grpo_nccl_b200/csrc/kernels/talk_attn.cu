@@ -26,8 +26,9 @@ typedef __nv_bfloat16 bf16;
 
 // ================================================================================================
 // Prompts: one CTA = 128 query rows of one head g, value heads [m0, m0 + mc). S (two buffers, so that the scores of tile
-// j + 1 are computed while the softmax of tile j runs) and the mc accumulators fill tensor memory. Warp 0 loads key tiles
-// page by page, warp 1 issues MMAs, warps 2-17 run the softmax in two groups that take alternating tiles (one group's loads
+// j + 1 are computed while the softmax of tile j runs) and the mc accumulators fill tensor memory. The keys that a step can
+// see are first gathered from their pages into one matrix (a TMA request per 16-token page would be the bottleneck). Warp 0
+// loads key tiles into a ring of slots, one slot per key head of a tile, warp 1 issues MMAs, warps 2-17 run the softmax in two groups that take alternating tiles (one group's loads
 // and maxima overlap the other's exponentials); in a group two threads share a query row, 64 keys each. The reference maximum
 // of a row is handed from tile to tile through shared memory, so that all weights of a row are on one scale. The key tile of a
 // head serves as K-major operand of Q K^T and as MN-major operand of P V.
@@ -37,11 +38,10 @@ constexpr int kPN = 128;
 constexpr int kPKeys = 64;                            // keys per thread and tile
 constexpr int kPThreads = 64 + 4 * kPM;
 constexpr int kRingBytes = 192 * 1024;
+constexpr int kMaxSlots = 12;
 
 struct TalkPrefillParams {
-  const int4* tiles;       // {first row, rows, position of the first row, slot}
-  const int* block_tables;
-  int max_blocks;
+  const int4* tiles;       // {first row, rows, position of the first row, row of position 0 among the gathered keys}
   const float* bias;
   int bias_len;
   const float* qscale;
@@ -49,7 +49,6 @@ struct TalkPrefillParams {
   int window;
   bf16* acc;               // [T, H, G, D], normalised products
   int H, G, group, mc;     // mc = value heads per CTA
-  int num_cache_blocks;
   int* status;
 };
 
@@ -61,6 +60,7 @@ __global__ void __launch_bounds__(kPThreads, 1)
 talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const TalkPrefillParams p) {
   constexpr int kTile = kPM * D * 2;
   constexpr int kChunks = D / 64;
+  constexpr int kSlots = kRingBytes / kTile;
   constexpr uint32_t kIdescS = umma_idesc_bf16(kPM, kPN, 0, 0);
   constexpr uint32_t kIdescO = umma_idesc_bf16(kPM, D, 0, 1);
   extern __shared__ __align__(1024) uint8_t tp_smem[];
@@ -71,23 +71,25 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   bf16* sref = reinterpret_cast<bf16*>(smax + 512);          // [2][128] reference maximum after the latest even / odd tile
   uint64_t* bars = reinterpret_cast<uint64_t*>(sref + 256);
   uint64_t* q_full = bars;
-  uint64_t* k_full = bars + 1;      // [3]
-  uint64_t* k_empty = bars + 4;     // [3]
-  uint64_t* s_full = bars + 7;      // [2]
-  uint64_t* p_ready = bars + 9;     // [2]
-  uint64_t* ref_set = bars + 11;    // [2]
-  uint64_t* o_done = bars + 13;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
+  uint64_t* s_full = bars + 1;      // [2]
+  uint64_t* p_ready = bars + 3;     // [2]
+  uint64_t* ref_set = bars + 5;     // [2]
+  // [2], even and odd tiles: a thread may look for tile j's products while those of tile j - 1 are still running, which one
+  // barrier's parity could not tell from finished
+  uint64_t* o_done = bars + 7;
+  uint64_t* k_full = bars + 9;      // [kSlots]
+  uint64_t* k_empty = k_full + kMaxSlots;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_empty + kMaxSlots);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.x;
   const int kv_own = head / p.group;
   const int m0 = blockIdx.y * p.mc;
   const int mc = p.G - m0 < p.mc ? p.G - m0 : p.mc;
-  const int own_in = kv_own >= m0 && kv_own < m0 + mc ? kv_own - m0 : mc;  // place of the head's own keys in a stage
-  const int n_t = own_in == mc ? mc + 1 : mc;
-  const int stage_bytes = n_t * kTile;
-  const int n_stages = kRingBytes / stage_bytes < 3 ? kRingBytes / stage_bytes : 3;
+  // a tile takes n_t slots: [own keys, when they are not among the value heads], value heads m0 ...
+  const int extra = kv_own >= m0 && kv_own < m0 + mc ? 0 : 1;
+  const int own_slot = extra ? 0 : kv_own - m0;
+  const int n_t = mc + extra;
   const int4 tile = p.tiles[blockIdx.z];
   const int pos0 = tile.z, n_rows = tile.y;
   const int key_end = pos0 + n_rows;
@@ -97,7 +99,7 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int i = 0; i < 3; ++i) {
+    for (int i = 0; i < kSlots; ++i) {
       mbar_init(&k_full[i], 1);
       mbar_init(&k_empty[i], 1);
     }
@@ -107,7 +109,8 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       mbar_init(&p_ready[i], 8);
       mbar_init(&ref_set[i], 8);
     }
-    mbar_init(o_done, 1);
+    mbar_init(&o_done[0], 1);
+    mbar_init(&o_done[1], 1);
     fence_mbar_init();
   }
   if (warp == 1) {
@@ -123,106 +126,92 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   const uint32_t tmem_O = tmem + 256;
 
   if (warp == 0) {
-    // ---------------- loads: lane b < 8 brings the b-th 16-token page of every tile ----------------
-    if (lane == 0) {
+    // ---------------- loads ----------------
+    if (elect_one()) {
       mbar_expect_tx(q_full, kTile);
 #pragma unroll
       for (int c = 0; c < kChunks; ++c) tma_load_2d(sQ + c * (kPM * 128), &tmQ, q_full, head * D + c * 64, tile.x);
-    }
-    const int* table = p.block_tables + (size_t)tile.w * p.max_blocks;
-    const int last_block = (key_end - 1) / 16;
-    int stage = 0;
-    uint32_t phase = 0;
-    for (int j = 0; j < n_kv; ++j) {
-      int phys = 0;
-      if (lane < 8) {
-        int bi = (j0 + j * kPN) / 16 + lane;
-        bi = bi > last_block ? last_block : bi;  // past the end: any valid page, masked below
-        phys = table[bi];
-        if (phys < 0 || phys >= p.num_cache_blocks) {
-          report_status(p.status, kStatusBadIndex);
-          phys = 0;
-        }
-      }
-      int good = 1;
-      if (lane == 0) {
-        if (j >= n_stages && !mbar_wait(&k_empty[stage], phase ^ 1)) {
-          report_status(p.status, kStatusWaitEmptyTimeout);
-          good = 0;
-        }
-        if (good) mbar_expect_tx(&k_full[stage], stage_bytes);
-      }
-      good = __shfl_sync(0xffffffffu, good, 0);
-      if (!good) break;
-      if (lane < 8) {
-        uint8_t* dst = sK + stage * stage_bytes + lane * (16 * 128);
-        for (int i = 0; i < n_t; ++i) {
-          const int m = i < mc ? m0 + i : kv_own;
+      int slot = 0;
+      uint32_t phase = 1;
+      bool ok = true;
+      for (int j = 0; j < n_kv && ok; ++j) {
+        const int row = tile.w + j0 + j * kPN;   // rows past the gathered keys read as zero, other segments' rows are masked
+        for (int k = 0; k < n_t; ++k) {
+          if (!mbar_wait(&k_empty[slot], phase)) {
+            report_status(p.status, kStatusWaitEmptyTimeout);
+            ok = false;
+            break;
+          }
+          const int m = extra ? (k == 0 ? kv_own : m0 + k - 1) : m0 + k;
+          mbar_expect_tx(&k_full[slot], kTile);
 #pragma unroll
-          for (int c = 0; c < kChunks; ++c)
-            tma_load_2d(dst + i * kTile + c * (kPN * 128), &tmK, &k_full[stage], c * 64, (phys * p.G + m) * 16);
+          for (int c = 0; c < kChunks; ++c) tma_load_2d(sK + slot * kTile + c * (kPN * 128), &tmK, &k_full[slot], m * D + c * 64, row);
+          if (++slot == kSlots) {
+            slot = 0;
+            phase ^= 1;
+          }
         }
-      }
-      if (++stage == n_stages) {
-        stage = 0;
-        phase ^= 1;
       }
     }
   } else if (warp == 1) {
     // ---------------- MMA issuer ----------------
     if (elect_one()) {
       const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK);
-      auto scores = [&](int j, int stage) {
-        const uint32_t kt = aK + stage * stage_bytes + own_in * kTile;
+      auto wait_slot = [&](int idx) { return mbar_wait(&k_full[idx % kSlots], (idx / kSlots) & 1); };
+      auto scores = [&](int j) {
+        const int slot = (j * n_t + own_slot) % kSlots;
+        const uint32_t kt = aK + slot * kTile;
 #pragma unroll
         for (int k = 0; k < D / 16; ++k) {
           const uint32_t off = (k / 4) * (kPM * 128) + (k % 4) * 32;
           tc_mma_f16(tmem + (j & 1) * 128, umma_smem_desc(aQ + off, 16, 1024), umma_smem_desc(kt + off, 16, 1024), kIdescS, k > 0 ? 1u : 0u);
         }
+        if (extra) tc_commit(&k_empty[slot]);   // these keys are not read as values
         tc_commit(&s_full[j & 1]);
       };
-      bool ok = mbar_wait(q_full, 0) && mbar_wait(&k_full[0], 0);
+      bool ok = mbar_wait(q_full, 0) && wait_slot(own_slot);
       if (ok) {
         tc_fence_after();
-        scores(0, 0);
+        scores(0);
       } else {
         report_status(p.status, kStatusWaitFullTimeout);
       }
-      int stage = 0, nstage = n_stages > 1 ? 1 : 0;
-      uint32_t nphase = n_stages > 1 ? 0 : 1;
       for (int j = 0; j < n_kv && ok; ++j) {
         if (j + 1 < n_kv) {
           // the buffer that the next scores go to holds the weights of tile j - 1 until their products are done
-          if (j >= 1 && !mbar_wait(o_done, (j - 1) & 1)) {
+          if (j >= 1 && !mbar_wait(&o_done[(j - 1) & 1], ((j - 1) >> 1) & 1)) {
             report_status(p.status, kStatusWaitTmemEmptyTimeout);
             break;
           }
-          if (!mbar_wait(&k_full[nstage], nphase)) {
+          if (!wait_slot((j + 1) * n_t + own_slot)) {
             report_status(p.status, kStatusWaitFullTimeout);
             break;
           }
           tc_fence_after();
-          scores(j + 1, nstage);
+          scores(j + 1);
         }
         if (!mbar_wait(&p_ready[j & 1], (j >> 1) & 1)) {
           report_status(p.status, kStatusWaitTmemFullTimeout);
           break;
         }
-        tc_fence_after();
-        for (int m = 0; m < mc; ++m) {
-          const uint32_t vt = aK + stage * stage_bytes + m * kTile;
+        for (int m = 0; m < mc && ok; ++m) {
+          const int idx = j * n_t + extra + m;
+          ok = wait_slot(idx);
+          tc_fence_after();
+          const uint32_t vt = aK + (idx % kSlots) * kTile;
+          if (ok) {
 #pragma unroll
-          for (int k = 0; k < kPN / 16; ++k)
-            tc_mma_f16_ts(tmem_O + m * D, tmem + (j & 1) * 128 + k * 8, umma_smem_desc(vt + k * 2048, kPN * 128, 1024), kIdescO,
-                          (j > 0 || k > 0) ? 1u : 0u);
+            for (int k = 0; k < kPN / 16; ++k)
+              tc_mma_f16_ts(tmem_O + m * D, tmem + (j & 1) * 128 + k * 8, umma_smem_desc(vt + k * 2048, kPN * 128, 1024), kIdescO,
+                            (j > 0 || k > 0) ? 1u : 0u);
+            tc_commit(&k_empty[idx % kSlots]);
+          }
         }
-        tc_commit(&k_empty[stage]);
-        tc_commit(o_done);
-        stage = nstage;
-        if (++nstage == n_stages) {
-          nstage = 0;
-          nphase ^= 1;
+        if (!ok) {
+          report_status(p.status, kStatusWaitFullTimeout);
+          break;
         }
+        tc_commit(&o_done[j & 1]);
       }
     }
   } else {
@@ -292,7 +281,7 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (lane == 0) mbar_arrive(&ref_set[group]);
       const float alpha = m_prev == -INFINITY ? 1.f : exp2f(m_prev - m_new);  // nothing is accumulated before the first visible key
       if (__any_sync(0xffffffffu, alpha != 1.f)) {
-        if (ok && !mbar_wait(o_done, (j - 1) & 1)) {
+        if (ok && !mbar_wait(&o_done[(j - 1) & 1], ((j - 1) >> 1) & 1)) {
           report_status(p.status, kStatusWaitTmemFullTimeout);
           ok = false;
         }
@@ -342,7 +331,7 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     smax[part * 128 + r] = l;
     softmax_all_bar();
     l = (smax[r] + smax[128 + r]) + (smax[256 + r] + smax[384 + r]);
-    if (ok && !mbar_wait(o_done, (n_kv - 1) & 1)) {
+    if (ok && !mbar_wait(&o_done[last], ((n_kv - 1) >> 1) & 1)) {
       report_status(p.status, kStatusWaitTmemFullTimeout);
       ok = false;
     }
@@ -373,6 +362,26 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (warp == 1) {
     tc_fence_after();
     tmem_dealloc(tmem, 512);
+  }
+}
+
+// Brings the pages that a step can see into one matrix [rows, G * D]: CTA = page, 16 rows of the matrix.
+__global__ void __launch_bounds__(128)
+gather_keys_kernel(const bf16* __restrict__ cache, const int2* __restrict__ pages, const int* __restrict__ block_tables, int max_blocks,
+                   bf16* __restrict__ keys, int G, int D, int num_cache_blocks, int* status) {
+  const int2 pg = pages[blockIdx.x];  // {slot, page of the sequence}
+  const int blk = block_tables[(size_t)pg.x * max_blocks + pg.y];
+  if (blk < 0 || blk >= num_cache_blocks) {
+    if (threadIdx.x == 0) report_status(status, kStatusBadIndex);
+    return;
+  }
+  const int per_row = D / 8;
+  const uint4* src = reinterpret_cast<const uint4*>(cache + (size_t)blk * G * 16 * D);
+  uint4* dst = reinterpret_cast<uint4*>(keys + (size_t)blockIdx.x * 16 * G * D);
+#pragma unroll 4
+  for (int i = threadIdx.x; i < G * 16 * per_row; i += 128) {
+    const int c = i % per_row, r = (i / per_row) % 16, m = i / (per_row * 16);
+    dst[(r * G + m) * per_row + c] = src[i];
   }
 }
 
@@ -445,7 +454,7 @@ talk_mix_gate_kernel(const bf16* __restrict__ acc, const bf16* __restrict__ talk
 
 template <int D>
 void launch_prefill_t(const CUtensorMap& tq, const CUtensorMap& tk, const TalkPrefillParams& p, int n_tiles, int chunks, cudaStream_t s) {
-  constexpr int smem = kPM * D * 2 + kRingBytes + 512 * 4 + 256 * 2 + 128;
+  constexpr int smem = kPM * D * 2 + kRingBytes + 512 * 4 + 256 * 2 + (9 + 2 * kMaxSlots) * 8 + 16;
   auto kernel = talk_prefill_kernel<D>;
   AGRPO_SET_MAX_DYN_SMEM(kernel, smem, "talk_prefill smem attr");
   launch_kernel(kernel, dim3(p.H, chunks, n_tiles), dim3(kPThreads), smem, s, "talk_prefill", tq, tk, p);
@@ -956,20 +965,22 @@ void launch_decode_d(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) 
 
 }  // namespace
 
-bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_tiles, void* acc, cudaStream_t s) {
+bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_tiles, const int* pages, int n_pages, void* keys, void* acc,
+                              cudaStream_t s) {
   if ((a.D != 64 && a.D != 128) || a.block_size != 16 || a.H % a.G != 0) return false;
   const int grp8 = (a.H / a.G + 7) & ~7;
   const size_t mix_smem = (size_t)a.G * a.H * grp8 * 4;
   if (mix_smem > 200 * 1024) return false;
   if (a.T == 0 || n_tiles == 0) return true;
+  gather_keys_kernel<<<n_pages, 128, 0, s>>>((const bf16*)a.k_cache, reinterpret_cast<const int2*>(pages), a.block_tables, a.max_blocks,
+                                             (bf16*)keys, a.G, a.D, a.num_cache_blocks, a.status);
+  check_cuda(cudaGetLastError(), "gather_keys");
   const int mc_max = 256 / a.D;
   const int chunks = (a.G + mc_max - 1) / mc_max;
   const CUtensorMap tq = make_tmap_2d(a.q, (uint64_t)a.H * a.D, a.T, a.ldq, 64, kPM);
-  const CUtensorMap tk = make_tmap_2d(a.k_cache, a.D, (uint64_t)a.num_cache_blocks * a.G * 16, a.D, 64, 16);
+  const CUtensorMap tk = make_tmap_2d(keys, (uint64_t)a.G * a.D, (uint64_t)n_pages * 16, (uint64_t)a.G * a.D, 64, kPN);
   TalkPrefillParams p;
   p.tiles = reinterpret_cast<const int4*>(tiles);
-  p.block_tables = a.block_tables;
-  p.max_blocks = a.max_blocks;
   p.bias = a.bias;
   p.bias_len = a.bias_len;
   p.qscale = a.qscale;
@@ -980,7 +991,6 @@ bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_t
   p.G = a.G;
   p.group = a.H / a.G;
   p.mc = (a.G + chunks - 1) / chunks;
-  p.num_cache_blocks = a.num_cache_blocks;
   p.status = a.status;
   if (a.D == 128) launch_prefill_t<128>(tq, tk, p, n_tiles, chunks, s);
   else launch_prefill_t<64>(tq, tk, p, n_tiles, chunks, s);

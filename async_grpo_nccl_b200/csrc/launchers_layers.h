@@ -75,9 +75,11 @@ struct WindowAttnArgs {
 };
 void launch_window_attn(bool fp32, const WindowAttnArgs& a, cudaStream_t s);
 
-// Tensor-core forms (bf16, D = 64 or 128, block_size 16). tiles: [n_tiles, 4] = {first row, rows, position of the first
-// row, slot}; acc: scratch [T, H, G, D] bf16. Returns false, having launched nothing, for shapes that are not served.
-bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_tiles, void* acc, cudaStream_t s);
+// Tensor-core forms (bf16, D = 64 or 128, block_size 16). pages [n_pages, 2] = {slot, page of the sequence}: what the step can see,
+// gathered into keys [16 n_pages, G * D]; tiles [n_tiles, 4] = {first row, rows, position of the first row, row of position 0 in
+// keys}; acc: scratch [T, H, G, D] bf16. Returns false, having launched nothing, for shapes that are not served.
+bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_tiles, const int* pages, int n_pages, void* keys, void* acc,
+                              cudaStream_t s);
 // Decode: short convolution of the new token, attention, mixing, gate and ring / cache update in one kernel (row = slot).
 struct TalkDecodeArgs {
   WindowAttnArgs at;      // q unused: the kernel convolves q itself

@@ -104,7 +104,7 @@ class ListedEngine(RolloutEngine):
     def _forward(self, segments: Sequence[Tuple[int, int, np.ndarray]]) -> torch.Tensor:
         """One step over segments (slot, tokens already cached, new tokens): keys and rings are updated, the final normed
         hidden states of all rows come back."""
-        flat, where = host_batch(segments, [l.mixer.conv for l in self.cfg.layers])
+        flat, where = host_batch(segments, [l.mixer.conv for l in self.cfg.layers], self.cfg.max_window)
         dev_flat = torch.from_numpy(flat).pin_memory().to(self.dev, non_blocking=True)
         self.h2d_bytes += flat.nbytes
         ids, sb = split_batch(dev_flat, where, self.block_tables)

@@ -22,6 +22,7 @@ from .layout import ParamLayout
 
 LOG2E = 1.4426950408889634
 TILE = 128  # query rows per attention tile
+PAGE = 16   # tokens per cache block
 
 
 @dataclass
@@ -31,16 +32,19 @@ class StepBatch:
     block_tables: torch.Tensor
     rows: Optional[torch.Tensor] = None      # [T, 4] int32: slot, position, first row of the segment, 0
     ring_rows: Optional[Dict[int, torch.Tensor]] = None  # taps -> the last `taps` rows of each segment
-    tiles: Optional[torch.Tensor] = None     # [n, 4]: first row, rows, position of the first row, slot
+    tiles: Optional[torch.Tensor] = None     # [n, 4]: first row, rows, position of the first row, row of position 0 in the gathered keys
+    pages: Optional[torch.Tensor] = None     # [n, 2]: slot, page: the key pages that the step can see, in the order they are gathered
     seq_lens: Optional[torch.Tensor] = None
     splits: int = 1
     scratch: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None  # decode: partial products, (max, sum), tickets
 
 
-def host_batch(segments: Sequence[Tuple[int, int, np.ndarray]], taps: Sequence[int]) -> Tuple[np.ndarray, Dict[str, Tuple[int, int]]]:
+def host_batch(segments: Sequence[Tuple[int, int, np.ndarray]], taps: Sequence[int], window: int) -> Tuple[np.ndarray, Dict[str, Tuple[int, int]]]:
     """(slot, tokens already there, new tokens) per segment -> one int32 array with the step's tables and where each of them
-    is in it: token ids, rows, attention tiles and, for every length in ``taps``, the rows that the convolution rings keep."""
-    ids, rows, tiles = [], [], []
+    is in it: token ids, rows, attention tiles, the key pages within ``window`` and, for every length in ``taps``, the rows
+    that the convolution rings keep."""
+    ids, rows, tiles, pages = [], [], [], []
+    n_pages = 0
     keep: Dict[int, List[np.ndarray]] = {k: [] for k in sorted(set(taps))}
     t0 = 0
     for slot, past, toks in segments:
@@ -49,13 +53,18 @@ def host_batch(segments: Sequence[Tuple[int, int, np.ndarray]], taps: Sequence[i
         r = np.zeros((n, 4), np.int32)
         r[:, 0], r[:, 1], r[:, 2] = slot, past + np.arange(n), t0
         rows.append(r)
-        tiles += [(t0 + a, min(TILE, n - a), past + a, slot) for a in range(0, n, TILE)]
+        first = max(0, past - window + 1) // PAGE
+        count = (past + n - 1) // PAGE + 1 - first
+        pages.append(np.stack([np.full(count, slot, np.int32), np.arange(first, first + count, dtype=np.int32)], axis=1))
+        tiles += [(t0 + a, min(TILE, n - a), past + a, (n_pages - first) * PAGE) for a in range(0, n, TILE)]
+        n_pages += count
         for k, v in keep.items():
             v.append(np.arange(t0 + max(0, n - k), t0 + n, dtype=np.int32))
         t0 += n
     tiles.sort(key=lambda t: -t[2])
-    parts = {"rows": np.concatenate(rows).ravel(), "tiles": np.asarray(tiles, np.int32).ravel(), "ids": np.concatenate(ids),
-             **{f"ring{k}": np.concatenate(v) for k, v in keep.items()}}   # the two tables of int4 come first: 16-byte aligned
+    parts = {"rows": np.concatenate(rows).ravel(), "tiles": np.asarray(tiles, np.int32).ravel(),
+             "pages": np.concatenate(pages).ravel(), "ids": np.concatenate(ids),
+             **{f"ring{k}": np.concatenate(v) for k, v in keep.items()}}   # tables of int4 and int2 come first: aligned
     where, o = {}, 0
     for k, v in parts.items():
         where[k] = (o, len(v))
@@ -67,6 +76,7 @@ def split_batch(flat: torch.Tensor, where: Dict[str, Tuple[int, int]], block_tab
     part = {k: flat[o:o + n] for k, (o, n) in where.items()}
     T = where["ids"][1]
     return part["ids"], StepBatch(T, block_tables, rows=part["rows"].view(T, 4), tiles=part["tiles"].view(-1, 4),
+                                  pages=part["pages"].view(-1, 2),
                                   ring_rows={int(k[4:]): v for k, v in part.items() if k.startswith("ring")})
 
 
@@ -168,9 +178,10 @@ class ListedDecoder:
         C.short_conv(u, self.conv[i], ring, sb.rows, sb.ring_rows[m.conv] if sb.rows is not None else None, sb.seq_lens, sb.block_tables, q, k_cache, self.status)
         if sb.rows is not None and not self.fp32:
             acc = torch.empty(sb.T * m.heads * m.k_dim, dtype=self.dtype, device=self.dev)
-            if C.talk_attn_prefill(q, k_cache, sb.tiles, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate, m.window,
+            keys = torch.empty(sb.pages.shape[0] * PAGE * m.k_dim, dtype=self.dtype, device=self.dev)
+            if C.talk_attn_prefill(q, k_cache, sb.tiles, sb.pages, keys, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate, m.window,
                                    acc, out, self.status):
-                self.launches += 4
+                self.launches += 5
                 return
         C.window_attn(q, k_cache, sb.rows, sb.seq_lens, sb.block_tables, self.bias[i], self.qscale[i], self.w(p + "talk"), gate,
                       m.window, out, self.status)

@@ -142,9 +142,10 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
     cache = R(n_seq * nb, G, 16, D)
     tables = torch.randperm(n_seq * nb, device=dev).int().view(n_seq, nb).contiguous()
     ring = torch.zeros(max(n_seq, B), m.conv, m.qk_dim, device=dev, dtype=bf)
-    flat, where = host_batch([(i, 0, np.zeros(prompt, np.int32)) for i in range(n_seq)], [m.conv])
+    flat, where = host_batch([(i, 0, np.zeros(prompt, np.int32)) for i in range(n_seq)], [m.conv], m.window)
     _, sb = split_batch(torch.from_numpy(flat).to(dev), where, tables)
     acc = torch.empty(T * H * G * D, device=dev, dtype=bf)
+    keys = torch.empty(sb.pages.shape[0] * 16 * G * D, device=dev, dtype=bf)
     lse = torch.empty(H, T, device=dev)
     tiles = _tiles([prompt] * n_seq)
     pairs = n_seq * sum(min(i + 1, m.window) for i in range(prompt))
@@ -162,7 +163,7 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
         C.rope_inplace(qkv, pos, cos, cos, H + G, D, False)
         C.kv_cache_write(qkv, slots, kc, vc, H, G, D, st, 0)
     add("prompt position op", "old", rope, 0.0, 4.0 * T * (H + G) * D + 8.0 * T * G * D)
-    add("prompt attention", "new", lambda: C.talk_attn_prefill(q, cache, sb.tiles, tables, bias, qscale, talk, u[:, m.qk_dim:], m.window, acc, a, st),
+    add("prompt attention", "new", lambda: C.talk_attn_prefill(q, cache, sb.tiles, sb.pages, keys, tables, bias, qscale, talk, u[:, m.qk_dim:], m.window, acc, a, st),
         4.0 * pairs * H * D, 0.0)
     add("prompt attention", "old", lambda: C.attn_varlen_fwd(qkv, a, lse, tiles, H, G, D, 0.1, st), 4.0 * pairs_old * H * D, 0.0)
     add("prompt out projection + tail", "new", lambda: C.gemm_dyt(a, wo, x, nrm, nrm, ho, st), *gm(T, W, H * D))

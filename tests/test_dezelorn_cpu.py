@@ -100,12 +100,15 @@ def test_random_init_clears_padding():
 
 
 def test_step_tables():
-    flat, where = host_batch([(3, 5, np.arange(130)), (1, 0, np.asarray([7, 8]))], [4, 1, 4])
+    flat, where = host_batch([(3, 5, np.arange(130)), (1, 0, np.asarray([7, 8]))], [4, 1, 4], 1000)
     ids, sb = split_batch(torch.from_numpy(flat), where, torch.zeros(4, 4, dtype=torch.int32))
     assert sb.T == 132 and ids.tolist() == list(range(130)) + [7, 8]
     assert sb.rows[0].tolist() == [3, 5, 0, 0] and sb.rows[129].tolist() == [3, 134, 0, 0] and sb.rows[131].tolist() == [1, 1, 130, 0]
     assert {k: v.tolist() for k, v in sb.ring_rows.items()} == {1: [129, 131], 4: [126, 127, 128, 129, 130, 131]}
-    assert sorted(map(tuple, sb.tiles.tolist())) == [(0, 128, 5, 3), (128, 2, 133, 3), (130, 2, 0, 1)]
+    assert sorted(map(tuple, sb.tiles.tolist())) == [(0, 128, 5, 0), (128, 2, 133, 0), (130, 2, 0, 144)]
+    assert sb.pages.tolist() == [[3, p] for p in range(9)] + [[1, 0]]
+    _, near = split_batch(*[f(x) for f, x in zip((torch.from_numpy, lambda w: w), host_batch([(2, 100, np.arange(3))], [1], 20))], None)
+    assert near.pages.tolist() == [[2, 5], [2, 6]] and near.tiles.tolist() == [[0, 3, 100, -80]]
     assert sb.rows.storage_offset() % 4 == 0 and sb.tiles.storage_offset() % 4 == 0
 
 

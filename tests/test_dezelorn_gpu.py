@@ -291,7 +291,7 @@ class AttnCase:
         out = torch.zeros(n, H * D, device="cuda", dtype=self.dt)
         part = (torch.empty(3 * 8 * H * G * D, device="cuda"), torch.empty(3 * 8 * H * 2, device="cuda"), torch.zeros(3, dtype=torch.int32, device="cuda"))
         if prompt:
-            flat, where = host_batch([(self.slot, 0, np.arange(prompt))], [self.taps])
+            flat, where = host_batch([(self.slot, 0, np.arange(prompt))], [self.taps], self.window)
             _, sb = split_batch(torch.from_numpy(flat).cuda(), where, tables)
             q = torch.empty(prompt, H * D, device="cuda", dtype=self.dt)
             C.short_conv(u[:prompt], conv, ring, sb.rows, sb.ring_rows[self.taps], None, tables, q, cache, st)
@@ -300,7 +300,8 @@ class AttnCase:
             if plain or self.dt == torch.float32:
                 C.window_attn(q, cache, sb.rows, None, tables, self.bias, self.qscale, talk, u[:prompt, qk:], self.window, o, st)
             else:
-                assert C.talk_attn_prefill(q, cache, sb.tiles, tables, self.bias, self.qscale, talk, u[:prompt, qk:], self.window, acc, o, st)
+                keys = torch.empty(sb.pages.shape[0] * 16 * G * D, device="cuda", dtype=self.dt)
+                assert C.talk_attn_prefill(q, cache, sb.tiles, sb.pages, keys, tables, self.bias, self.qscale, talk, u[:prompt, qk:], self.window, acc, o, st)
         for t in range(prompt, n):
             lens = torch.tensor([0, t + 1, 0], dtype=torch.int32, device="cuda")
             ub = torch.zeros(3, u.shape[1], device="cuda", dtype=self.dt)
