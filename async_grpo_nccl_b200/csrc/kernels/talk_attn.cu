@@ -461,7 +461,8 @@ void launch_prefill_t(const CUtensorMap& tq, const CUtensorMap& tk, const TalkPr
 }
 
 // ================================================================================================
-// Decode: CTA = (split, sequence), all heads: 8 warps per MTW row tiles of 16 heads plus one warp that loads. The prologue convolves the new token's q (every split) and k (the
+// Decode: CTA = (split, sequence), all heads: 8 warps per MTW row tiles of 16 heads; with one group of warps a further warp
+// loads, with two (where it would cost the others registers) the first warp does. The prologue convolves the new token's q (every split) and k (the
 // split that owns the newest token, which also writes the key page and the ring). Key tiles of 64 tokens arrive by TMA, page
 // by page, from before the new token's projections are complete. Per tile: a warp scores its 8 keys against its heads, the
 // CTA agrees on the row maxima, the weights meet in shared memory, and the warp accumulates its share of the G * D value
@@ -515,12 +516,12 @@ __device__ __forceinline__ void compute_bar() { asm volatile("bar.sync 1, %0;" :
 
 // MW groups of 8 warps, MTW row tiles of 16 heads per warp, up to NTW 8-wide value-column tiles per warp
 template <int D, int MW, int MTW, int NTW>
-__global__ void __launch_bounds__(MW * 256 + 32, (MW == 1 && NTW <= 4) ? 2 : 1)
+__global__ void __launch_bounds__(MW == 1 ? 288 : 512, (MW == 1 && NTW <= 4) ? 2 : 1)
 talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs a, const int n_stages) {
   constexpr int MT = MW * MTW;
   constexpr int kDThreads = MW * 256;                            // computing threads
   constexpr int kPl = D / 64;                                    // planes of 64 channels
-  constexpr bool kQReg = MTW == 1 && NTW <= (MW == 1 ? 8 : 4);                   // query fragments stay in registers
+  constexpr bool kQReg = MTW == 1 && NTW <= 8;                   // query fragments stay in registers
   extern __shared__ __align__(1024) uint8_t td_smem[];
   const WindowAttnArgs& p = a.at;
   const int H = p.H, G = p.G, grp = H / G, GD = G * D;
@@ -559,43 +560,49 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
     fence_mbar_init();
   }
   __syncthreads();
-  if (warp == MW * 8) {
-    // ---- the loading warp: lane -> page (lane & 3) of a tile, looked up one tile ahead ----
-    int stage = 0;
-    uint32_t phase = 1;
-    auto page_of = [&](int t) {
-      const int bi = (jb + t * kDT) / 16 + (lane & 3);
-      return table[bi > pos / 16 ? pos / 16 : bi];  // past the end: any valid page, masked
-    };
-    int next = t_begin < t_end ? page_of(t_begin) : 0;
+  // ---- loads: lane -> page (lane & 3) of a tile, looked up one tile ahead ----
+  auto page_of = [&](int t) {
+    const int bi = (jb + t * kDT) / 16 + (lane & 3);
+    return t < t_end ? table[bi > pos / 16 ? pos / 16 : bi] : 0;  // past the end: any valid page, masked
+  };
+  int next_page = 0;
+  auto load_tile = [&](int t, int st) {
+    int page = next_page;
+    next_page = page_of(t + 1);
+    if (page < 0 || page >= p.num_cache_blocks) {
+      report_status(p.status, kStatusBadIndex);
+      page = 0;
+    }
+    if (lane == 0) mbar_expect_tx(&full[st], stage_bytes);
+    __syncwarp();
+    uint8_t* dst = sKV + st * stage_bytes + (lane & 3) * (16 * 128);
+    for (int i = lane >> 2; i < G * kPl; i += 8)
+      tma_load_2d(dst + i * (kDT * 128), &tmK, &full[st], (i % kPl) * 64, (page * G + i / kPl) * 16);
+  };
+  if (MW == 1 && warp == 8) {
+    next_page = page_of(t_begin);
+    int st = 0;
+    uint32_t ph = 1;
     for (int t = t_begin; t < t_end; ++t) {
-      int page = next;
-      if (t + 1 < t_end) next = page_of(t + 1);
-      if (page < 0 || page >= p.num_cache_blocks) {
-        report_status(p.status, kStatusBadIndex);
-        page = 0;
-      }
       int good = 1;
-      if (lane == 0) {
-        if (!mbar_wait(&empty[stage], phase)) {
-          report_status(p.status, kStatusWaitEmptyTimeout);
-          good = 0;
-        } else {
-          mbar_expect_tx(&full[stage], stage_bytes);
-        }
+      if (lane == 0 && !mbar_wait(&empty[st], ph)) {
+        report_status(p.status, kStatusWaitEmptyTimeout);
+        good = 0;
       }
-      good = __shfl_sync(0xffffffffu, good, 0);
-      if (!good) break;
-      uint8_t* dst = sKV + stage * stage_bytes + (lane & 3) * (16 * 128);
-      for (int i = lane >> 2; i < G * kPl; i += 8)
-        tma_load_2d(dst + i * (kDT * 128), &tmK, &full[stage], (i % kPl) * 64, (page * G + i / kPl) * 16);
-      if (++stage == n_stages) {
-        stage = 0;
-        phase ^= 1;
+      if (!__shfl_sync(0xffffffffu, good, 0)) break;
+      load_tile(t, st);
+      if (++st == n_stages) {
+        st = 0;
+        ph ^= 1;
       }
     }
     pdl_wait();
     return;
+  }
+  if (MW == 2 && warp == 0) {
+    next_page = page_of(t_begin);
+    for (int i = 0; i < (n_stages > 1 ? n_stages - 1 : 1); ++i)
+      if (t_begin + i < t_end) load_tile(t_begin + i, i);
   }
   if (p.talk != nullptr)
     for (int i = tid; i < H * H; i += kDThreads) sTalk[i] = ldf(reinterpret_cast<const bf16*>(p.talk) + i);
@@ -628,24 +635,17 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
   }
 
   const float qs = p.qscale[pos < p.qscale_len ? pos : p.qscale_len - 1];
-  const int npw = (GD / 8 + 7) / 8;              // 8-wide value-column tiles per warp
   const int cw = warp & 7, mt0 = (warp >> 3) * MTW;  // warp within its group, first row tile
-  const int nt0 = cw * npw;
+  const int nt0 = cw * NTW;                      // first of this warp's 8-wide value-column tiles
+  const int n_cols = GD / 8;
   const int r0 = lane >> 2, cq = (lane & 3) * 2;
   // fragment addresses that do not change from tile to tile (inside a stage)
   const uint32_t k_off = sw_off(cw * 8 + (lane & 7), lane >> 3);                       // keys: chunks 0-3; chunks 4-7 at ^ 64
   const uint32_t q_off = smem_u32(sQ) + mt0 * kPl * 2048 + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, lane >> 4);  // queries: k-step s at ^ (s * 32)
   const uint32_t p_off = smem_u32(sP) + ((mt0 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + (lane >> 4) * 8) * 2;
-  constexpr int kPairs = NTW > 1 ? NTW / 2 : 1;
-  uint32_t v_off[kPairs];                        // value columns: two neighbouring 8-wide tiles per ldmatrix
-#pragma unroll
-  for (int i = 0; i < kPairs; ++i) {
-    const int n1 = nt0 + 2 * i < GD / 8 ? nt0 + 2 * i : GD / 8 - 1;
-    const int n2 = n1 + 1 < GD / 8 ? n1 + 1 : n1;
-    const int nn = (lane >> 4) ? n2 : n1;
-    const int m = nn / (D / 8), ch = nn % (D / 8);
-    v_off[i] = (m * kPl + (ch >> 3)) * (kDT * 128) + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, ch & 7);
-  }
+  constexpr int kPairs = NTW / 2;
+  // value columns, two neighbouring 8-wide tiles per ldmatrix: pair i at (+ (i >> 2) planes) ^ (i & 3) * 32
+  const uint32_t v_off = (nt0 >> 3) * (kDT * 128) + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, (nt0 & 7) + (lane >> 4));
   const float* bias_row[MTW][2];                  // rows past the last head read the last head's biases; they are never stored
   int key_head[MTW][2];
 #pragma unroll
@@ -764,6 +764,10 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
       }
     }
     compute_bar<kDThreads>();
+    if (MW == 2 && n_stages > 1 && warp == 0) {  // everybody is done with the tile before: its stage is free
+      const int t_next = t + n_stages - 1;
+      if (t_next < t_end) load_tile(t_next, stage == 0 ? n_stages - 1 : stage - 1);
+    }
     // ---- weights ----
 #pragma unroll
     for (int mt = 0; mt < MTW; ++mt) {
@@ -798,19 +802,24 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
       for (int mt = 0; mt < MTW; ++mt) ldsm4(pf[mt], p_off + (mt * 16 * kPPitch + kk * 16) * 2);
 #pragma unroll
       for (int i = 0; i < kPairs; ++i) {
-        if (2 * i < npw) {   // columns past the end repeat the last ones; they are never stored
+        if (nt0 + 2 * i < n_cols) {
           uint32_t vf[4];
-          ldsm4_t(vf, kts + v_off[i] + kk * 2048);
+          ldsm4_t(vf, (kts + v_off + kk * 2048 + (i >> 2) * (kDT * 128)) ^ ((i & 3) * 32));
 #pragma unroll
           for (int mt = 0; mt < MTW; ++mt) {
             mma_16816(acc[mt][2 * i], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[0], vf[1]);
-            if constexpr (NTW > 1) mma_16816(acc[mt][2 * i + 1], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[2], vf[3]);
+            mma_16816(acc[mt][2 * i + 1], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[2], vf[3]);
           }
         }
       }
     }
-    __syncwarp();
-    if (lane == 0) mbar_arrive(&empty[stage]);
+    if (MW == 1) {
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&empty[stage]);
+    } else if (n_stages == 1) {
+      compute_bar<kDThreads>();
+      if (warp == 0 && t + 1 < t_end) load_tile(t + 1, 0);
+    }
     if (++stage == n_stages) {
       stage = 0;
       phase ^= 1;
@@ -843,7 +852,7 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
       float* dst = a.splits == 1 ? prod + (size_t)h * GD : a.part_o + (part + h) * GD;
 #pragma unroll
       for (int i = 0; i < NTW; ++i)
-        if (i < npw && nt0 + i < GD / 8)
+        if (nt0 + i < n_cols)
           *reinterpret_cast<float2*>(dst + (nt0 + i) * 8 + cq) = make_float2(acc[mt][i][2 * q] * inv, acc[mt][i][2 * q + 1] * inv);
       if (a.splits > 1 && cw == 0 && (lane & 3) == 0)
         *reinterpret_cast<float2*>(a.part_ml + (part + h) * 2) = make_float2(mrow[mt][q], l);
@@ -944,7 +953,7 @@ void launch_decode_t(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) 
   AGRPO_SET_MAX_DYN_SMEM(kernel, 226 * 1024, "talk_decode smem attr");
   AGRPO_PREFER_SMEM(kernel);
   const CUtensorMap tk = make_tmap_2d(a.k_cache, D, (uint64_t)a.at.num_cache_blocks * a.at.G * 16, D, 64, 16);
-  launch_kernel(kernel, dim3(a.splits, a.at.T), dim3(MW * 256 + 32), d.smem, s, "talk_decode", tk, a, d.stages);
+  launch_kernel(kernel, dim3(a.splits, a.at.T), dim3(MW == 1 ? 288 : 512), d.smem, s, "talk_decode", tk, a, d.stages);
 }
 template <int D, int MW, int MTW>
 void launch_decode_n(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) {
