@@ -566,6 +566,11 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
     return t < t_end ? table[bi > pos / 16 ? pos / 16 : bi] : 0;  // past the end: any valid page, masked
   };
   int next_page = 0;
+  auto issue_tile = [&](int page, int st) {
+    uint8_t* dst = sKV + st * stage_bytes + (lane & 3) * (16 * 128);
+    for (int i = lane >> 2; i < G * kPl; i += 8)
+      tma_load_2d(dst + i * (kDT * 128), &tmK, &full[st], (i % kPl) * 64, (page * G + i / kPl) * 16);
+  };
   auto load_tile = [&](int t, int st) {
     int page = next_page;
     next_page = page_of(t + 1);
@@ -575,22 +580,30 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
     }
     if (lane == 0) mbar_expect_tx(&full[st], stage_bytes);
     __syncwarp();
-    uint8_t* dst = sKV + st * stage_bytes + (lane & 3) * (16 * 128);
-    for (int i = lane >> 2; i < G * kPl; i += 8)
-      tma_load_2d(dst + i * (kDT * 128), &tmK, &full[st], (i % kPl) * 64, (page * G + i / kPl) * 16);
+    issue_tile(page, st);
   };
   if (MW == 1 && warp == 8) {
-    next_page = page_of(t_begin);
     int st = 0;
     uint32_t ph = 1;
+    int next = t_begin < t_end ? page_of(t_begin) : 0;
     for (int t = t_begin; t < t_end; ++t) {
+      int page = next;
+      if (t + 1 < t_end) next = page_of(t + 1);
+      if (page < 0 || page >= p.num_cache_blocks) {
+        report_status(p.status, kStatusBadIndex);
+        page = 0;
+      }
       int good = 1;
-      if (lane == 0 && !mbar_wait(&empty[st], ph)) {
-        report_status(p.status, kStatusWaitEmptyTimeout);
-        good = 0;
+      if (lane == 0) {
+        if (!mbar_wait(&empty[st], ph)) {
+          report_status(p.status, kStatusWaitEmptyTimeout);
+          good = 0;
+        } else {
+          mbar_expect_tx(&full[st], stage_bytes);
+        }
       }
       if (!__shfl_sync(0xffffffffu, good, 0)) break;
-      load_tile(t, st);
+      issue_tile(page, st);
       if (++st == n_stages) {
         st = 0;
         ph ^= 1;
@@ -644,8 +657,13 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
   const uint32_t q_off = smem_u32(sQ) + mt0 * kPl * 2048 + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, lane >> 4);  // queries: k-step s at ^ (s * 32)
   const uint32_t p_off = smem_u32(sP) + ((mt0 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + (lane >> 4) * 8) * 2;
   constexpr int kPairs = NTW / 2;
-  // value columns, two neighbouring 8-wide tiles per ldmatrix: pair i at (+ (i >> 2) planes) ^ (i & 3) * 32
+  // value columns, two neighbouring 8-wide tiles per ldmatrix: pair i at (+ (i >> 2) planes) ^ (i & 3) * 32; few pairs keep
+  // their addresses in registers
+  constexpr bool kVReg = NTW <= 4;
   const uint32_t v_off = (nt0 >> 3) * (kDT * 128) + sw_off((lane & 7) + ((lane >> 3) & 1) * 8, (nt0 & 7) + (lane >> 4));
+  uint32_t v_pair[kVReg ? kPairs : 1];
+#pragma unroll
+  for (int i = 0; i < (kVReg ? kPairs : 1); ++i) v_pair[i] = v_off ^ (i * 32);
   const float* bias_row[MTW][2];                  // rows past the last head read the last head's biases; they are never stored
   int key_head[MTW][2];
 #pragma unroll
@@ -804,7 +822,7 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
       for (int i = 0; i < kPairs; ++i) {
         if (nt0 + 2 * i < n_cols) {
           uint32_t vf[4];
-          ldsm4_t(vf, (kts + v_off + kk * 2048 + (i >> 2) * (kDT * 128)) ^ ((i & 3) * 32));
+          ldsm4_t(vf, kVReg ? kts + v_pair[kVReg ? i : 0] + kk * 2048 : (kts + v_off + kk * 2048 + (i >> 2) * (kDT * 128)) ^ ((i & 3) * 32));
 #pragma unroll
           for (int mt = 0; mt < MTW; ++mt) {
             mma_16816(acc[mt][2 * i], pf[mt][0], pf[mt][1], pf[mt][2], pf[mt][3], vf[0], vf[1]);
