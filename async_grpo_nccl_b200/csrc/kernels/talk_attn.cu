@@ -231,32 +231,42 @@ talk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const int tk = j0 + j * kPN;            // first key of the tile
       const int d0 = qi - (tk + half * kPKeys);  // distance of this thread's first key
       const bool inside = tk + kPN - 1 <= pos0 && pos0 + kPM - 1 - tk < p.window && pos0 + kPM - 1 - tk < p.bias_len;
-      float v[kPKeys];                        // distance biases, on their way while the scores are computed
-      if (inside) {
-#pragma unroll
-        for (int i = 0; i < kPKeys; ++i) v[i] = __ldg(bias + d0 - i);
-      } else {
-#pragma unroll
-        for (int i = 0; i < kPKeys; ++i) {
-          const int d = d0 - i;
-          v[i] = d >= 0 && d < p.window && d < p.bias_len ? __ldg(bias + d) : INFINITY;
-        }
-      }
       if (ok && !mbar_wait(&s_full[group], (j >> 1) & 1)) {
         report_status(p.status, kStatusWaitTmemFullTimeout);
         ok = false;
       }
       tc_fence_after();
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+      float v[kPKeys];
+      // small pieces: a spill would cost an L2 round trip next to this much shared memory
+      if (inside) {
 #pragma unroll
-      for (int c = 0; c < kPKeys; c += 16) {
-        uint32_t s0[16];
-        tmem_ld_32x16(tS + half * kPKeys + c, s0);
-        tc_wait_ld();
+        for (int c = 0; c < kPKeys; c += 8) {
+          uint32_t s0[8];
+          tmem_ld_32x8(tS + half * kPKeys + c, s0);
+          float b[8];
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          v[c + i] = fmaf(__uint_as_float(s0[i]), qs, -v[c + i]);  // masked keys: minus infinity
-          mx4[i & 3] = fmaxf(mx4[i & 3], v[c + i]);
+          for (int i = 0; i < 8; ++i) b[i] = __ldg(bias + d0 - c - i);
+          tc_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            v[c + i] = fmaf(__uint_as_float(s0[i]), qs, -b[i]);
+            mx4[i & 3] = fmaxf(mx4[i & 3], v[c + i]);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int c = 0; c < kPKeys; c += 8) {
+          uint32_t s0[8];
+          tmem_ld_32x8(tS + half * kPKeys + c, s0);
+          tc_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const int d = d0 - c - i;
+            const float b = d >= 0 && d < p.window && d < p.bias_len ? __ldg(bias + d) : INFINITY;
+            v[c + i] = fmaf(__uint_as_float(s0[i]), qs, -b);  // masked keys: minus infinity
+            mx4[i & 3] = fmaxf(mx4[i & 3], v[c + i]);
+          }
         }
       }
       // the maximum is only a reference point: kept in bf16, the same rounded value for all threads of a row
@@ -803,12 +813,14 @@ talk_decode_kernel(const __grid_constant__ CUtensorMap tmK, const TalkDecodeArgs
         lrow[mt][q] = lrow[mt][q] * al[q] + p0 + p1;
         *reinterpret_cast<uint32_t*>(sP + (row * kPPitch + cw * 8 + cq) * 2) = pack_bf16x2(p0, p1);
       }
+      if (__any_sync(0xffffffffu, al[0] != 1.f || al[1] != 1.f)) {
 #pragma unroll
-      for (int i = 0; i < NTW; ++i) {
-        acc[mt][i][0] *= al[0];
-        acc[mt][i][1] *= al[0];
-        acc[mt][i][2] *= al[1];
-        acc[mt][i][3] *= al[1];
+        for (int i = 0; i < NTW; ++i) {
+          acc[mt][i][0] *= al[0];
+          acc[mt][i][1] *= al[0];
+          acc[mt][i][2] *= al[1];
+          acc[mt][i][3] *= al[1];
+        }
       }
     }
     compute_bar<kDThreads>();
