@@ -248,7 +248,7 @@ void bind_layer_ops(pybind11::module_& m) {
   m.def("talk_attn_decode", &talk_attn_decode, py::arg("u"), py::arg("conv_w"), py::arg("ring"), py::arg("k_cache"), py::arg("seq_lens"),
         py::arg("block_tables"), py::arg("bias"), py::arg("qscale"), py::arg("talk"), py::arg("gate"), py::arg("window"), py::arg("out"),
         py::arg("splits"), py::arg("part_o"), py::arg("part_ml"), py::arg("tickets"), py::arg("status"), NoGil());
-  m.def("talk_decode_supported", &agrpo::talk_decode_supported);
+  m.def("talk_decode_ctas_per_sm", &agrpo::talk_decode_ctas_per_sm);
   m.def("gemm_dyt", &gemm_dyt, py::arg("a"), py::arg("b"), py::arg("x"), py::arg("n1"), py::arg("n2"), py::arg("h"), py::arg("status"),
         py::arg("num_sms") = 0, NoGil());
   m.def("gemm_f32", &gemm_f32, NoGil());

@@ -1039,7 +1039,10 @@ bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_t
   return true;
 }
 
-bool talk_decode_supported(int H, int G, int D) { return plan_decode_kernel(H, G, D).mw > 0; }
+int talk_decode_ctas_per_sm(int H, int G, int D) {
+  const DecPlan d = plan_decode_kernel(H, G, D);
+  return d.mw == 0 ? 0 : (d.mw == 1 && d.ntw <= 4 ? 2 : 1);
+}
 
 void launch_talk_attn_decode(const TalkDecodeArgs& a, cudaStream_t s) {
   const DecPlan d = plan_decode_kernel(a.at.H, a.at.G, a.at.D);

@@ -96,7 +96,7 @@ struct TalkDecodeArgs {
   float* part_ml;         // [B, splits, H, 2]
   int* tickets;           // [B], zero-initialised, re-armed by the kernel
 };
-bool talk_decode_supported(int H, int G, int D);
+int talk_decode_ctas_per_sm(int H, int G, int D);  // 0: shape not served
 void launch_talk_attn_decode(const TalkDecodeArgs& a, cudaStream_t s);
 
 // y = a . b^T in true fp32 (no tensor cores), every output summed over K in the same order whatever the batch.

@@ -66,6 +66,7 @@ class ListedEngine(RolloutEngine):
         self.b_h = torch.zeros(S, W, dtype=self.dtype, device=self.dev)
         self.b_buf = {k: t.zero_() for k, t in self.dec.buffers(S).items()}  # idle rows hold numbers, not garbage
         self.max_splits = 8
+        self.ctas_per_sm = max(1, min(self.dec.decode_ctas_per_sm(i) for i in range(len(self.cfg.layers))))
         ms = [l.mixer for l in self.cfg.layers]
         f32 = dict(dtype=torch.float32, device=self.dev)
         self.b_scratch = (torch.empty(S * self.max_splits * max(m.heads * m.k_dim for m in ms), **f32),
@@ -165,14 +166,14 @@ class ListedEngine(RolloutEngine):
             self.C.set_pdl(False)
 
     def _choose_splits(self, B: int, n_active: int, max_len: int) -> int:
-        """Two CTAs per SM where there are few sequences, each with at least two tiles of 64 keys."""
-        want = (self.sm_count * 2) // max(1, n_active)
+        """One wave of CTAs where there are few sequences, each with at least two tiles of 64 keys."""
+        want = (self.sm_count * self.ctas_per_sm) // max(1, n_active)
         return int(max(1, min(self.max_splits, want, min(max_len, self.cfg.max_window) // 128)))
 
     def _launch_count_decode(self, splits: int, B: int = 0) -> int:
         n = 1 + 2
         for i, l in enumerate(self.cfg.layers):
-            n += (3 if self.dec.tensor_core_decode(i) else 5) + (0 if l.ff is None else 2)
+            n += (3 if self.dec.decode_ctas_per_sm(i) else 5) + (0 if l.ff is None else 2)
         return n
 
     # ------------------------------------------------------------------ step-wise driving

@@ -135,9 +135,10 @@ class ListedDecoder:
             self.status.zero_()
             raise RuntimeError(f"device kernel reported status {code} (bounded wait ran out or bad index)")
 
-    def tensor_core_decode(self, i: int) -> bool:
+    def decode_ctas_per_sm(self, i: int) -> int:
+        """CTAs of the fused decode mixer that fit an SM; 0 = the layer decodes with the plain kernels."""
         m = self.cfg.layers[i].mixer
-        return not self.fp32 and self.C.talk_decode_supported(m.heads, m.kv_heads, m.dim_p)
+        return 0 if self.fp32 else int(self.C.talk_decode_ctas_per_sm(m.heads, m.kv_heads, m.dim_p))
 
     def next_norm(self, i: int) -> str:
         return f"layers.{i + 1}.norm1" if i + 1 < len(self.cfg.layers) else "final_norm"
@@ -170,7 +171,7 @@ class ListedDecoder:
                    out: torch.Tensor) -> None:
         m, C, p = self.cfg.layers[i].mixer, self.C, f"layers.{i}."
         gate = u[:, m.qk_dim:]
-        if sb.rows is None and sb.scratch is not None and self.tensor_core_decode(i):
+        if sb.rows is None and sb.scratch is not None and self.decode_ctas_per_sm(i):
             C.talk_attn_decode(u, self.conv[i], ring, k_cache, sb.seq_lens, sb.block_tables, self.bias[i], self.qscale[i],
                                self.w(p + "talk"), gate, m.window, out, sb.splits, *sb.scratch, self.status)
             self.launches += 1

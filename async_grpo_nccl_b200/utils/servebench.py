@@ -196,7 +196,7 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
     tick = torch.zeros(B * G, device=dev, dtype=torch.int32)
     n_sm = torch.cuda.get_device_properties(0).multi_processor_count
     seen = min(ctx, m.window)
-    sp_new = max(1, min(8, 2 * n_sm // B, seen // 128))
+    sp_new = max(1, min(8, C.talk_decode_ctas_per_sm(H, G, D) * n_sm // B, seen // 128))
     sp_old = max(1, min(8, 3 * n_sm // (B * G), ctx // 256))
     wb = lambda N, K, extra=0: 2.0 * N * K + 2.0 * B * (N + K) + extra
     ss = torch.full((B,), W << 30, device=dev, dtype=torch.int64)
