@@ -29,7 +29,7 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "--use_fast_math",
 ]
 # files that hold 32-bit reference-grade arithmetic: no fast-math substitutions
-PRECISE_SOURCES = {"layer_ops.cu"}
+PRECISE_SOURCES = {"layer_ops.cu", "hybrid_ops.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function"]
 
 

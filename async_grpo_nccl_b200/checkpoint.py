@@ -89,7 +89,7 @@ def load_hf_model(path: str, layout: ParamLayout, out: Optional[torch.Tensor] = 
         with safe_open(os.path.join(path, fn), framework="pt", device="cpu") as f:
             for key in f.keys():
                 if key not in dest:
-                    if key == "lm_head.weight" and getattr(layout.cfg, "tie_word_embeddings", False):
+                    if layout.hf_unused(key):
                         continue
                     raise KeyError(f"unexpected tensor {key} in {fn}")
                 t = f.get_tensor(key)

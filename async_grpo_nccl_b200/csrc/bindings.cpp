@@ -545,7 +545,7 @@ void paged_decode_attn(const Tensor& qkv, const Tensor& k_cache, const Tensor& v
 int64_t lm_sample_num_groups(int64_t V, int64_t rows) { return agrpo::lm_sample_num_groups((int)V, (int)rows); }
 
 void lm_sample(const Tensor& hidden, const Tensor& weight, double temperature, const Tensor& seeds, Tensor& part_f,
-               Tensor& part_i, Tensor& tokens, const OptTensor& logprobs, const OptTensor& status) {
+               Tensor& part_i, Tensor& tokens, const OptTensor& logprobs, const OptTensor& status, double softcap) {
   check_bf16(hidden, "hidden"); check_bf16(weight, "weight"); check_f32(part_f, "part_f"); check_i32(part_i, "part_i");
   check_i32(tokens, "tokens");
   TORCH_CHECK(seeds.is_cuda() && seeds.scalar_type() == torch::kInt64 && seeds.is_contiguous(), "lm_sample: seeds int64");
@@ -558,7 +558,7 @@ void lm_sample(const Tensor& hidden, const Tensor& weight, double temperature, c
   agrpo::launch_lm_sample(hidden.data_ptr(), hidden.stride(0), weight.data_ptr(), weight.stride(0), (int)R, (int)H, (int)V,
                           (float)temperature, reinterpret_cast<const unsigned long long*>(seeds.data_ptr<int64_t>()),
                           part_f.data_ptr<float>(), part_i.data_ptr<int>(), tokens.data_ptr<int>(), opt_ptr<float>(logprobs),
-                          opt_ptr<int>(status), num_sms(), cur_stream());
+                          opt_ptr<int>(status), num_sms(), cur_stream(), (float)softcap);
 }
 
 // ---- peer-memory kernels ----
@@ -881,6 +881,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
       .def("clear_prefix_cache", &agrpo::Scheduler::clear_prefix_cache);
 
   bind_layer_ops(m);
+  bind_hybrid_ops(m);
   m.def("gemm_bf16", &gemm_bf16, py::arg("a"), py::arg("b"), py::arg("d"), py::arg("a_mn") = false,
         py::arg("b_mn") = false, py::arg("bias") = py::none(), py::arg("alpha") = 1.0, py::arg("accumulate") = false,
         py::arg("status") = py::none(), py::arg("residual") = py::none(), NOGIL);
@@ -950,7 +951,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("lm_sample_num_groups", &lm_sample_num_groups);
   m.def("lm_sample", &lm_sample, py::arg("hidden"), py::arg("weight"), py::arg("temperature"), py::arg("seeds"),
         py::arg("part_f"), py::arg("part_i"), py::arg("tokens"), py::arg("logprobs") = py::none(),
-        py::arg("status") = py::none(), NOGIL);
+        py::arg("status") = py::none(), py::arg("softcap") = 0.0, NOGIL);
   m.def("pack_count_tiles", &pack_count_tiles);
   m.def("pack_microbatch", &pack_microbatch);
   m.def("normalize_rewards", &normalize_rewards_cpu);

@@ -205,13 +205,13 @@ void gemm_dyt(const Tensor& a, const Tensor& b, Tensor& x, const std::vector<Ten
                                 num_sms > 0 ? (int)num_sms : at::cuda::getCurrentDeviceProperties()->multiProcessorCount, cur_stream());
 }
 
-void gemm_f32(const Tensor& a, const Tensor& b, Tensor& d) {
+void gemm_f32(const Tensor& a, const Tensor& b, Tensor& d, bool relu2, double softcap, bool accumulate) {
   check_f32(a, "a"); check_f32(b, "b"); check_f32(d, "d");
   rows2d(a, "a"); rows2d(b, "b"); rows2d(d, "d");
   TORCH_CHECK(a.size(1) == b.size(1) && d.size(0) == a.size(0) && d.size(1) == b.size(0), "gemm_f32: shapes");
   const c10::cuda::CUDAGuard guard(a.device());
   agrpo::launch_gemm_f32(a.data_ptr<float>(), a.stride(0), b.data_ptr<float>(), b.stride(0), d.data_ptr<float>(), d.stride(0), (int)a.size(0),
-                         (int)b.size(0), (int)a.size(1), cur_stream());
+                         (int)b.size(0), (int)a.size(1), cur_stream(), agrpo::GemmF32Post{relu2 ? 1 : 0, (float)softcap, accumulate ? 1 : 0});
 }
 void gemm_swiglu_f32(const Tensor& a, const Tensor& b, Tensor& d) {
   check_f32(a, "a"); check_f32(b, "b"); check_f32(d, "d");
@@ -251,7 +251,8 @@ void bind_layer_ops(pybind11::module_& m) {
   m.def("talk_decode_ctas_per_sm", &agrpo::talk_decode_ctas_per_sm);
   m.def("gemm_dyt", &gemm_dyt, py::arg("a"), py::arg("b"), py::arg("x"), py::arg("n1"), py::arg("n2"), py::arg("h"), py::arg("status"),
         py::arg("num_sms") = 0, NoGil());
-  m.def("gemm_f32", &gemm_f32, NoGil());
+  m.def("gemm_f32", &gemm_f32, py::arg("a"), py::arg("b"), py::arg("d"), py::arg("relu2") = false, py::arg("softcap") = 0.0,
+        py::arg("accumulate") = false, NoGil());
   m.def("gemm_swiglu_f32", &gemm_swiglu_f32, NoGil());
   m.def("sample_logits", &sample_logits, py::arg("logits"), py::arg("temperature"), py::arg("seeds"), py::arg("tokens"),
         py::arg("logprobs") = py::none(), NoGil());

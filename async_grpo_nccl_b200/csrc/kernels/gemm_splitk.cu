@@ -23,6 +23,7 @@
 #include "../launchers.h"
 #include "../launchers_layers.h"
 #include "layer_ops.cuh"
+#include "parallel_block.cuh"
 
 namespace agrpo {
 
@@ -62,6 +63,10 @@ struct SkParams {
   int M, N, K;
   SkRope rope;
   SkTail tail;
+  ProjOut proj;          // proj.u != nullptr: both projections of a parallel block (columns [n1, N) read A at column a2)
+  ResidualOut resid;     // resid.x != nullptr: fp32 residual stream and its consumers
+  int n1, a2;
+  float* d32;            // fp32 result instead of D
   __nv_bfloat16* D;
   long long ldd;
   const __nv_bfloat16* bias;
@@ -166,7 +171,11 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t crank = cluster_ctarank();
   if (threadIdx.x == 0) SK_STAMP(0);
-  const int n0 = blockIdx.y * BN;
+  const int tiles1 = p.n1 > 0 ? (p.n1 + BN - 1) / BN : 0;
+  const bool second = p.n1 > 0 && (int)blockIdx.y >= tiles1;
+  const int n0 = second ? p.n1 + ((int)blockIdx.y - tiles1) * BN : (int)blockIdx.y * BN;
+  const int n_end = p.n1 > 0 && !second ? p.n1 : p.N;
+  const int a0 = second ? p.a2 : 0;
   const int num_kb = (p.K + kBK - 1) / kBK;
   const int kb0 = (int)((long long)num_kb * crank / S);
   const int kb1 = (int)((long long)num_kb * (crank + 1) / S);
@@ -194,7 +203,7 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
     for (int i = 0; i < n_pre; ++i) {
       uint8_t* sa = smem + i * kStageBytes;
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) tma_load_2d(sa + mt * (kBM * kBK * 2), &tmA, &full_bar[i], (kb0 + i) * kBK, mt * kBM);
+      for (int mt = 0; mt < MT; ++mt) tma_load_2d(sa + mt * (kBM * kBK * 2), &tmA, &full_bar[i], a0 + (kb0 + i) * kBK, mt * kBM);
     }
     SK_STAMP(3);
   }
@@ -225,7 +234,7 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
         uint8_t* sb = sa + kABytes;
         mbar_expect_tx(&full_bar[stage], kStageBytes);
 #pragma unroll
-        for (int mt = 0; mt < MT; ++mt) tma_load_2d(sa + mt * (kBM * kBK * 2), &tmA, &full_bar[stage], kb * kBK, mt * kBM);
+        for (int mt = 0; mt < MT; ++mt) tma_load_2d(sa + mt * (kBM * kBK * 2), &tmA, &full_bar[stage], a0 + kb * kBK, mt * kBM);
         tma_load_2d(sb, &tmB, &full_bar[stage], kb * kBK, n0);
         if (++stage == STAGES) {
           stage = 0;
@@ -408,8 +417,9 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
       for (int mt = 0; mt < MT; ++mt) {
         if (mt * kBM + quarter * 32 >= p.M) continue;
         const int row = mt * kBM + row_in_tile;
-        const float rs = (p.ss_in != nullptr && row < p.M) ? rsqrtf(sumsq_from_fixed(p.ss_in[row]) * p.inv_k + p.eps) : 1.f;
-        float sq = 0.f;
+        const float rs = p.proj.u != nullptr ? p.proj.row_scale(row, p.M)
+                         : (p.ss_in != nullptr && row < p.M) ? rsqrtf(sumsq_from_fixed(p.ss_in[row]) * p.inv_k + p.eps) : 1.f;
+        float sq = 0.f, sk = 0.f;
 #pragma unroll 1
         for (int cb = 0; cb < w; cb += 8) {
           float acc[8];
@@ -425,9 +435,24 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
             }
           }
           const int col = n0 + c0 + cb;
-          if (row < p.M && col < p.N) {
+          if (row < p.M && col < n_end) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) acc[i] *= rs;
+            if (p.proj.u != nullptr) {
+              p.proj.store8(row, col, acc, sq, sk);
+              continue;
+            }
+            if (p.resid.x != nullptr) {
+              float x0[8];
+              if (p.resid.accumulate) ld8(p.resid.x + (long long)row * p.resid.ldx + col, x0);
+              p.resid.store8(row, col, x0, acc, sq);
+              continue;
+            }
+            if (p.d32 != nullptr) {
+              for (int i = 0; i < 8; ++i)
+                if (col + i < p.N) p.d32[(long long)row * p.ldd + col + i] = acc[i];
+              continue;
+            }
             if (p.tail.x != nullptr) {  // N is a multiple of 8 in this mode
               dyt_residual8(acc, p.tail.x + (long long)row * p.tail.ldx + col, p.tail.h + (long long)row * p.tail.ldh + col, p.tail.n1,
                             p.tail.n2, col, ldf(p.tail.n1.alpha), ldf(p.tail.n2.alpha));
@@ -460,6 +485,10 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
                 if (col + i < p.N) dst[i] = __float2bfloat16(acc[i]);
             }
           }
+        }
+        if (row < p.M) {
+          if (p.proj.u != nullptr) p.proj.add_stats(row, sq, sk);
+          if (p.resid.x != nullptr) p.resid.add_stats(row, sq);
         }
         if (p.ss_out != nullptr && row < p.M) sumsq_atomic_add(p.ss_out + row, sq);
       }
@@ -501,14 +530,16 @@ void launch_sk(const CUtensorMap& ta, const CUtensorMap& tb, const SkParams& p, 
 }  // namespace
 
 // Number of K splits (= cluster size) the skinny kernel would use, 0 when it does not serve the shape.
-int gemm_skinny_splits(int M, int N, int K, int num_sms) {
+static int splits_for(int n_tiles, int M, int N, int K, int num_sms) {
   if (M > 256 || K < 512 || N < 64) return 0;
-  const int BN = M <= 128 ? 128 : 64;
-  const int n_tiles = (N + BN - 1) / BN;
   const int num_kb = (K + kBK - 1) / kBK;
   int S = 8;
   while (S > 1 && (n_tiles * S > (num_sms * 3) / 2 || num_kb / S < 2)) S >>= 1;
   return S == 1 ? 0 : S;
+}
+int gemm_skinny_splits(int M, int N, int K, int num_sms) {
+  const int BN = M <= 128 ? 128 : 64;
+  return splits_for((N + BN - 1) / BN, M, N, K, num_sms);
 }
 
 // Returns false when the shape is not one this kernel serves (the caller then uses the general GEMM).
@@ -538,6 +569,10 @@ bool launch_gemm_skinny(const void* a, long long lda, const void* b, long long l
   p.ldr = ldr;
   p.rope = SkRope{};
   p.tail = SkTail{};
+  p.proj = ProjOut{};
+  p.resid = ResidualOut{};
+  p.n1 = p.a2 = 0;
+  p.d32 = nullptr;
   if (tail != nullptr) {
     typedef const __nv_bfloat16* P;
     p.tail.x = tail->x;
@@ -564,6 +599,59 @@ bool launch_gemm_skinny(const void* a, long long lda, const void* b, long long l
   p.trace = trace;
   if (MT == 1) launch_sk<128, 1, 4>(ta, tb, p, S, n_tiles, stream);
   else         launch_sk<64, 2, 3>(ta, tb, p, S, n_tiles, stream);
+  return true;
+}
+
+namespace {
+SkParams blank_params(int M, int N, int K, int* status) {
+  SkParams p{};
+  p.M = M; p.N = N; p.K = K;
+  p.inv_k = 1.f / (float)K;
+  p.status = status;
+  return p;
+}
+void launch_blank(const void* a, long long lda, int a_cols, const void* b, long long ldb, const SkParams& p, int S, int n_tiles, cudaStream_t s) {
+  const int BN = p.M <= 128 ? 128 : 64;
+  const CUtensorMap ta = make_tmap_2d(a, a_cols, p.M, lda, 64, kBM);
+  const CUtensorMap tb = make_tmap_2d(b, p.K, p.N, ldb, 64, BN);
+  if (p.M <= 128) launch_sk<128, 1, 4>(ta, tb, p, S, n_tiles, s);
+  else            launch_sk<64, 2, 3>(ta, tb, p, S, n_tiles, s);
+}
+}  // namespace
+
+bool launch_gemm_skinny_proj(const ParallelProjArgs& a, const ProjOut& out, int num_sms, cudaStream_t s) {
+  const int BN = a.M <= 128 ? 128 : 64;
+  const int n_tiles = (a.n1 + BN - 1) / BN + (a.n2 + BN - 1) / BN;
+  const int S = splits_for(n_tiles, a.M, a.n1 + a.n2, a.K, num_sms);
+  if (S == 0) return false;
+  SkParams p = blank_params(a.M, a.n1 + a.n2, a.K, a.status);
+  p.proj = out;
+  p.n1 = a.n2 > 0 ? a.n1 : 0;
+  p.a2 = a.a2;
+  launch_blank(a.h, a.lda, a.n2 > 0 ? a.a2 + a.K : a.K, a.w, a.ldw, p, S, n_tiles, s);
+  return true;
+}
+
+bool launch_gemm_skinny_residual(const ResidualArgs& a, const ResidualOut& out, int num_sms, cudaStream_t s) {
+  const int S = gemm_skinny_splits(a.M, a.N, a.K, num_sms);
+  if (S == 0) return false;
+  const int BN = a.M <= 128 ? 128 : 64;
+  SkParams p = blank_params(a.M, a.N, a.K, a.status);
+  p.resid = out;
+  launch_blank(a.a, a.lda, a.K, a.w, a.ldw, p, S, (a.N + BN - 1) / BN, s);
+  return true;
+}
+
+// fp32 result of a plain product (e.g. the narrow projection of a scan's input)
+bool launch_gemm_skinny_f32out(const void* a, long long lda, const void* b, long long ldb, float* d, long long ldd, int M, int N, int K, int* status,
+                               int num_sms, cudaStream_t s) {
+  const int S = gemm_skinny_splits(M, N, K, num_sms);
+  if (S == 0) return false;
+  const int BN = M <= 128 ? 128 : 64;
+  SkParams p = blank_params(M, N, K, status);
+  p.d32 = d;
+  p.ldd = ldd;
+  launch_blank(a, lda, K, b, ldb, p, S, (N + BN - 1) / BN, s);
   return true;
 }
 

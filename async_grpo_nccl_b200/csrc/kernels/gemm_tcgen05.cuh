@@ -31,6 +31,15 @@ struct GemmShape {
   // [dual_b + t * BN/2, ...): accumulator columns [0, BN/2) and [BN/2, BN) of tile t then hold the two projections of
   // the same output columns (gate and up of a SwiGLU MLP). N counts both halves (2 * dual_b).
   int dual_b = 0;
+  // > 0: two products side by side. Rows [0, n1) of B meet the first K columns of A, rows [n1, N) the K columns that start at
+  // a2; column tiles never straddle n1, and an epilogue sees as N the end of the product that its tile belongs to.
+  int n1 = 0;
+  int a2 = 0;
+
+  __host__ __device__ int tiles_n(int BN) const { return n1 > 0 ? (n1 + BN - 1) / BN + (N - n1 + BN - 1) / BN : (N + BN - 1) / BN; }
+  __device__ __forceinline__ bool second(int tn, int BN) const { return n1 > 0 && tn >= (n1 + BN - 1) / BN; }
+  __device__ __forceinline__ int first_col(int tn, int BN) const { return second(tn, BN) ? n1 + (tn - (n1 + BN - 1) / BN) * BN : tn * BN; }
+  __device__ __forceinline__ int end_col(int tn, int BN) const { return n1 > 0 && !second(tn, BN) ? n1 : N; }
 };
 
 // Default epilogue: D = alpha * acc (+ bias) (+ D), bf16 or fp32 output.
@@ -390,9 +399,9 @@ __device__ __forceinline__ void gemm_item_coords(int idx, int tiles_m, int tiles
     count = min(group_n, tiles_n - tn0);
   }
 }
-__host__ __device__ inline int gemm_num_items(int M, int N, int BN, int group_n) {
+__host__ __device__ inline int gemm_num_items(int M, int N, int BN, int group_n, int n1 = 0) {
   const int tiles_m = (M + kGemmBM - 1) / kGemmBM;
-  const int tiles_n = (N + BN - 1) / BN;
+  const int tiles_n = n1 > 0 ? (n1 + BN - 1) / BN + (N - n1 + BN - 1) / BN : (N + BN - 1) / BN;
   const int g = group_n <= 1 ? 1 : group_n;
   return tiles_m * ((tiles_n + g - 1) / g);
 }
@@ -417,8 +426,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
   const int tiles_m = (p.M + kGemmBM - 1) / kGemmBM;
-  const int tiles_n = (p.N + BN - 1) / BN;
-  const int num_items = gemm_num_items(p.M, p.N, BN, p.group_n);
+  const int tiles_n = p.tiles_n(BN);
+  const int num_items = gemm_num_items(p.M, p.N, BN, p.group_n, p.n1);
   const int num_kb = (p.K + kGemmBK - 1) / kGemmBK;
 
   if (threadIdx.x == 0) {
@@ -468,7 +477,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
         gemm_item_coords(item, tiles_m, tiles_n, p.group_n, tm, tn0, count);
         const int m0 = tm * kGemmBM;
         for (int t = 0; t < count && ok; ++t) {
-          const int n0 = (tn0 + t) * BN;
+          const int n0 = p.first_col(tn0 + t, BN);
+          const int a0 = p.second(tn0 + t, BN) ? p.a2 : 0;
           if constexpr (Gather::kEnabled) {
             if (!gj.wait_rows(n0, BN, p.N)) {
               report_status(p.status, kStatusPeerFlagTimeout);
@@ -487,7 +497,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             mbar_expect_tx(&full_bar[stage], S::kStageBytes);
             const int k0 = kb * kGemmBK;
             if constexpr (!A_MN) {
-              tma_load_2d(sa, &tmA, &full_bar[stage], k0, m0);
+              tma_load_2d(sa, &tmA, &full_bar[stage], a0 + k0, m0);
             } else {
 #pragma unroll
               for (int j = 0; j < kGemmBM / 64; ++j) tma_load_2d(sa + j * 8192, &tmA, &full_bar[stage], m0 + j * 64, k0);
@@ -569,21 +579,21 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       for (int t = 0; t < count; ++t, ++local) {
         const int buf = local & 1;
         const uint32_t acc_phase = (local >> 1) & 1;
-        epi_tile_begin(epi, row, (tn0 + t) * BN, p.M, p.N, 0);
+        const int n0 = p.first_col(tn0 + t, BN), n_end = p.end_col(tn0 + t, BN);
+        epi_tile_begin(epi, row, n0, p.M, n_end, 0);
         if (!mbar_wait(&tfull_bar[buf], acc_phase)) {
           report_status(p.status, kStatusWaitTmemFullTimeout);
           ok = false;
           break;
         }
         tc_fence_after();
-        const int n0 = (tn0 + t) * BN;
         const uint32_t taddr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + buf * BN;
 #pragma unroll 1
         for (int c = 0; c < BN / 32; ++c) {
           uint32_t r[32];
           tmem_ld_32x32(taddr + c * 32, r);
           tc_wait_ld();
-          epi.chunk(row, n0 + c * 32, r, p.M, p.N);
+          epi.chunk(row, n0 + c * 32, r, p.M, n_end);
         }
         tc_fence_before();
         __syncwarp();
@@ -608,7 +618,7 @@ inline void gemm_launch(const CUtensorMap& ta, const CUtensorMap& tb, const Gemm
   using S = GemmSmem<BN>;
   auto kernel = gemm_tcgen05_kernel<BN, A_MN, B_MN, Epi, Gather>;
   AGRPO_SET_MAX_DYN_SMEM(kernel, S::kTotal, "gemm smem attr");
-  const int items = gemm_num_items(p.M, p.N, BN, p.group_n);
+  const int items = gemm_num_items(p.M, p.N, BN, p.group_n, p.n1);
   // every CTA of the grid must be resident at once when CTAs wait on one another (copiers + workers <= SMs)
   const int n_copy = Gather::kEnabled ? gj.n_copy : 0;
   const int workers = items < num_sms - n_copy ? items : num_sms - n_copy;

@@ -73,7 +73,17 @@ struct ConvVec<float> {
 };
 
 template <typename T>
-__device__ __forceinline__ void conv_store(const ShortConvArgs& p, int t, const int4& r, int c, const float (&acc)[8]) {
+__device__ __forceinline__ void conv_store(const ShortConvArgs& p, int t, const int4& r, int c, float (&acc)[8]) {
+  if (p.bias != nullptr) {
+    float b[8];
+    ld8(reinterpret_cast<const T*>(p.bias) + c, b);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] += b[i];
+  }
+  if (p.silu) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] = acc[i] / (1.f + expf(-acc[i]));
+  }
   if (c < p.q_cols) {
     st8(reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_cols + c, acc);
     return;
@@ -324,7 +334,13 @@ constexpr int kFT = 64, kFK = 16;
 struct F32Store {
   float* d;
   long long ldd;
-  __device__ __forceinline__ void operator()(int row, int col, float v, float) const { d[(size_t)row * ldd + col] = v; }
+  GemmF32Post post;
+  __device__ __forceinline__ void operator()(int row, int col, float v, float) const {
+    float& o = d[(size_t)row * ldd + col];
+    if (post.relu2) v = v > 0.f ? v * v : 0.f;
+    if (post.softcap > 0.f) v = post.softcap * tanhf(v / post.softcap);
+    o = post.accumulate ? o + v : v;
+  }
 };
 struct F32Swiglu {
   float* d;
@@ -523,8 +539,8 @@ void launch_window_attn(bool fp32, const WindowAttnArgs& a, cudaStream_t s) {
 }
 
 void launch_gemm_f32(const float* a, long long lda, const float* b, long long ldb, float* d, long long ldd, int M, int N, int K,
-                     cudaStream_t s) {
-  run_gemm_f32<false>(a, lda, b, ldb, M, N, K, F32Store{d, ldd}, s);
+                     cudaStream_t s, const GemmF32Post& post) {
+  run_gemm_f32<false>(a, lda, b, ldb, M, N, K, F32Store{d, ldd, post}, s);
 }
 void launch_gemm_swiglu_f32(const float* a, long long lda, const float* b, long long ldb, float* d, long long ldd, int M, int F, int K,
                             cudaStream_t s) {

@@ -8,6 +8,7 @@
 #include "../launchers.h"
 #include "decode_attn.cuh"
 #include "gemm_tcgen05.cuh"
+#include "layer_ops.cuh"
 
 namespace agrpo {
 
@@ -184,13 +185,14 @@ struct LmSampleEpilogue {
   const unsigned long long* seeds;  // [rows] per-row stream id (request seed mixed with the step)
   float inv_temp;                   // 1/temperature (1 when greedy)
   int greedy;
+  float softcap;                    // > 0: logits are softcap * tanh(z / softcap)
   float* part_best;                 // [groups, rows] best perturbed value
   int* part_idx;                    // [groups, rows]
   float* part_z;                    // [groups, rows] unperturbed scaled logit at the best index
   float* part_m;                    // [groups, rows] online softmax
   float* part_s;
   // per-thread state
-  float best, best_z, m, s;
+  float best, best_z, m, s, inv_cap;
   int best_idx;
   uint32_t seed_lo, seed_hi;
 
@@ -200,6 +202,7 @@ struct LmSampleEpilogue {
     best_idx = 0;
     m = -INFINITY;
     s = 0.f;
+    inv_cap = softcap > 0.f ? __fdividef(1.f, softcap) : 0.f;
     const unsigned long long sd = row < M ? seeds[row] : 0ull;
     seed_lo = (uint32_t)sd;
     seed_hi = (uint32_t)(sd >> 32);
@@ -210,7 +213,8 @@ struct LmSampleEpilogue {
     float z[32];
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
-      z[i] = (col0 + i < N) ? __uint_as_float(r[i]) * inv_temp : -INFINITY;
+      const float raw = __uint_as_float(r[i]);
+      z[i] = (col0 + i < N) ? (softcap > 0.f ? softcap * tanh_abs_f32(raw * inv_cap) : raw) * inv_temp : -INFINITY;
       cm = fmaxf(cm, z[i]);
     }
     if (cm > m) {
@@ -220,7 +224,8 @@ struct LmSampleEpilogue {
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       s += __expf(z[i] - m);
-      float v = z[i];
+      // the cap is monotonic: the best raw logit is the best capped one, without the ties that saturation rounds to
+      float v = greedy && col0 + i < N ? __uint_as_float(r[i]) : z[i];
       if (!greedy) {
         const uint32_t h = hash_u32(hash_u32((uint32_t)(col0 + i) ^ seed_lo) + seed_hi);
         const float u = ((float)(h >> 8) + 0.5f) * (1.0f / 16777216.0f);  // (0, 1)
@@ -406,7 +411,7 @@ int lm_sample_num_groups(int V, int rows) { return lmhead_num_groups(V, rows); }
 
 void launch_lm_sample(const void* hidden, long long ldh, const void* weight, long long ldw, int rows, int H, int V,
                       float temperature, const unsigned long long* seeds, float* part_f, int* part_i, int* tokens,
-                      float* logprobs, int* status, int num_sms, cudaStream_t stream) {
+                      float* logprobs, int* status, int num_sms, cudaStream_t stream, float softcap) {
   if (rows == 0) return;
   const int groups = lmhead_num_groups(V, rows);
   const int tiles_n = (V + 255) / 256;
@@ -421,6 +426,8 @@ void launch_lm_sample(const void* hidden, long long ldh, const void* weight, lon
   e.seeds = seeds;
   e.greedy = temperature <= 0.f ? 1 : 0;
   e.inv_temp = e.greedy ? 1.f : 1.f / temperature;
+  e.softcap = softcap;
+  e.inv_cap = 0.f;
   const size_t n = (size_t)groups * rows;
   e.part_best = part_f;
   e.part_z = part_f + n;

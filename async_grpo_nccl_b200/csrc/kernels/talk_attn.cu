@@ -14,6 +14,7 @@
 #include "../common/ptx.cuh"
 #include "../common/tensormap.h"
 #include "../launchers.h"
+#include "../launchers_hybrid.h"
 #include "../launchers_layers.h"
 #include "decode_attn.cuh"
 #include "layer_ops.cuh"
@@ -1004,6 +1005,14 @@ void launch_decode_d(const TalkDecodeArgs& a, const DecPlan& d, cudaStream_t s) 
 
 }  // namespace
 
+void launch_gather_pages(const void* cache, const int* pages, int n_pages, const int* block_tables, int max_blocks, void* out, int G, int D,
+                         int num_cache_blocks, int* status, cudaStream_t s) {
+  if (n_pages == 0) return;
+  gather_keys_kernel<<<n_pages, 128, 0, s>>>((const bf16*)cache, reinterpret_cast<const int2*>(pages), block_tables, max_blocks, (bf16*)out, G, D,
+                                             num_cache_blocks, status);
+  check_cuda(cudaGetLastError(), "gather_pages");
+}
+
 bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_tiles, const int* pages, int n_pages, void* keys, void* acc,
                               cudaStream_t s) {
   if ((a.D != 64 && a.D != 128) || a.block_size != 16 || a.H % a.G != 0) return false;
@@ -1011,9 +1020,7 @@ bool launch_talk_attn_prefill(const WindowAttnArgs& a, const int* tiles, int n_t
   const size_t mix_smem = (size_t)a.G * a.H * grp8 * 4;
   if (mix_smem > 200 * 1024) return false;
   if (a.T == 0 || n_tiles == 0) return true;
-  gather_keys_kernel<<<n_pages, 128, 0, s>>>((const bf16*)a.k_cache, reinterpret_cast<const int2*>(pages), a.block_tables, a.max_blocks,
-                                             (bf16*)keys, a.G, a.D, a.num_cache_blocks, a.status);
-  check_cuda(cudaGetLastError(), "gather_keys");
+  launch_gather_pages(a.k_cache, pages, n_pages, a.block_tables, a.max_blocks, keys, a.G, a.D, a.num_cache_blocks, a.status, s);
   const int mc_max = 256 / a.D;
   const int chunks = (a.G + mc_max - 1) / mc_max;
   const CUtensorMap tq = make_tmap_2d(a.q, (uint64_t)a.H * a.D, a.T, a.ldq, 64, kPM);

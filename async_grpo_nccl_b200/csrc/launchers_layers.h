@@ -44,6 +44,8 @@ struct ShortConvArgs {
   void* k_cache;
   int q_cols, k_cols, D, block_size, num_cache_blocks, T;
   int* status;
+  const void* bias = nullptr;  // [q_cols + k_cols], optional
+  int silu = 0;                // 1: y / (1 + e^-y) of the result
 };
 void launch_short_conv(bool fp32, const ShortConvArgs& a, cudaStream_t s);
 // Writes the values that later steps need into the ring: ring_rows lists the last ring_len rows of each segment
@@ -100,8 +102,13 @@ int talk_decode_ctas_per_sm(int H, int G, int D);  // 0: shape not served
 void launch_talk_attn_decode(const TalkDecodeArgs& a, cudaStream_t s);
 
 // y = a . b^T in true fp32 (no tensor cores), every output summed over K in the same order whatever the batch.
+struct GemmF32Post {       // what happens to a result on its way out, in this order
+  int relu2 = 0;           // max(y, 0)^2
+  float softcap = 0.f;     // > 0: cap * tanh(y / cap)
+  int accumulate = 0;      // d += y
+};
 void launch_gemm_f32(const float* a, long long lda, const float* b, long long ldb, float* d, long long ldd, int M, int N, int K,
-                     cudaStream_t s);
+                     cudaStream_t s, const GemmF32Post& post = GemmF32Post());
 // d = silu(a . bg^T) * (a . bu^T), b = [bg; bu] with 2F rows
 void launch_gemm_swiglu_f32(const float* a, long long lda, const float* b, long long ldb, float* d, long long ldd, int M, int F, int K,
                             cudaStream_t s);

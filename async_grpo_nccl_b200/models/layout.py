@@ -158,6 +158,10 @@ class ParamLayout:
         hands out views with the heads as a dimension of their own; the checkpoint has them flattened)."""
         return tuple(view.shape)
 
+    def hf_unused(self, name: str) -> bool:
+        """Checkpoint tensors that a file may hold although the model has no place for them."""
+        return name == "lm_head.weight" and bool(getattr(self.cfg, "tie_word_embeddings", False))
+
     def hf_items(self, flat: torch.Tensor) -> Iterator[Tuple[str, torch.Tensor]]:
         """Yield (hf_name, tensor view) pairs in HF naming; fused matrices are split into row ranges."""
         cfg = self.cfg

@@ -11,7 +11,7 @@ import os
 from dataclasses import dataclass
 from typing import Any, Callable, Dict, Optional
 
-from . import dezelorn
+from . import dezelorn, vazatar
 from .config import PRESETS as DENSE_PRESETS
 from .config import ModelConfig
 from .layout import ParamLayout
@@ -29,23 +29,45 @@ def _listed_engine() -> Any:
     return ListedEngine
 
 
+def _dense_decoder() -> Any:
+    from .decoder import NativeDecoder
+
+    return NativeDecoder
+
+
+def _dezelorn_decoder() -> Any:
+    from .dezelorn_decoder import DezelornDecoder
+
+    return DezelornDecoder
+
+
+def _vazatar_decoder() -> Any:
+    from .vazatar_decoder import VazatarDecoder
+
+    return VazatarDecoder
+
+
 @dataclass(frozen=True)
 class Architecture:
     name: str
     config_from_dict: Callable[[Dict[str, Any]], Any]
     layout: Callable[..., ParamLayout]
     engine: Callable[[], Any]         # returns the engine class (imported on demand: it needs the extension)
+    decoder: Callable[[], Any]        # returns the executor class, likewise
     trainable: bool                   # has a backward pass (trainer role) and a dense logprob forward
     dtypes: tuple                     # parameter types that the native engine runs
 
 
 ARCHITECTURES: Dict[str, Architecture] = {
-    "dense": Architecture("dense", ModelConfig.from_dict, ParamLayout, _dense_engine, True, ("bfloat16",)),
-    "Dezelorn": Architecture("Dezelorn", dezelorn.DezelornConfig.from_dict, dezelorn.DezelornLayout, _listed_engine, False,
+    "dense": Architecture("dense", ModelConfig.from_dict, ParamLayout, _dense_engine, _dense_decoder, True, ("bfloat16",)),
+    "Dezelorn": Architecture("Dezelorn", dezelorn.DezelornConfig.from_dict, dezelorn.DezelornLayout, _listed_engine, _dezelorn_decoder, False,
                              ("bfloat16", "float32")),
+    "Vazatar": Architecture("Vazatar", vazatar.VazatarConfig.from_dict, vazatar.VazatarLayout, _listed_engine, _vazatar_decoder, False,
+                            ("bfloat16", "float32")),
 }
 
-PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **dezelorn.PRESETS}
+LISTED_PRESETS: Dict[str, Any] = {**dezelorn.PRESETS, **vazatar.PRESETS}
+PRESETS: Dict[str, Any] = {**DENSE_PRESETS, **LISTED_PRESETS}
 
 
 def architecture_of(cfg: Any) -> Architecture:
@@ -53,8 +75,8 @@ def architecture_of(cfg: Any) -> Architecture:
 
 
 def config_from_dict(d: Dict[str, Any]) -> Any:
-    if "preset" in d and d["preset"] in dezelorn.PRESETS:
-        base = dezelorn.PRESETS[d["preset"]].to_hf_dict()
+    if "preset" in d and d["preset"] in LISTED_PRESETS:
+        base = LISTED_PRESETS[d["preset"]].to_hf_dict()
         base.update({k: v for k, v in d.items() if k != "preset"})
         d = base
     name = d.get("architecture")
