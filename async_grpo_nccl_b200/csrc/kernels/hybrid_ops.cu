@@ -295,6 +295,22 @@ __global__ void __launch_bounds__(128) chunk_attn_kernel(ChunkAttnArgs p) {
 // Selective scan, thread = channel of a segment, states in shared memory, token after token.
 constexpr int kPlainChannels = 64;
 
+// exp(z) for z <= 0. A state that fades slowly multiplies by numbers just below one many times over, so what counts there is the
+// rounding of the last bit: near zero the Taylor series, whose last step (one plus a small number) is rounded once.
+__device__ __forceinline__ float decay(float z) {
+  if (z < -0.5f) return expf(z);
+  float p = 1.f / 362880.f;
+  p = fmaf(p, z, 1.f / 40320.f);
+  p = fmaf(p, z, 1.f / 5040.f);
+  p = fmaf(p, z, 1.f / 720.f);
+  p = fmaf(p, z, 1.f / 120.f);
+  p = fmaf(p, z, 1.f / 24.f);
+  p = fmaf(p, z, 1.f / 6.f);
+  p = fmaf(p, z, 0.5f);
+  p = fmaf(p, z, 1.f);
+  return fmaf(p, z, 1.f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kPlainChannels) selective_scan_plain_kernel(ScanArgs p) {
   pdl_wait();
@@ -330,7 +346,7 @@ __global__ void __launch_bounds__(kPlainChannels) selective_scan_plain_kernel(Sc
     const float in = dt * x;
     float y = 0.f;
     for (int i = 0; i < N; ++i) {
-      const float s = fmaf(expf(dt * A[i]), S[i], in * r[p.rank + i]);
+      const float s = fmaf(decay(dt * A[i]), S[i], in * r[p.rank + i]);
       S[i] = s;
       y = fmaf(s, r[p.rank + N + i], y);
     }

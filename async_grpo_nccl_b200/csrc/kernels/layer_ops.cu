@@ -383,6 +383,12 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       if constexpr (DUAL) sb2[k][r] = (kin && n0 + r < N) ? b[(size_t)(N + n0 + r) * ldb + k0 + k] : 0.f;
     }
     __syncthreads();
+    // sums of kFK products first, then the sum of those: the rounding error of a long K stays that of a short one
+    float part[4][4], part2[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) part[i][j] = part2[i][j] = 0.f;
 #pragma unroll
     for (int k = 0; k < kFK; ++k) {
       float av[4], bv[4], cv[4];
@@ -396,10 +402,17 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
-          if constexpr (DUAL) acc2[i][j] = fmaf(av[i], cv[j], acc2[i][j]);
+          part[i][j] = fmaf(av[i], bv[j], part[i][j]);
+          if constexpr (DUAL) part2[i][j] = fmaf(av[i], cv[j], part2[i][j]);
         }
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        acc[i][j] += part[i][j];
+        if constexpr (DUAL) acc2[i][j] += part2[i][j];
+      }
     __syncthreads();
   }
 #pragma unroll
