@@ -96,7 +96,8 @@ __device__ __forceinline__ void load_wdt(const ScanArgs& p, const ScanSizes& z, 
   }
 }
 
-// Tile rows [0, n) of r, x and z into a stage; x and z rows are kCh channels.
+// Tile rows [0, n) of r, x and z into a stage; x and z rows are kCh channels. Rows of r from n on become zeros: their tokens are
+// computed like the others, with a step size of zero, and must find finite numbers.
 template <int TT>
 __device__ __forceinline__ void load_tile(const ScanArgs& p, const ScanSizes& z, int row0, int n, int c0, uint8_t* stage) {
   const int per = z.r_floats / 4;
@@ -104,6 +105,8 @@ __device__ __forceinline__ void load_tile(const ScanArgs& p, const ScanSizes& z,
     const int t = i / per, k = (i % per) * 4;
     cp_async16(stage + (t * z.rpitch + k) * 4, p.r + (size_t)(row0 + t) * p.ldr + k);
   }
+  for (int i = n * per + threadIdx.x; i < TT * per; i += kScanThreads)
+    *reinterpret_cast<float4*>(stage + ((i / per) * z.rpitch + (i % per) * 4) * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
   uint8_t* sx = stage + TT * z.rpitch * 4;
   uint8_t* sz = sx + TT * kCh * 2;
   for (int i = threadIdx.x; i < n * 4; i += kScanThreads) {

@@ -697,10 +697,14 @@ class RolloutEngine:
                 # Warm up outside capture (sets function attributes, fills tensor-map caches), then put back what the
                 # warm-up step changed so that the captured step starts from the same state.
                 keep_tok, keep_gen = self.last_tokens.clone(), self.gen_index.clone()
+                keep_state = [t.clone() for t in self._slot_tensors()]
                 self._decode_forward(B, temperature, splits)
                 torch.cuda.synchronize(self.dev)
                 self.last_tokens.copy_(keep_tok)
                 self.gen_index.copy_(keep_gen)
+                for t, kept in zip(self._slot_tensors(), keep_state):
+                    t.copy_(kept)
+                del keep_state
                 g = torch.cuda.CUDAGraph()
                 # thread-local capture: the trainer / logprob threads keep allocating while this thread captures
                 with torch.cuda.graph(g, capture_error_mode="thread_local"):

@@ -16,7 +16,7 @@ out views without the padding.
 from __future__ import annotations
 
 import math
-from dataclasses import asdict, dataclass
+from dataclasses import asdict, dataclass, replace
 from typing import Any, Dict, Iterator, List, Optional, Tuple
 
 import torch
@@ -100,6 +100,10 @@ class DezelornConfig:
     @property
     def max_window(self) -> int:
         return max(l.mixer.window for l in self.layers)
+
+    def first_layers(self, n: int) -> "DezelornConfig":
+        """The same model with its first ``n`` layers (benchmarks)."""
+        return replace(self, layers=self.layers[:n])
 
     def num_parameters(self) -> int:
         n = 2 * self.vocab_size * self.width + 2 * self.width + 1

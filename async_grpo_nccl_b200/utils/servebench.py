@@ -1,8 +1,8 @@
 """Serving throughput of a listed-layer design beside the dense model of equal size, and the kernels behind it.
 
-    python bench.py --serving dezelorn-1.5b:qwen2.5-1.5b,dezelorn-7b:qwen2.5-7b
+    python bench.py --serving vazatar-1.5b:qwen2.5-1.5b,dezelorn-7b:qwen2.5-7b
 
-Random weights, synthetic prompts. Prefill: prompts of ``--serving-prompt`` tokens through the engine's own prompt step;
+Random weights, synthetic prompts; every preset with its first layers only. Prefill: prompts of ``--serving-prompt`` tokens through the engine's own prompt step;
 decode: the engine's captured decode step. Times are CUDA events on the launching stream after warm-up; kernel times are
 medians with the L2 flushed (a buffer larger than L2 is written) between iterations. One JSON line per record.
 """
@@ -42,7 +42,7 @@ def make_engine(model: str, max_seqs: int, max_len: int, n_layers: int, blocks: 
     if architecture_of(cfg).name == "dense":
         cfg = replace(cfg, num_hidden_layers=n_layers)
     else:
-        cfg = replace(cfg, layers=cfg.layers[:n_layers])
+        cfg = cfg.first_layers(n_layers)
     layout = make_layout(cfg)
     params = torch.empty(layout.total, dtype=torch.bfloat16, device="cuda")
     layout.init_random_device_(params, 0)
@@ -103,7 +103,10 @@ def bench_decode(model: str, batch: int, context: int, n_layers: int, steps: int
             "tokens_per_s": round(batch / ms * 1e3)}
 
 
-def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> List[Tuple[str, str, Callable[[], Any], float, float]]:
+Case = Tuple[str, str, Callable[[], Any], float, float]
+
+
+def dezelorn_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> List[Case]:
     """(phase / role, side, launch, FLOPs, bytes) of like kernels of one layer: ``new`` a listed-layer configuration, ``old`` the
     dense one. FLOPs count what the operation needs, not what a kernel spends (scores and one product per pair)."""
     from ..ops import native
@@ -117,7 +120,7 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
     W, F, H, G, D = new.hidden_size, new.layers[0].ff_p, m.heads, m.kv_heads, m.dim_p
     R = lambda *s: torch.randn(*s, device=dev).to(bf)
     Wr = lambda *s: (torch.randn(*s, device=dev) * 0.02).to(bf)
-    cases: List[Tuple[str, str, Callable[[], Any], float, float]] = []
+    cases: List[Case] = []
 
     def add(role: str, side: str, fn: Callable[[], Any], flops: float, nbytes: float) -> None:
         cases.append((role, side, fn, flops, nbytes))
@@ -217,19 +220,163 @@ def kernel_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> L
     return cases
 
 
+def vazatar_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> List[Case]:
+    """Like kernels of one attention layer and one scan layer against those of a dense layer. The input GEMM of a parallel block
+    stands against the dense layer's two norms, two projections and SwiGLU, its output GEMM against two projections with residual.
+    Convolution, narrow projection and scan have no counterpart."""
+    from ..models.listed import LOG2E, host_batch, split_batch
+    from ..ops import native
+    from .microbench import _tiles
+
+    C, bf, dev = native(), torch.bfloat16, "cuda"
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    la, ls = next(l for l in new.layers if l.attends), next(l for l in new.layers if not l.attends)
+    m, sc = la.mixer, ls.mixer
+    W, F, Fo, H, G, D, E = new.hidden_size, la.ff_p, old.intermediate_size, m.heads, m.kv_heads, m.dim_p, m.vdim_p
+    R = lambda *s: torch.randn(*s, device=dev).to(bf)
+    Wr = lambda *s: (torch.randn(*s, device=dev) * 0.02).to(bf)
+    Z = lambda *s: torch.empty(*s, device=dev, dtype=bf)
+    cases: List[Case] = []
+    add = lambda role, side, fn, flops, nbytes: cases.append((role, side, fn, flops, nbytes))
+    win, wout = Wr(m.u_dim + F, W), Wr(W, m.out_dim + F)
+    swin, swout = Wr(sc.u_dim + F, W), Wr(W, sc.out_dim + F)
+    wqkv, wo, wgu, wd = Wr(old.qkv_dim, W), Wr(W, H * D), Wr(2 * Fo, W), Wr(W, Fo)
+    ln, qn, kn = Wr(W), R(m.q_dim), R(m.k_dim)
+    maxlen = max(prompt, ctx) + 64
+    ang = torch.rand(maxlen, m.rot.dims // 2, device=dev)
+    cos, sin = torch.cos(ang), torch.sin(ang)
+    n_st = 4 * C.scan_states_per_lane(sc.state)
+    wx, wdt, conv, conv_b = Wr(sc.rank_p + 2 * n_st, sc.inner_p), Wr(sc.inner_p, sc.rank_p), R(sc.conv, sc.inner_p), Wr(sc.inner_p)
+    dt_b, skip = torch.full((sc.inner_p,), -4.0, device=dev), torch.ones(sc.inner_p, device=dev)
+    A = -torch.arange(1, n_st + 1, device=dev, dtype=torch.float32).expand(sc.inner_p, n_st).contiguous() * LOG2E
+    gm = lambda M, N, K: (2.0 * M * N * K, 2.0 * (M * K + N * K + M * N))
+
+    def gemms(*shapes: Tuple[int, int, int], extra: float = 0.0) -> Tuple[float, float]:
+        f, b = zip(*(gm(*s) for s in shapes))
+        return sum(f), sum(b) + extra
+
+    def pair(phase: str, M: int) -> Tuple[torch.Tensor, ...]:
+        """Input and output GEMMs of a layer; returns what the mixer cases of the phase work on."""
+        h, x, u, cat, ss = R(M, 2 * W), torch.randn(M, W, device=dev), R(M, m.u_dim), R(M, m.out_dim + F), torch.zeros(6, M, dtype=torch.int64, device=dev)
+        su, scat = R(M, sc.u_dim), R(M, sc.out_dim + F)
+        ss[0] = W << 30
+        ss[4], ss[5] = (H * m.dim) << 30, (G * m.dim) << 30
+        add(f"{phase} input projections", "new", lambda: C.gemm_parallel_proj(h, win, u, cat[:, m.out_dim:], ss[0], W, 1e-5, ss[1], ss[2], m.q_dim,
+                                                                              m.q_dim + m.k_dim, st), *gemms((M, m.u_dim + F, W), extra=2.0 * M * W))
+        add(f"{phase} scan input projections", "new", lambda: C.gemm_parallel_proj(h, swin, su, scat[:, sc.out_dim:], ss[0], W, 1e-5, None, None, 0, 0, st),
+            *gemms((M, sc.u_dim + F, W), extra=2.0 * M * W))
+        add(f"{phase} output projections", "new", lambda: C.gemm_residual(cat, wout, x, True, h[:, :W], ln, h[:, W:], ln, ss[3], st),
+            *gemms((M, W, m.out_dim + F), extra=10.0 * M * W))
+        add(f"{phase} scan output projections", "new", lambda: C.gemm_residual(scat, swout, x, True, h[:, :W], ln, h[:, W:], ln, ss[3], st),
+            *gemms((M, W, sc.out_dim + F), extra=10.0 * M * W))
+        return u, cat, ss, su, scat
+
+    # ---------------- prompts ----------------
+    n_seq, nb = T // prompt, (prompt + 15) // 16
+    u, cat, ss, su, scat = pair("prompt", T)
+    hb, xb, xb2, qkv, a, gu, act = R(T, W), R(T, W), Z(T, W), R(T, old.qkv_dim), R(T, H * D), Z(T, 2 * Fo), R(T, Fo)
+
+    def in_old():
+        C.rmsnorm_fwd(xb, ln, hb, None, 1e-6)
+        C.gemm_bf16(hb, wqkv, qkv, False, False, None, 1.0, False, st, None)
+        C.rmsnorm_fwd(xb, ln, hb, None, 1e-6)
+        C.gemm_bf16(hb, wgu, gu, False, False, None, 1.0, False, st, None)
+        C.swiglu_fwd(gu, act)
+
+    def out_old():
+        C.gemm_bf16(a, wo, xb2, False, False, None, 1.0, False, st, xb)
+        C.gemm_bf16(act, wd, xb2, False, False, None, 1.0, False, st, xb)
+    in_shapes, out_shapes = [(T, old.qkv_dim, W), (T, 2 * Fo, W)], [(T, W, H * D), (T, W, Fo)]
+    for role in ("prompt input projections", "prompt scan input projections"):
+        add(role, "old", in_old, *gemms(*in_shapes))
+    for role in ("prompt output projections", "prompt scan output projections"):
+        add(role, "old", out_old, *gemms(*out_shapes))
+    kc, vc = R(n_seq * nb, G, 16, D), R(n_seq * nb, G, 16, E)
+    tables = torch.randperm(n_seq * nb, device=dev).int().view(n_seq, nb).contiguous()
+    flat, where = host_batch([(i, 0, np.zeros(prompt, np.int32)) for i in range(n_seq)], [sc.conv], 1, [m.chunk])
+    _, sb = split_batch(torch.from_numpy(flat).to(dev), where, tables)
+    rows = sb.pages.shape[0] * 16
+    keys, values = Z(rows * G * D), Z(rows * G * E)
+    add("prompt position op", "new", lambda: C.qk_norm_rope(u, qn, kn, 1e-5, m.dim, cos, sin, ss[4], ss[5], sb.rows, None, tables, kc, vc, st), 0.0,
+        4.0 * T * (H + G) * D + 4.0 * T * G * E)
+    pos, slots, cs = torch.arange(T, device=dev, dtype=torch.int32) % prompt, torch.arange(T, device=dev, dtype=torch.int32), torch.rand(maxlen, D // 2, device=dev)
+
+    def rope():
+        C.rope_inplace(qkv, pos, cs, cs, H + G, D, False)
+        C.kv_cache_write(qkv, slots, kc, vc, H, G, D, st, 0)
+    add("prompt position op", "old", rope, 0.0, 4.0 * T * (H + G) * D + 8.0 * T * G * D)
+    pairs_n = n_seq * sum(i % m.chunk + 1 for i in range(prompt))
+    pairs_o = n_seq * prompt * (prompt + 1) / 2
+    C.qk_norm_rope(u, qn, kn, 1e-5, m.dim, cos, sin, None, None, sb.rows, None, tables, kc, vc, st)
+    add("prompt attention", "new", lambda: C.chunk_attn_prefill(u, kc, vc, sb.tiles, sb.pages, keys, values, tables, m.scale, m.softcap, m.chunk, cat[:, :m.out_dim], st),
+        2.0 * pairs_n * H * (D + E), 0.0)
+    lse, tiles = torch.empty(H, T, device=dev), _tiles([prompt] * n_seq)
+    add("prompt attention", "old", lambda: C.attn_varlen_fwd(qkv, a, lse, tiles, H, G, D, 0.1, st), 4.0 * pairs_o * H * D, 0.0)
+    n_slots = max(n_seq, B)
+    ring, state = torch.zeros(n_slots, sc.conv, sc.inner_p, device=dev, dtype=bf), torch.zeros(n_slots, sc.inner_p, n_st, device=dev)
+    xc, r = R(T, sc.inner_p), torch.randn(T, wx.shape[0], device=dev)
+    add("prompt convolution", "new", lambda: C.conv_silu(su, conv, conv_b, ring, sb.rows, sb.ring_rows[sc.conv], None, xc, st), 0.0, 4.0 * T * sc.inner_p)
+    add("prompt narrow projection", "new", lambda: C.gemm_bf16(xc, wx, r, False, False, None, 1.0, False, st, None), 0.0, 2.0 * T * sc.inner_p + 4.0 * T * wx.shape[0])
+    add("prompt scan", "new", lambda: C.selective_scan(xc, r, su[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state, sb.segs, None, scat[:, :sc.inner_p]), 0.0,
+        6.0 * T * sc.inner_p + 4.0 * T * wx.shape[0])
+
+    # ---------------- decode ----------------
+    nbd = (ctx + 15) // 16 + 1
+    dk, dv = R(B * nbd, G, 16, D), R(B * nbd, G, 16, E)
+    dtab = torch.randperm(B * nbd, device=dev).int().view(B, nbd).contiguous()
+    lens = torch.full((B,), ctx, device=dev, dtype=torch.int32)
+    du, dcat, dss, dsu, dscat = pair("decode", B)
+    xr, qb, ab, actb, hob, xs = R(B, W), R(B, old.qkv_dim), R(B, H * D), R(B, Fo), Z(B, W), R(B, W)
+    ssq, so = torch.full((B,), W << 30, device=dev, dtype=torch.int64), torch.zeros(B, device=dev, dtype=torch.int64)
+
+    def din_old():
+        C.gemm_decode(xr, wqkv, qb, None, None, ssq, None, 1e-6, st)
+        C.gemm_swiglu(xr, wgu, actb, ssq, 1e-6, st)
+
+    def dout_old():
+        C.gemm_decode(ab, wo, hob, None, xs, None, so, 1e-6, st)
+        C.gemm_decode(actb, wd, hob, None, xs, None, so, 1e-6, st)
+    for role in ("decode input projections", "decode scan input projections"):
+        add(role, "old", din_old, *gemms((B, old.qkv_dim, W), (B, 2 * Fo, W)))
+    for role in ("decode output projections", "decode scan output projections"):
+        add(role, "old", dout_old, *gemms((B, W, H * D), (B, W, Fo), extra=8.0 * B * W))
+    n_sm = torch.cuda.get_device_properties(0).multi_processor_count
+    part = (torch.empty(B * 8 * H * max(D, E) * 2, device=dev), torch.empty(B * 8 * H * 16, device=dev), torch.zeros(B * H, device=dev, dtype=torch.int32))
+    seen = (ctx - 1) % m.chunk + 1
+    sp_new = max(1, min(8, 3 * n_sm // (B * G), seen // 128))
+    sp_old = max(1, min(8, 3 * n_sm // (B * G), ctx // 256))
+    add("decode attention", "new", lambda: C.chunk_attn_decode(du, qn, kn, 1e-5, m.dim, cos, sin, dss[4], dss[5], lens, dtab, dk, dv, m.scale, m.softcap, m.chunk,
+                                                               dcat[:, :m.out_dim], sp_new, *part, st), 0.0, 2.0 * B * seen * G * (D + E))
+    add("decode attention", "old", lambda: C.paged_decode_attn(qb, dk, dv, dtab, lens, ab, H, G, D, 0.1, sp_old, part[0], part[1], st, part[2]), 0.0,
+        4.0 * B * ctx * G * D)
+    dxc, dr = R(B, sc.inner_p), torch.randn(B, wx.shape[0], device=dev)
+    add("decode convolution", "new", lambda: C.conv_silu(dsu, conv, conv_b, ring[:B], None, None, lens, dxc, st), 0.0, 2.0 * B * sc.inner_p * (sc.conv + 2))
+    add("decode narrow projection", "new", lambda: C.gemm_bf16(dxc, wx, dr, False, False, None, 1.0, False, st, None), 0.0,
+        2.0 * (B + wx.shape[0]) * sc.inner_p + 4.0 * B * wx.shape[0])
+    add("decode scan", "new", lambda: C.selective_scan(dxc, dr, dsu[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state[:B], None, lens, dscat[:, :sc.inner_p]), 0.0,
+        8.0 * B * sc.inner_p * n_st + 2.0 * sc.inner_p * sc.rank_p + 4.0 * sc.inner_p * n_st + 6.0 * B * sc.inner_p)
+    return cases
+
+
+KERNEL_CASES = {"Dezelorn": dezelorn_cases, "Vazatar": vazatar_cases}
+
+
 def bench_kernels(new_name: str, old_name: str, T: int, prompt: int, B: int, ctx: int) -> None:
     from ..models.registry import PRESETS
 
     pk = peaks()
     res: Dict[str, Dict[str, Dict[str, float]]] = {}
-    for role, side, fn, flops, nbytes in kernel_cases(PRESETS[new_name], PRESETS[old_name], T, prompt, B, ctx):
+    cases = KERNEL_CASES[PRESETS[new_name].architecture](PRESETS[new_name], PRESETS[old_name], T, prompt, B, ctx)
+    for role, side, fn, flops, nbytes in cases:
         ms = timeit(fn, iters=10, flush=True)
         bound = max(flops / (pk["bf16_tflops"] * 1e9), nbytes / (pk["hbm_gbs"] * 1e6))  # ms
         res.setdefault(role, {})[side] = {"us": round(ms * 1e3, 1), "of_roofline": round(bound / ms, 3)}
     for role, r in res.items():
-        out({"bench": "kernel", "pair": f"{new_name}:{old_name}", "shape": f"T={T} prompt={prompt}" if role.startswith("prompt") else f"B={B} ctx={ctx}",
-             "role": role, "new": r["new"], "old": r["old"], "distance_ratio": round(r["old"]["of_roofline"] / r["new"]["of_roofline"], 2),
-             "peaks": pk["source"]})
+        rec = {"bench": "kernel", "pair": f"{new_name}:{old_name}", "shape": f"T={T} prompt={prompt}" if role.startswith("prompt") else f"B={B} ctx={ctx}",
+               "role": role, **r}
+        if "old" in r:
+            rec["distance_ratio"] = round(r["old"]["of_roofline"] / max(1e-9, r["new"]["of_roofline"]), 2)
+        out({**rec, "peaks": pk["source"]})
 
 
 def run(pairs: str, prompt: int = 4096, n_layers: int = 8, kernels: bool = True) -> None:

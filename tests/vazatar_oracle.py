@@ -129,7 +129,9 @@ def feed_forward(h, w, p):
 
 def layer_order(config):
     """(layer, first of a pass of the loop) in the order they run."""
-    n, loop = len(config["layers"]), config["loop"]
+    n, loop = len(config["layers"]), config.get("loop")
+    if loop is None:
+        return [(i, False) for i in range(n)]
     order = [(i, False) for i in range(loop["start"])]
     for _ in range(loop["times"]):
         order += [(i, i == loop["start"]) for i in range(loop["start"], loop["stop"])]
