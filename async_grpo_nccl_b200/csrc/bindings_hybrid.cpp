@@ -123,8 +123,9 @@ void conv_silu(const Tensor& u, const Tensor& w, const Tensor& bias, Tensor& rin
   a.T = (int)T; a.status = iptr(status);
   a.bias = bias.data_ptr(); a.silu = 1;
   const c10::cuda::CUDAGuard guard(u.device());
+  if (!given(rows)) return agrpo::launch_short_conv_decode(f, a, cur_stream());
   agrpo::launch_short_conv(f, a, cur_stream());
-  agrpo::launch_short_conv_ring(f, a, given(rows) ? ring_rows->data_ptr<int>() : nullptr, given(rows) ? (int)ring_rows->numel() : 0, cur_stream());
+  agrpo::launch_short_conv_ring(f, a, ring_rows->data_ptr<int>(), (int)ring_rows->numel(), cur_stream());
 }
 
 agrpo::QkRopeArgs qk_args(const Tensor& u, const Tensor& qn, const Tensor& kn, double eps, int64_t dim, const Tensor& cos_t, const Tensor& sin_t,
@@ -279,17 +280,34 @@ void selective_scan_plain(const Tensor& xc, const Tensor& r, const Tensor& z, co
   agrpo::launch_selective_scan_plain(xc.scalar_type() == torch::kFloat32, a, cur_stream());
 }
 
-// Packed form (bf16): A in log2 units and the state have 4 * scan_states_per_lane(N) entries per channel.
-void selective_scan(const Tensor& xc, const Tensor& r, const Tensor& z, const Tensor& wdt, int64_t rank, const Tensor& dt_b, const Tensor& a_,
-                    const Tensor& d_, Tensor& state, const OptTensor& segs, const OptTensor& seq_lens, Tensor& out) {
+// Packed form (bf16): step-size code by itself, r = B and C by quarters; A in log2 units and the state have
+// 4 * scan_states_per_lane(N) entries per channel.
+void selective_scan(const Tensor& xc, const Tensor& code, const Tensor& r, const Tensor& z, const Tensor& wdt, int64_t rank, const Tensor& dt_b,
+                    const Tensor& a_, const Tensor& d_, Tensor& state, const OptTensor& segs, const OptTensor& seq_lens, Tensor& out) {
   TORCH_CHECK(xc.scalar_type() == torch::kBFloat16, "selective_scan: bf16");
-  const agrpo::ScanArgs a = scan_args(xc, r, z, wdt, rank, dt_b, a_, d_, state, segs, seq_lens, out);
+  agrpo::ScanArgs a = scan_args(xc, r, z, wdt, rank, dt_b, a_, d_, state, segs, seq_lens, out);
+  same_type(code, false, "code"); mat(code, "code");
   const int64_t rank_p = (rank + 15) / 16 * 16;
   TORCH_CHECK(4 * agrpo::scan_states_per_lane(a.N) == a.N && agrpo::selective_scan_serves(a.N, a.rank), "selective_scan: states");
-  TORCH_CHECK(r.size(1) == rank_p + 2 * a.N && wdt.size(1) >= rank_p && a.C % 32 == 0 && state.stride(0) % 4 == 0 && aligned16(state) && aligned16(a_),
-              "selective_scan: packed layout");
+  TORCH_CHECK(code.size(0) >= a.T && code.size(1) == rank_p && r.size(1) == 2 * a.N && wdt.size(1) >= rank_p && a.C % 32 == 0 &&
+              state.stride(0) % 4 == 0 && aligned16(state) && aligned16(a_), "selective_scan: packed layout");
+  a.code = code.data_ptr(); a.ldcode = code.stride(0);
   const c10::cuda::CUDAGuard guard(xc.device());
   TORCH_CHECK(agrpo::launch_selective_scan(a, cur_stream()), "selective_scan: shape not served");
+}
+
+void gemm_split_store(const Tensor& a_, const Tensor& w, Tensor& d16, Tensor& d32, const OptTensor& status) {
+  same_type(a_, false, "a"); same_type(w, false, "w"); same_type(d16, false, "d16"); check_f32(d32, "d32");
+  mat(a_, "a"); mat(w, "w"); mat(d16, "d16"); mat(d32, "d32");
+  agrpo::SplitStoreArgs a{};
+  a.M = (int)a_.size(0); a.K = (int)w.size(1); a.n1 = (int)d16.size(1); a.n2 = (int)d32.size(1);
+  TORCH_CHECK(a_.size(1) == a.K && a.K % 8 == 0 && a.n1 % 8 == 0 && a.n2 % 8 == 0 && w.size(0) == a.n1 + a.n2 && d16.size(0) >= a.M && d32.size(0) >= a.M,
+              "gemm_split_store: shapes");
+  a.a = a_.data_ptr(); a.lda = a_.stride(0); a.w = w.data_ptr(); a.ldw = w.stride(0);
+  a.d16 = d16.data_ptr(); a.ld16 = d16.stride(0); a.d32 = d32.data_ptr<float>(); a.ld32 = d32.stride(0);
+  a.status = iptr(status);
+  const c10::cuda::CUDAGuard guard(a_.device());
+  agrpo::launch_gemm_split_store(a, sms(), cur_stream());
 }
 
 void gemm_parallel_proj(const Tensor& h, const Tensor& w, Tensor& u, const OptTensor& act, const OptTensor& ss_in, int64_t width, double eps,
@@ -360,7 +378,8 @@ void bind_hybrid_ops(pybind11::module_& m) {
   m.def("selective_scan_serves", &agrpo::selective_scan_serves);
   m.def("selective_scan_plain", &selective_scan_plain, py::arg("xc"), py::arg("r"), py::arg("z"), py::arg("wdt"), py::arg("rank"), py::arg("dt_b"),
         py::arg("a"), py::arg("d"), py::arg("state"), py::arg("segs"), py::arg("seq_lens"), py::arg("out"), NoGil());
-  m.def("selective_scan", &selective_scan, py::arg("xc"), py::arg("r"), py::arg("z"), py::arg("wdt"), py::arg("rank"), py::arg("dt_b"), py::arg("a"),
+  m.def("gemm_split_store", &gemm_split_store, py::arg("a"), py::arg("w"), py::arg("d16"), py::arg("d32"), py::arg("status"), NoGil());
+  m.def("selective_scan", &selective_scan, py::arg("xc"), py::arg("code"), py::arg("r"), py::arg("z"), py::arg("wdt"), py::arg("rank"), py::arg("dt_b"), py::arg("a"),
         py::arg("d"), py::arg("state"), py::arg("segs"), py::arg("seq_lens"), py::arg("out"), NoGil());
   m.def("gemm_parallel_proj", &gemm_parallel_proj, py::arg("h"), py::arg("w"), py::arg("u"), py::arg("act"), py::arg("ss_in"), py::arg("width"),
         py::arg("eps"), py::arg("ss_q"), py::arg("ss_k"), py::arg("q_end"), py::arg("k_end"), py::arg("status"), NoGil());

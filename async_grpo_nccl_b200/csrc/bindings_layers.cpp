@@ -85,9 +85,9 @@ void short_conv(const Tensor& u, const Tensor& w, Tensor& ring, const OptTensor&
   const bool f = u.scalar_type() == torch::kFloat32;
   if (given(rows)) { TORCH_CHECK(given(ring_rows) && ring_rows->is_contiguous(), "short_conv: ring_rows with rows"); check_i32(*ring_rows, "ring_rows"); }
   const c10::cuda::CUDAGuard guard(u.device());
+  if (!given(rows)) return agrpo::launch_short_conv_decode(f, a, cur_stream());
   agrpo::launch_short_conv(f, a, cur_stream());
-  agrpo::launch_short_conv_ring(f, a, given(rows) ? ring_rows->data_ptr<int>() : nullptr,
-                                given(rows) ? (int)ring_rows->numel() : 0, cur_stream());
+  agrpo::launch_short_conv_ring(f, a, ring_rows->data_ptr<int>(), (int)ring_rows->numel(), cur_stream());
 }
 
 agrpo::WindowAttnArgs attn_args(const OptTensor& q, const Tensor& k_cache, const OptTensor& rows, const OptTensor& seq_lens,

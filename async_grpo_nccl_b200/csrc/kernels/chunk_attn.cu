@@ -81,7 +81,8 @@ struct ChunkPrefillParams {
 
 // 32 raw scores -> weights (not normalised); adds them to l. Small arguments of tanh (the usual case) take the odd series up to
 // z^9, two at a time; if any score of the warp is larger, all take the exponential form.
-__device__ __forceinline__ void free_weights(const uint32_t (&s)[32], const CapScale& sc, bool masked, int lo, int hi, uint32_t (&w)[16], float& l) {
+template <bool MASKED>
+__device__ __forceinline__ void free_weights(const uint32_t (&s)[32], const CapScale& sc, int lo, int hi, uint32_t (&w)[16], float& l) {
   float mx[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
   for (int i = 0; i < 32; ++i) mx[i & 3] = fmaxf(mx[i & 3], fabsf(__uint_as_float(s[i])));
@@ -100,7 +101,7 @@ __device__ __forceinline__ void free_weights(const uint32_t (&s)[32], const CapS
       unpack2(e, a, b);
       a = ex2(a);
       b = ex2(b);
-      if (masked) {
+      if (MASKED) {
         if (2 * i < lo || 2 * i > hi) a = 0.f;
         if (2 * i + 1 < lo || 2 * i + 1 > hi) b = 0.f;
       }
@@ -113,7 +114,7 @@ __device__ __forceinline__ void free_weights(const uint32_t (&s)[32], const CapS
     for (int i = 0; i < 16; ++i) {
       float a = ex2(sc.out * tanh_abs_f32(__uint_as_float(s[2 * i]) * sc.in));
       float b = ex2(sc.out * tanh_abs_f32(__uint_as_float(s[2 * i + 1]) * sc.in));
-      if (masked) {
+      if (MASKED) {
         if (2 * i < lo || 2 * i > hi) a = 0.f;
         if (2 * i + 1 < lo || 2 * i + 1 > hi) b = 0.f;
       }
@@ -264,7 +265,8 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         for (int c = 0; c < kBN / 32; ++c) {
           if (c + 1 < kBN / 32) tmem_ld_32x32(tmem_S + lane_off + (c + 1) * 32, s[(c + 1) & 1]);
           uint32_t w[16];
-          free_weights(s[c & 1], p.sc, masked, lo - c * 32, hi - c * 32, w, l);
+          if (masked) free_weights<true>(s[c & 1], p.sc, lo - c * 32, hi - c * 32, w, l);
+          else free_weights<false>(s[c & 1], p.sc, 0, 0, w, l);
           tc_wait_ld();
           tmem_st_32x16(tmem_S + lane_off + c * 16, w);
         }
@@ -410,7 +412,7 @@ __device__ __forceinline__ void norm_rotate(const QkRopeArgs& p, const bf16* src
 }
 
 template <int D, int E, int ROWS>
-__global__ void __launch_bounds__(kWarps * 32) chunk_decode_kernel(const ChunkDecodeArgs a, const CapScale sc) {
+__global__ void __launch_bounds__(kWarps * 32, 3) chunk_decode_kernel(const ChunkDecodeArgs a, const CapScale sc) {
   constexpr int kTile = kPage * (D + E) * 2;
   constexpr int kQPitch = D + 8;
   extern __shared__ __align__(128) uint8_t cd_smem[];

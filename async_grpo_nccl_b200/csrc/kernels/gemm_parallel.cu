@@ -73,6 +73,25 @@ struct ResidualEpilogue {
   }
 };
 
+struct SplitEpilogue {
+  SplitOut o;
+
+  __device__ __forceinline__ void item_begin(int, int, int) {}
+  __device__ __forceinline__ void chunk(int row, int col0, const uint32_t (&r)[32], int M, int N) {
+    if (row >= M) return;
+#pragma unroll
+    for (int c = 0; c < 32; c += 8) {
+      if (col0 + c < N) {
+        float v[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(r[c + i]);
+        o.store8(row, col0 + c, v);
+      }
+    }
+  }
+  __device__ __forceinline__ void item_end(int, int, int, int) {}
+};
+
 template <class Epi>
 void launch_tiles(const void* a, long long lda, int a_cols, const void* b, long long ldb, const GemmShape& p, const Epi& e, int BN, int num_sms,
                   cudaStream_t s) {
@@ -123,6 +142,17 @@ void launch_gemm_residual(const ResidualArgs& a, int num_sms, cudaStream_t s) {
   e.sq = 0.f;
   e.bn = pick_bn(p);
   launch_tiles(a.a, a.lda, a.K, a.w, a.ldw, p, e, e.bn, num_sms, s);
+}
+
+void launch_gemm_split_store(const SplitStoreArgs& a, int num_sms, cudaStream_t s) {
+  if (a.M == 0) return;
+  const SplitOut out = split_out(a);
+  if (launch_gemm_skinny_split(a, out, num_sms, s)) return;
+  GemmShape p;
+  p.M = a.M; p.N = a.n1 + a.n2; p.K = a.K;
+  p.group_n = 1;
+  p.status = a.status;
+  launch_tiles(a.a, a.lda, a.K, a.w, a.ldw, p, SplitEpilogue{out}, pick_bn(p), num_sms, s);
 }
 
 }  // namespace agrpo

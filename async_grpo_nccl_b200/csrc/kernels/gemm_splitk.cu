@@ -66,7 +66,7 @@ struct SkParams {
   ProjOut proj;          // proj.u != nullptr: both projections of a parallel block (columns [n1, N) read A at column a2)
   ResidualOut resid;     // resid.x != nullptr: fp32 residual stream and its consumers
   int n1, a2;
-  float* d32;            // fp32 result instead of D
+  SplitOut split;        // split.d16 != nullptr: leading columns as bf16, the others as fp32
   __nv_bfloat16* D;
   long long ldd;
   const __nv_bfloat16* bias;
@@ -448,9 +448,8 @@ gemm_splitk_cluster_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
               p.resid.store8(row, col, x0, acc, sq);
               continue;
             }
-            if (p.d32 != nullptr) {
-              for (int i = 0; i < 8; ++i)
-                if (col + i < p.N) p.d32[(long long)row * p.ldd + col + i] = acc[i];
+            if (p.split.d16 != nullptr) {
+              p.split.store8(row, col, acc);
               continue;
             }
             if (p.tail.x != nullptr) {  // N is a multiple of 8 in this mode
@@ -572,7 +571,7 @@ bool launch_gemm_skinny(const void* a, long long lda, const void* b, long long l
   p.proj = ProjOut{};
   p.resid = ResidualOut{};
   p.n1 = p.a2 = 0;
-  p.d32 = nullptr;
+  p.split = SplitOut{};
   if (tail != nullptr) {
     typedef const __nv_bfloat16* P;
     p.tail.x = tail->x;
@@ -642,16 +641,13 @@ bool launch_gemm_skinny_residual(const ResidualArgs& a, const ResidualOut& out, 
   return true;
 }
 
-// fp32 result of a plain product (e.g. the narrow projection of a scan's input)
-bool launch_gemm_skinny_f32out(const void* a, long long lda, const void* b, long long ldb, float* d, long long ldd, int M, int N, int K, int* status,
-                               int num_sms, cudaStream_t s) {
-  const int S = gemm_skinny_splits(M, N, K, num_sms);
+bool launch_gemm_skinny_split(const SplitStoreArgs& a, const SplitOut& out, int num_sms, cudaStream_t s) {
+  const int S = gemm_skinny_splits(a.M, a.n1 + a.n2, a.K, num_sms);
   if (S == 0) return false;
-  const int BN = M <= 128 ? 128 : 64;
-  SkParams p = blank_params(M, N, K, status);
-  p.d32 = d;
-  p.ldd = ldd;
-  launch_blank(a, lda, K, b, ldb, p, S, (N + BN - 1) / BN, s);
+  const int BN = a.M <= 128 ? 128 : 64;
+  SkParams p = blank_params(a.M, a.n1 + a.n2, a.K, a.status);
+  p.split = out;
+  launch_blank(a.a, a.lda, a.K, a.w, a.ldw, p, S, (a.n1 + a.n2 + BN - 1) / BN, s);
   return true;
 }
 

@@ -88,9 +88,6 @@ void launch_gemm_bf16(const void* a, long long lda, const void* b, long long ldb
   if (!a_mn && !b_mn && !out_fp32 && !accumulate && alpha == 1.f && M <= 256 &&
       launch_gemm_skinny(a, lda, b, ldb, d, ldd, M, N, K, bias, residual, ldr, status, num_sms, stream))
     return;
-  if (!a_mn && !b_mn && out_fp32 && !accumulate && alpha == 1.f && M <= 256 && N <= 1024 && bias == nullptr && residual == nullptr &&
-      launch_gemm_skinny_f32out(a, lda, b, ldb, reinterpret_cast<float*>(d), ldd, M, N, K, status, num_sms, stream))
-    return;
   launch_gemm_impl(a, lda, b, ldb, d, ldd, M, N, K, a_mn, b_mn, bias, alpha, out_fp32, accumulate, status, num_sms,
                    stream, residual, ldr, NoGather{0});
 }

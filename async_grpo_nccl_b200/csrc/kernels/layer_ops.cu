@@ -82,7 +82,7 @@ __device__ __forceinline__ void conv_store(const ShortConvArgs& p, int t, const 
   }
   if (p.silu) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i] = acc[i] / (1.f + expf(-acc[i]));
+    for (int i = 0; i < 8; ++i) acc[i] = sizeof(T) == 4 ? acc[i] / (1.f + expf(-acc[i])) : acc[i] * sigmoid_f32(acc[i]);
   }
   if (c < p.q_cols) {
     st8(reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_cols + c, acc);
@@ -159,6 +159,38 @@ __global__ void __launch_bounds__(128) short_conv_kernel(ShortConvArgs p) {
     }
   }
   for (int r = 0; r < n; ++r) conv_row<T>(p, map, t0 + r, c, C);
+}
+
+// Decode rows (row = slot), thread = 8 channels of one row: convolution and ring in one pass. The ring has room for `taps` values,
+// so the new one takes the place of one that no tap reads any more.
+template <typename T>
+__global__ void __launch_bounds__(128) short_conv_decode_kernel(ShortConvArgs p) {
+  pdl_wait();
+  pdl_launch();
+  const int C = p.q_cols + p.k_cols;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8, t = blockIdx.x;
+  const int pos = p.seq_lens[t] - 1;
+  if (c >= C || pos < 0) return;
+  const T* w = reinterpret_cast<const T*>(p.w) + c;
+  T* ring = reinterpret_cast<T*>(p.ring) + (size_t)t * p.ring_pitch + c;
+  float v[8], acc[8], x[8];
+  ld8(reinterpret_cast<const T*>(p.u) + (size_t)t * p.ldu + c, v);
+  ld8(w + (size_t)(p.taps - 1) * C, x);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+#pragma unroll 4
+  for (int back = p.taps - 1; back > 0; --back) {  // oldest first
+    if (pos - back < 0) continue;
+    float y[8], xw[8];
+    ld8(ring + (size_t)((pos - back) % p.ring_len) * C, y);
+    ld8(w + (size_t)(p.taps - 1 - back) * C, xw);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] = fmaf(xw[i], y[i], acc[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = fmaf(x[i], v[i], acc[i]);
+  if (p.taps > 1) st8(ring + (size_t)(pos % p.ring_len) * C, v);
+  conv_store<T>(p, t, make_int4(t, pos, t, 0), c, acc);
 }
 
 // ring_rows: the rows whose values later steps need (the last ring_len of each segment); decode: every row
@@ -530,6 +562,13 @@ void short_conv_t(const ShortConvArgs& a, cudaStream_t s) {
   launch_kernel(kernel, grid, block, 0, s, "short_conv", a);
 }
 }  // namespace
+
+void launch_short_conv_decode(bool fp32, const ShortConvArgs& a, cudaStream_t s) {
+  if (a.T == 0) return;
+  if (a.ring_len < a.taps) throw std::runtime_error("short_conv: ring shorter than the taps");
+  const dim3 grid(a.T, ((a.q_cols + a.k_cols) / 8 + 127) / 128), block(128);
+  launch_kernel(fp32 ? short_conv_decode_kernel<float> : short_conv_decode_kernel<bf16>, grid, block, 0, s, "short_conv_decode", a);
+}
 
 void launch_short_conv(bool fp32, const ShortConvArgs& a, cudaStream_t s) {
   if (a.T == 0) return;

@@ -125,8 +125,25 @@ inline ResidualOut residual_out(const ResidualArgs& a) {
   return o;
 }
 
+// First n1 columns as bf16, the others as fp32; see SplitStoreArgs.
+struct SplitOut {
+  __nv_bfloat16* d16;   // nullptr = off
+  long long ld16;
+  float* d32;
+  long long ld32;
+  int n1;
+  __device__ __forceinline__ void store8(int row, int col, const float (&v)[8]) const {
+    if (col < n1) st8(d16 + (size_t)row * ld16 + col, v);
+    else st8(d32 + (size_t)row * ld32 + (col - n1), v);
+  }
+};
+inline SplitOut split_out(const SplitStoreArgs& a) {
+  return SplitOut{reinterpret_cast<__nv_bfloat16*>(a.d16), a.ld16, a.d32, a.ld32, a.n1};
+}
+
 // Split-K forms (gemm_splitk.cu) for up to 256 rows; false when the shape is not served.
 bool launch_gemm_skinny_proj(const ParallelProjArgs& a, const ProjOut& out, int num_sms, cudaStream_t s);
+bool launch_gemm_skinny_split(const SplitStoreArgs& a, const SplitOut& out, int num_sms, cudaStream_t s);
 bool launch_gemm_skinny_residual(const ResidualArgs& a, const ResidualOut& out, int num_sms, cudaStream_t s);
 
 }  // namespace agrpo

@@ -7,8 +7,8 @@
 // block's rows of W_dt, done by mma.sync in place, so that they never exist in memory (they would be as large as the input in
 // fp32). Read-outs of four tokens are summed over the four lanes at once: three shuffles, after which each lane finishes one.
 //
-// Layout of r [T, ldr] fp32: step-size code (rank_p columns, a multiple of 16), then for each quarter q of the states NS values
-// of B and NS values of C. A in log2 units, [C, 4 NS]; state [slots, C, 4 NS].
+// The projection of the input arrives as the step-size code, bf16 [T, rank_p] (rank_p a multiple of 16), and B and C, fp32
+// [T, 8 NS]: for each quarter of the states NS values of B, then NS of C. A in log2 units [C, 4 NS]; state [slots, C, 4 NS].
 #include <cuda_bf16.h>
 
 #include "../common/ptx.cuh"
@@ -50,116 +50,148 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
 }
 
 // ln(1 + e^v) = max(v, 0) + ln(1 + e) with e = exp(-|v|) <= 1, and ln(1 + e) = 2 artanh(e / (2 + e)): the argument is at most 1/3,
-// where the odd series converges by 1/9 a term (the first one left out is below 1e-9 of the sum).
-__device__ __forceinline__ float softplus_f32(float v) {
-  const float e = __expf(-fabsf(v));
-  const float s = __fdividef(e, 2.f + e);
-  const float q = s * s;
-  float p = 1.f / 17.f;
-  p = fmaf(p, q, 1.f / 15.f);
-  p = fmaf(p, q, 1.f / 13.f);
-  p = fmaf(p, q, 1.f / 11.f);
-  p = fmaf(p, q, 1.f / 9.f);
-  p = fmaf(p, q, 1.f / 7.f);
-  p = fmaf(p, q, 1.f / 5.f);
-  p = fmaf(p, q, 1.f / 3.f);
-  p = fmaf(p, q, 1.f);
-  return fmaxf(v, 0.f) + 2.f * s * p;
+// where the odd series converges by 1/9 a term (the first one left out is below 1e-9 of the sum). Two at a time.
+__device__ __forceinline__ void softplus_pair(float v0, float v1, float& r0, float& r1) {
+  const float e0 = __expf(-fabsf(v0)), e1 = __expf(-fabsf(v1));
+  const f32x2 s = pack2(__fdividef(e0, 2.f + e0), __fdividef(e1, 2.f + e1));
+  const f32x2 q = mul2(s, s);
+  f32x2 p = pack2(1.f / 17.f, 1.f / 17.f);
+  p = fma2(p, q, pack2(1.f / 15.f, 1.f / 15.f));
+  p = fma2(p, q, pack2(1.f / 13.f, 1.f / 13.f));
+  p = fma2(p, q, pack2(1.f / 11.f, 1.f / 11.f));
+  p = fma2(p, q, pack2(1.f / 9.f, 1.f / 9.f));
+  p = fma2(p, q, pack2(1.f / 7.f, 1.f / 7.f));
+  p = fma2(p, q, pack2(1.f / 5.f, 1.f / 5.f));
+  p = fma2(p, q, pack2(1.f / 3.f, 1.f / 3.f));
+  p = fma2(p, q, pack2(1.f, 1.f));
+  p = fma2(mul2(s, pack2(2.f, 2.f)), p, pack2(fmaxf(v0, 0.f), fmaxf(v1, 0.f)));
+  unpack2(p, r0, r1);
 }
 
 struct ScanSizes {
-  int rank_p, wpitch, rpitch;   // bf16 elements / floats per row in shared memory
-  int r_floats;                 // columns of r
+  int rank_p, cpitch;     // step-size code: columns, bf16 elements per row in shared memory (also of W_dt's rows)
+  int bc, bpitch;         // B and C: columns, floats per row
 };
 __host__ __device__ inline ScanSizes scan_sizes(int rank, int ns) {
   ScanSizes z;
   z.rank_p = (rank + 15) / 16 * 16;
-  z.r_floats = z.rank_p + 8 * ns;
-  z.wpitch = z.rank_p + 8;
-  z.rpitch = z.r_floats;
-  while (z.rpitch % 32 != 8) z.rpitch += 4;   // rows of a fragment fall into different banks
+  z.cpitch = z.rank_p + 8;   // rows of a fragment fall into different banks
+  z.bc = 8 * ns;
+  z.bpitch = z.bc;
   return z;
 }
-// stage: r tile, x tile, z tile; then W_dt rows, {dt, dt x} pairs
-__host__ __device__ inline int scan_stage_bytes(const ScanSizes& z, int tt) { return tt * z.rpitch * 4 + 2 * tt * kCh * 2; }
+// A stage holds tt tokens: code, B and C, x, z (kCh channels each)
+__host__ __device__ inline int scan_stage_bytes(const ScanSizes& z, int tt) { return tt * (z.cpitch * 2 + z.bpitch * 4 + 2 * kCh * 2); }
 inline int scan_smem_bytes(const ScanSizes& z, int tt, int stages) {
-  return stages * scan_stage_bytes(z, tt) + kCh * z.wpitch * 2 + tt * kCh * 8;
+  return stages * scan_stage_bytes(z, tt) + kCh * z.cpitch * 2 + tt * kCh * 8;
 }
+template <int TT>
+struct Stage {
+  bf16* code;
+  float* bc;
+  bf16* x;
+  bf16* z;
+  __device__ __forceinline__ Stage(uint8_t* base, const ScanSizes& s)
+      : code(reinterpret_cast<bf16*>(base)), bc(reinterpret_cast<float*>(base + TT * s.cpitch * 2)),
+        x(reinterpret_cast<bf16*>(base + TT * (s.cpitch * 2 + s.bpitch * 4))), z(x + TT * kCh) {}
+};
 
 __device__ __forceinline__ void load_wdt(const ScanArgs& p, const ScanSizes& z, int c0, bf16* sw) {
-  const int per = z.rank_p / 8;
-  for (int i = threadIdx.x; i < kCh * per; i += kScanThreads) {
-    const int c = i / per, k = (i % per) * 8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (c0 + c < p.C) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.wdt) + (size_t)(c0 + c) * p.ldw + k);
-    *reinterpret_cast<uint4*>(sw + c * z.wpitch + k) = v;
-  }
+  for (int c = threadIdx.x >> 5; c < kCh; c += 4)
+    for (int k = (threadIdx.x & 31) * 8; k < z.rank_p; k += 256) {
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (c0 + c < p.C) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.wdt) + (size_t)(c0 + c) * p.ldw + k);
+      *reinterpret_cast<uint4*>(sw + c * z.cpitch + k) = v;
+    }
 }
 
-// Tile rows [0, n) of r, x and z into a stage; x and z rows are kCh channels. Rows of r from n on become zeros: their tokens are
-// computed like the others, with a step size of zero, and must find finite numbers.
+// Tile rows [0, n) into a stage. Rows of the code, B and C from n on become zeros: their tokens are computed like the others, with a
+// step size of zero, and must find finite numbers.
 template <int TT>
-__device__ __forceinline__ void load_tile(const ScanArgs& p, const ScanSizes& z, int row0, int n, int c0, uint8_t* stage) {
-  const int per = z.r_floats / 4;
-  for (int i = threadIdx.x; i < n * per; i += kScanThreads) {
-    const int t = i / per, k = (i % per) * 4;
-    cp_async16(stage + (t * z.rpitch + k) * 4, p.r + (size_t)(row0 + t) * p.ldr + k);
+__device__ __forceinline__ void load_tile(const ScanArgs& p, const ScanSizes& z, int row0, int n, int c0, const Stage<TT>& st) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bf16* code = reinterpret_cast<const bf16*>(p.code);
+  for (int t = warp; t < TT; t += 4) {
+    const size_t row = row0 + t;
+    if (t < n) {
+      for (int k = lane * 8; k < z.rank_p; k += 256) cp_async16(st.code + t * z.cpitch + k, code + row * p.ldcode + k);
+      for (int k = lane * 4; k < z.bc; k += 128) cp_async16(st.bc + t * z.bpitch + k, p.r + row * p.ldr + k);
+    } else {
+      for (int k = lane * 8; k < z.rank_p; k += 256) *reinterpret_cast<uint4*>(st.code + t * z.cpitch + k) = make_uint4(0u, 0u, 0u, 0u);
+      for (int k = lane * 4; k < z.bc; k += 128) *reinterpret_cast<uint4*>(st.bc + t * z.bpitch + k) = make_uint4(0u, 0u, 0u, 0u);
+    }
   }
-  for (int i = n * per + threadIdx.x; i < TT * per; i += kScanThreads)
-    *reinterpret_cast<float4*>(stage + ((i / per) * z.rpitch + (i % per) * 4) * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
-  uint8_t* sx = stage + TT * z.rpitch * 4;
-  uint8_t* sz = sx + TT * kCh * 2;
   for (int i = threadIdx.x; i < n * 4; i += kScanThreads) {
     const int t = i >> 2, k = (i & 3) * 8;
     if (c0 + k < p.C) {
-      cp_async16(sx + (t * kCh + k) * 2, reinterpret_cast<const bf16*>(p.xc) + (size_t)(row0 + t) * p.ldx + c0 + k);
-      cp_async16(sz + (t * kCh + k) * 2, reinterpret_cast<const bf16*>(p.z) + (size_t)(row0 + t) * p.ldz + c0 + k);
+      cp_async16(st.x + t * kCh + k, reinterpret_cast<const bf16*>(p.xc) + (size_t)(row0 + t) * p.ldx + c0 + k);
+      cp_async16(st.z + t * kCh + k, reinterpret_cast<const bf16*>(p.z) + (size_t)(row0 + t) * p.ldz + c0 + k);
     }
   }
 }
 
 // {dt, dt x} of TT tokens x 32 channels; tokens from n on get zeros, which leave a state as it is. Warp = 8 channels.
 template <int TT>
-__device__ __forceinline__ void step_sizes(const ScanSizes& z, const float* sr, const bf16* sx, const bf16* sw, const float (&bias)[2], int n, float2* sdt) {
+__device__ __forceinline__ void step_sizes(const ScanSizes& z, const Stage<TT>& st, const bf16* sw, const float (&bias)[2], int n, float2* sdt) {
+  constexpr int M = TT / 16;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, q2 = (lane & 3) * 2;
-  const bf16* wrow = sw + (warp * 8 + g) * z.wpitch;
+  float acc[M][4];
 #pragma unroll
-  for (int m = 0; m < TT / 16; ++m) {
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    const float* r0 = sr + (m * 16 + g) * z.rpitch;
-    const float* r1 = r0 + 8 * z.rpitch;
-    for (int k = 0; k < z.rank_p; k += 16) {
-      const float2 a0 = *reinterpret_cast<const float2*>(r0 + k + q2), a1 = *reinterpret_cast<const float2*>(r1 + k + q2);
-      const float2 a2 = *reinterpret_cast<const float2*>(r0 + k + q2 + 8), a3 = *reinterpret_cast<const float2*>(r1 + k + q2 + 8);
-      mma_16816(acc, pack_bf16x2(a0.x, a0.y), pack_bf16x2(a1.x, a1.y), pack_bf16x2(a2.x, a2.y), pack_bf16x2(a3.x, a3.y),
-                *reinterpret_cast<const uint32_t*>(wrow + k + q2), *reinterpret_cast<const uint32_t*>(wrow + k + q2 + 8));
-    }
+  for (int m = 0; m < M; ++m)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int t = m * 16 + g + (e >> 1) * 8, c = warp * 8 + q2 + (e & 1);
-      float2 o = make_float2(0.f, 0.f);
-      if (t < n) {
-        o.x = softplus_f32(acc[e] + bias[e & 1]);
-        o.y = o.x * __bfloat162float(sx[t * kCh + c]);
-      }
-      sdt[t * kCh + c] = o;
+    for (int e = 0; e < 4; ++e) acc[m][e] = 0.f;
+  const bf16* arow = st.code + (lane & 15) * z.cpitch + (lane >> 4) * 8;
+  const bf16* wrow = sw + (warp * 8 + g) * z.cpitch + q2;
+  for (int k = 0; k < z.rank_p; k += 16) {
+    const uint32_t b0 = *reinterpret_cast<const uint32_t*>(wrow + k), b1 = *reinterpret_cast<const uint32_t*>(wrow + k + 8);
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+      uint32_t a[4];
+      ldmatrix_x4(a, arow + m * 16 * z.cpitch + k);
+      mma_16816(acc[m], a[0], a[1], a[2], a[3], b0, b1);
     }
   }
+#pragma unroll
+  for (int m = 0; m < M; ++m)
+#pragma unroll
+    for (int e = 0; e < 4; e += 2) {
+      const int t = m * 16 + g + (e >> 1) * 8, c = warp * 8 + q2;
+      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (t < n) {
+        const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(st.x + t * kCh + c));
+        softplus_pair(acc[m][e] + bias[0], acc[m][e + 1] + bias[1], o.x, o.z);
+        o.y = o.x * x.x;
+        o.w = o.z * x.y;
+      }
+      *reinterpret_cast<float4*>(sdt + t * kCh + c) = o;
+    }
 }
 
 // One token of one channel quarter: S <- exp2(dt A) S + (dt x) B, returns this quarter's part of S . C.
 template <int NS>
 __device__ __forceinline__ float scan_step(const float2 d, const float* bc, const f32x2 (&A)[NS / 2], f32x2 (&S)[NS / 2]) {
   const f32x2 dt = pack2(d.x, d.x), dx = pack2(d.y, d.y);
+  f32x2 B[NS / 2], C[NS / 2];
+  if constexpr (NS >= 4) {
+#pragma unroll
+    for (int i = 0; i < NS / 4; ++i) {
+      const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(bc + 4 * i), c = *reinterpret_cast<const ulonglong2*>(bc + NS + 4 * i);
+      B[2 * i] = b.x; B[2 * i + 1] = b.y;
+      C[2 * i] = c.x; C[2 * i + 1] = c.y;
+    }
+  } else {
+    const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(bc);
+    B[0] = v.x;
+    C[0] = v.y;
+  }
   f32x2 y = 0;  // bits of {0.f, 0.f}
 #pragma unroll
   for (int i = 0; i < NS / 2; ++i) {
     float a, b;
     unpack2(mul2(dt, A[i]), a, b);
-    const f32x2 B = *reinterpret_cast<const f32x2*>(bc + 2 * i), C = *reinterpret_cast<const f32x2*>(bc + NS + 2 * i);
-    S[i] = fma2(pack2(ex2(a), ex2(b)), S[i], mul2(dx, B));
-    y = fma2(S[i], C, y);
+    S[i] = fma2(pack2(ex2(a), ex2(b)), S[i], mul2(dx, B[i]));
+    y = i == 0 ? mul2(S[i], C[i]) : fma2(S[i], C[i], y);
   }
   float a, b;
   unpack2(y, a, b);
@@ -175,12 +207,43 @@ __device__ __forceinline__ float quad_transpose_sum(const float (&y)[4], int q) 
   return (high ? b : a) + __shfl_xor_sync(0xffffffffu, high ? a : b, 2);
 }
 
+// Finished read-outs of a tile (in sdt[t][c].x) -> skip, gate, store: thread = 8 channels of a token.
+template <int TT>
+__device__ __forceinline__ void store_tile(const ScanArgs& p, const Stage<TT>& st, const float2* sdt, const float* sskip, size_t row0, int n, int c0,
+                                           const int* s_pos) {
+  for (int i = threadIdx.x; i < n * 4; i += kScanThreads) {
+    const int t = i >> 2, k = (i & 3) * 8;
+    if (c0 + k >= p.C || (s_pos != nullptr && s_pos[t] < 0)) continue;
+    float x[8], z[8], o[8];
+    ld8(st.x + t * kCh + k, x);
+    ld8(st.z + t * kCh + k, z);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float y = fmaf(sskip[k + e], x[e], sdt[t * kCh + k + e].x);
+      o[e] = y * z[e] * sigmoid_f32(z[e]);
+    }
+    st8(reinterpret_cast<bf16*>(p.out) + (row0 + t) * p.ldo + c0 + k, o);
+  }
+}
+
+// Per-thread constants of a CTA's channel block.
+__device__ __forceinline__ void load_channels(const ScanArgs& p, int c0, float (&bias)[2], float* sskip) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int cb = c0 + warp * 8 + (lane & 3) * 2 + i;
+    bias[i] = cb < p.C ? p.dt_b[cb] : 0.f;
+  }
+  if (threadIdx.x < kCh) sskip[threadIdx.x] = c0 + threadIdx.x < p.C ? p.d[c0 + threadIdx.x] : 0.f;
+}
+
 template <int NS, int TT>
 __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const ScanArgs p, const ScanSizes z) {
   extern __shared__ __align__(16) uint8_t ss_smem[];
+  __shared__ float sskip[kCh];
   const int stage_bytes = scan_stage_bytes(z, TT);
   bf16* sw = reinterpret_cast<bf16*>(ss_smem + 2 * stage_bytes);
-  float2* sdt = reinterpret_cast<float2*>(reinterpret_cast<uint8_t*>(sw) + kCh * z.wpitch * 2);
+  float2* sdt = reinterpret_cast<float2*>(sw + kCh * z.cpitch);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, q = lane & 3;
   const int c0 = blockIdx.x * kCh, cl = warp * 8 + (lane >> 2), c = c0 + cl;
   const bool in = c < p.C;
@@ -189,12 +252,7 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Scan
   pdl_launch();
   load_wdt(p, z, c0, sw);
   float bias[2];
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int cb = c0 + warp * 8 + (lane & 3) * 2 + i;
-    bias[i] = cb < p.C ? p.dt_b[cb] : 0.f;
-  }
-  const float skip = in ? p.d[c] : 0.f;
+  load_channels(p, c0, bias, sskip);
   f32x2 A[NS / 2], S[NS / 2];
   float* st = p.state + (size_t)seg.z * p.state_pitch + (size_t)c * (4 * NS) + q * NS;
 #pragma unroll
@@ -204,39 +262,27 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Scan
   }
   const int n_tiles = (seg.y + TT - 1) / TT;
   auto rows_of = [&](int j) { return seg.y - j * TT < TT ? seg.y - j * TT : TT; };
-  load_tile<TT>(p, z, seg.x, rows_of(0), c0, ss_smem);
+  load_tile<TT>(p, z, seg.x, rows_of(0), c0, Stage<TT>(ss_smem, z));
   cp_async_commit();
   for (int j = 0; j < n_tiles; ++j) {
-    uint8_t* stage = ss_smem + (j & 1) * stage_bytes;
-    if (j + 1 < n_tiles) load_tile<TT>(p, z, seg.x + (j + 1) * TT, rows_of(j + 1), c0, ss_smem + ((j + 1) & 1) * stage_bytes);
+    const Stage<TT> stage(ss_smem + (j & 1) * stage_bytes, z);
+    if (j + 1 < n_tiles) load_tile<TT>(p, z, seg.x + (j + 1) * TT, rows_of(j + 1), c0, Stage<TT>(ss_smem + ((j + 1) & 1) * stage_bytes, z));
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
-    const float* sr = reinterpret_cast<const float*>(stage);
-    bf16* sx = reinterpret_cast<bf16*>(stage + TT * z.rpitch * 4);
-    const bf16* sz = sx + TT * kCh;
     const int n = rows_of(j);
-    step_sizes<TT>(z, sr, sx, sw, bias, n, sdt);
+    step_sizes<TT>(z, stage, sw, bias, n, sdt);
     __syncwarp();   // a warp computes the step sizes of its own channels
-    const float* bc = sr + z.rank_p + q * (2 * NS);
+    const float* bc = stage.bc + q * (2 * NS);
 #pragma unroll 2
     for (int t0 = 0; t0 < TT; t0 += 4) {
       float y[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) y[e] = scan_step<NS>(sdt[(t0 + e) * kCh + cl], bc + (t0 + e) * z.rpitch, A, S);
-      float v = quad_transpose_sum(y, q);
-      const int t = t0 + q;
-      const float x = __bfloat162float(sx[t * kCh + cl]), g = __bfloat162float(sz[t * kCh + cl]);
-      v = fmaf(skip, x, v);
-      sx[t * kCh + cl] = __float2bfloat16(v * g * sigmoid_f32(g));  // read for the last time: the result takes its place
+      for (int e = 0; e < 4; ++e) y[e] = scan_step<NS>(sdt[(t0 + e) * kCh + cl], bc + (t0 + e) * z.bc, A, S);
+      sdt[(t0 + q) * kCh + cl].x = quad_transpose_sum(y, q);   // all four lanes of the channel have read their step sizes
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < n * 4; i += kScanThreads) {
-      const int t = i >> 2, k = (i & 3) * 8;
-      if (c0 + k < p.C)
-        *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.out) + (size_t)(seg.x + j * TT + t) * p.ldo + c0 + k) =
-            *reinterpret_cast<const uint4*>(sx + t * kCh + k);
-    }
+    store_tile<TT>(p, stage, sdt, sskip, (size_t)seg.x + j * TT, n, c0, nullptr);
     __syncthreads();
   }
   if (in) {
@@ -252,23 +298,19 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_decode_kernel(con
   constexpr int kAhead = NS <= 4 ? 16 : (NS == 8 ? 8 : 4);   // slots whose states are in registers at a time
   extern __shared__ __align__(16) uint8_t ss_smem[];
   __shared__ int s_pos[kSlots];
-  const int stage_bytes = scan_stage_bytes(z, kSlots);
-  bf16* sw = reinterpret_cast<bf16*>(ss_smem + stage_bytes);
-  float2* sdt = reinterpret_cast<float2*>(reinterpret_cast<uint8_t*>(sw) + kCh * z.wpitch * 2);
+  __shared__ float sskip[kCh];
+  const Stage<kSlots> stage(ss_smem, z);
+  bf16* sw = reinterpret_cast<bf16*>(ss_smem + scan_stage_bytes(z, kSlots));
+  float2* sdt = reinterpret_cast<float2*>(sw + kCh * z.cpitch);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, q = lane & 3;
   const int c0 = blockIdx.x * kCh, cl = warp * 8 + (lane >> 2), c = c0 + cl;
   const bool in = c < p.C;
   const int b0 = blockIdx.y * kSlots;
   const int n = p.T - b0 < kSlots ? p.T - b0 : kSlots;
-  load_wdt(p, z, c0, sw);
   if (threadIdx.x < kSlots) s_pos[threadIdx.x] = threadIdx.x < n ? p.seq_lens[b0 + threadIdx.x] - 1 : -1;
+  load_wdt(p, z, c0, sw);
   float bias[2];
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int cb = c0 + warp * 8 + (lane & 3) * 2 + i;
-    bias[i] = cb < p.C ? p.dt_b[cb] : 0.f;
-  }
-  const float skip = in ? p.d[c] : 0.f;
+  load_channels(p, c0, bias, sskip);
   f32x2 A[NS / 2];
 #pragma unroll
   for (int i = 0; i < NS / 2; ++i) A[i] = in ? *reinterpret_cast<const f32x2*>(p.a + (size_t)c * (4 * NS) + q * NS + 2 * i) : 0ull;
@@ -285,16 +327,13 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_decode_kernel(con
   request(0);
   pdl_wait();
   pdl_launch();
-  load_tile<kSlots>(p, z, b0, n, c0, ss_smem);
+  load_tile<kSlots>(p, z, b0, n, c0, stage);
   cp_async_commit();
   cp_async_wait<0>();
   __syncthreads();
-  const float* sr = reinterpret_cast<const float*>(ss_smem);
-  bf16* sx = reinterpret_cast<bf16*>(ss_smem + kSlots * z.rpitch * 4);
-  const bf16* sz = sx + kSlots * kCh;
-  step_sizes<kSlots>(z, sr, sx, sw, bias, n, sdt);
+  step_sizes<kSlots>(z, stage, sw, bias, n, sdt);
   __syncwarp();
-  const float* bc = sr + z.rank_p + q * (2 * NS);
+  const float* bc = stage.bc + q * (2 * NS);
 #pragma unroll
   for (int s0 = 0; s0 < kSlots; s0 += kAhead) {
     if (s0 > 0) request(s0);
@@ -304,31 +343,24 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_decode_kernel(con
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = s0 + t0 + e;
-        y[e] = scan_step<NS>(sdt[t * kCh + cl], bc + t * z.rpitch, A, S[t0 + e]);
+        y[e] = scan_step<NS>(sdt[t * kCh + cl], bc + t * z.bc, A, S[t0 + e]);
         if (in && s_pos[t] >= 0) {
 #pragma unroll
           for (int i = 0; i < NS / 2; ++i) *reinterpret_cast<f32x2*>(st + (size_t)t * p.state_pitch + 2 * i) = S[t0 + e][i];
         }
       }
-      float v = quad_transpose_sum(y, q);
-      const int t = s0 + t0 + q;
-      const float x = __bfloat162float(sx[t * kCh + cl]), g = __bfloat162float(sz[t * kCh + cl]);
-      v = fmaf(skip, x, v);
-      sx[t * kCh + cl] = __float2bfloat16(v * g * sigmoid_f32(g));
+      sdt[(s0 + t0 + q) * kCh + cl].x = quad_transpose_sum(y, q);
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < n * 4; i += kScanThreads) {
-    const int t = i >> 2, k = (i & 3) * 8;
-    if (c0 + k < p.C && s_pos[t] >= 0)
-      *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.out) + (size_t)(b0 + t) * p.ldo + c0 + k) = *reinterpret_cast<const uint4*>(sx + t * kCh + k);
-  }
+  store_tile<kSlots>(p, stage, sdt, sskip, (size_t)b0, n, c0, s_pos);
 }
 
 template <int NS, int TT>
 void launch_prompt(const ScanArgs& a, const ScanSizes& z, cudaStream_t s) {
   auto kernel = selective_scan_kernel<NS, TT>;
   AGRPO_SET_MAX_DYN_SMEM(kernel, 220 * 1024, "selective_scan smem attr");
+  AGRPO_PREFER_SMEM(kernel);
   launch_kernel(kernel, dim3((a.C + kCh - 1) / kCh, a.n_segs), dim3(kScanThreads), scan_smem_bytes(z, TT, 2), s, "selective_scan", a, z);
 }
 
@@ -347,6 +379,7 @@ bool launch_ns(const ScanArgs& a, cudaStream_t s) {
   if (a.T == 0) return true;
   auto kernel = selective_scan_decode_kernel<NS>;
   AGRPO_SET_MAX_DYN_SMEM(kernel, 220 * 1024, "selective_scan_decode smem attr");
+  AGRPO_PREFER_SMEM(kernel);
   launch_kernel(kernel, dim3((a.C + kCh - 1) / kCh, (a.T + 15) / 16), dim3(kScanThreads), smem, s, "selective_scan_decode", a, z);
   return true;
 }

@@ -80,10 +80,6 @@ inline void launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_
   check_cuda(cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...), what);
 }
 
-// Split-K form of a plain product with an fp32 result, up to 256 rows; false when the shape is not served.
-bool launch_gemm_skinny_f32out(const void* a, long long lda, const void* b, long long ldb, float* d, long long ldd, int M, int N, int K, int* status,
-                               int num_sms, cudaStream_t s);
-
 // d[M,N] = alpha * A . B^T (+ bias[N]) (+ d). bf16 operands, fp32 accumulation on tcgen05.
 //   a_mn = false: a is [M, K] row-major with pitch lda; a_mn = true: a is [K, M] row-major
 //   b_mn = false: b is [N, K] row-major with pitch ldb; b_mn = true: b is [K, N] row-major

@@ -115,6 +115,8 @@ struct ScanArgs {
   long long ldx;
   const float* r;
   long long ldr;
+  const void* code;        // packed form: step-size code
+  long long ldcode;
   const void* z;
   long long ldz;
   const void* wdt;         // [C, ldw], columns beyond rank are zero
@@ -132,8 +134,9 @@ struct ScanArgs {
   int T, C, N, rank;
 };
 void launch_selective_scan_plain(bool fp32, const ScanArgs& a, cudaStream_t s);
-// bf16, N up to 64, packed: r = step-size code (padded to a multiple of 16) | for each quarter of the states n values of B, n of C
-// (n = scan_states_per_lane(N)); a in log2 units; a and the state have 4 n entries per channel, zero beyond N.
+// bf16, N up to 64, packed: the step-size code by itself (bf16, padded to a multiple of 16 columns), r = for each quarter of the
+// states n values of B, n of C (n = scan_states_per_lane(N)); a in log2 units; a and the state have 4 n entries per channel, zero
+// beyond N.
 int scan_states_per_lane(int N);   // 0: not served
 bool selective_scan_serves(int N, int rank);
 bool launch_selective_scan(const ScanArgs& a, cudaStream_t s);   // false (nothing launched): not served
@@ -178,5 +181,20 @@ struct ResidualArgs {
   int* status;
 };
 void launch_gemm_residual(const ResidualArgs& a, int num_sms, cudaStream_t s);
+
+// Product whose first n1 columns are stored as bf16 and the others as fp32 (both multiples of 8).
+struct SplitStoreArgs {
+  const void* a;
+  long long lda;
+  const void* w;
+  long long ldw;
+  int M, n1, n2, K;
+  void* d16;
+  long long ld16;
+  float* d32;
+  long long ld32;
+  int* status;
+};
+void launch_gemm_split_store(const SplitStoreArgs& a, int num_sms, cudaStream_t s);
 
 }  // namespace agrpo

@@ -48,6 +48,8 @@ struct ShortConvArgs {
   int silu = 0;                // 1: y / (1 + e^-y) of the result
 };
 void launch_short_conv(bool fp32, const ShortConvArgs& a, cudaStream_t s);
+// Decode rows only: convolution and ring in one launch.
+void launch_short_conv_decode(bool fp32, const ShortConvArgs& a, cudaStream_t s);
 // Writes the values that later steps need into the ring: ring_rows lists the last ring_len rows of each segment
 // (nullptr: decode rows, every row). A launch of its own: the convolution of a segment's first rows reads the ring.
 void launch_short_conv_ring(bool fp32, const ShortConvArgs& a, const int* ring_rows, int n_ring_rows, cudaStream_t s);

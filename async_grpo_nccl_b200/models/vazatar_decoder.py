@@ -126,6 +126,7 @@ class VazatarDecoder(ListedDecoder):
         scans = [l.mixer for l in ls if not l.attends]
         flat = {"u": max(l.mixer.u_dim for l in ls), "cat": max(l.mixer.out_dim + l.ff_p for l in ls), "xc": max([m.inner_p for m in scans], default=0)}
         buf = {k: torch.empty(T * d, **kw) for k, d in flat.items()}
+        buf["code"] = torch.empty(T * max([m.rank_p for m in scans], default=0), **kw)
         buf["x"] = torch.empty(T, W, dtype=torch.float32, device=self.dev)
         buf["h"] = torch.empty(T, 2 * W, **kw)
         buf["loop"] = torch.empty(T if self.cfg.loop is not None else 0, 2 * W, **kw)
@@ -145,7 +146,7 @@ class VazatarDecoder(ListedDecoder):
         n = 2  # embedding, final norm
         for i, first in self.runs:
             l = self.cfg.layers[i]
-            n += int(first) + (3 if l.attends and self._decode_fused(l.mixer) else 4 if l.attends else 6)
+            n += int(first) + (3 if l.attends and self._decode_fused(l.mixer) else 4 if l.attends else 5)
         return n
 
     def _decode_fused(self, m: ChunkAttentionSpec) -> bool:
@@ -227,18 +228,22 @@ class VazatarDecoder(ListedDecoder):
         m, C, T, t = self.cfg.layers[i].mixer, self.C, sb.T, self.scan[i]
         ring, state = self.state[j]
         xc = buf["xc"][:T * m.inner_p].view(T, m.inner_p)
-        n_r = t["wx"].shape[0]
-        r = buf["r"][:T * n_r].view(T, n_r)
         C.conv_silu(u, t["conv"], self.w(f"layers.{i}.conv_b"), ring, sb.rows, sb.ring_rows[m.conv] if sb.rows is not None else None, sb.seq_lens, xc,
                     self.status)
-        if self.fp32:
-            C.gemm_f32(xc, t["wx"], r)
+        n, rest = t["wx"].shape[0], (self.w(f"layers.{i}.wdt"), m.dt_rank, t["dt_b"], t["A"], t["D"], state, sb.segs if sb.rows is not None else None,
+                                     sb.seq_lens, out)
+        if self.packed(i):
+            code, bc = buf["code"][:T * m.rank_p].view(T, m.rank_p), buf["r"][:T * (n - m.rank_p)].view(T, n - m.rank_p)
+            C.gemm_split_store(xc, t["wx"], code, bc, self.status)
+            C.selective_scan(xc, code, bc, u[:, m.inner_p:], *rest)
         else:
-            C.gemm_bf16(xc, t["wx"], r, False, False, None, 1.0, False, self.status, None)
-        scan = C.selective_scan if self.packed(i) else C.selective_scan_plain
-        scan(xc, r, u[:, m.inner_p:], self.w(f"layers.{i}.wdt"), m.dt_rank, t["dt_b"], t["A"], t["D"], state, sb.segs if sb.rows is not None else None,
-             sb.seq_lens, out)
-        self.launches += 4
+            r = buf["r"][:T * n].view(T, n)
+            if self.fp32:
+                C.gemm_f32(xc, t["wx"], r)
+            else:
+                C.gemm_bf16(xc, t["wx"], r, False, False, None, 1.0, False, self.status, None)
+            C.selective_scan_plain(xc, r, u[:, m.inner_p:], *rest)
+        self.launches += 3 if sb.rows is None else 4
 
     # ---- a step ----
     def forward(self, ids: torch.Tensor, sb: StepBatch, buf: Dict[str, torch.Tensor]) -> None:

@@ -241,7 +241,7 @@ def vazatar_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> 
     win, wout = Wr(m.u_dim + F, W), Wr(W, m.out_dim + F)
     swin, swout = Wr(sc.u_dim + F, W), Wr(W, sc.out_dim + F)
     wqkv, wo, wgu, wd = Wr(old.qkv_dim, W), Wr(W, H * D), Wr(2 * Fo, W), Wr(W, Fo)
-    ln, qn, kn = Wr(W), R(m.q_dim), R(m.k_dim)
+    ln, qn, kn = Wr(W), 1 + Wr(m.q_dim), 1 + Wr(m.k_dim)
     maxlen = max(prompt, ctx) + 64
     ang = torch.rand(maxlen, m.rot.dims // 2, device=dev)
     cos, sin = torch.cos(ang), torch.sin(ang)
@@ -297,6 +297,8 @@ def vazatar_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> 
     _, sb = split_batch(torch.from_numpy(flat).to(dev), where, tables)
     rows = sb.pages.shape[0] * 16
     keys, values = Z(rows * G * D), Z(rows * G * E)
+    uq, kc2, vc2 = R(T, m.u_dim), torch.zeros_like(kc), torch.zeros_like(vc)   # the op works in place: attention gets inputs of its own
+    C.qk_norm_rope(uq, qn, kn, 1e-5, m.dim, cos, sin, None, None, sb.rows, None, tables, kc2, vc2, st)
     add("prompt position op", "new", lambda: C.qk_norm_rope(u, qn, kn, 1e-5, m.dim, cos, sin, ss[4], ss[5], sb.rows, None, tables, kc, vc, st), 0.0,
         4.0 * T * (H + G) * D + 4.0 * T * G * E)
     pos, slots, cs = torch.arange(T, device=dev, dtype=torch.int32) % prompt, torch.arange(T, device=dev, dtype=torch.int32), torch.rand(maxlen, D // 2, device=dev)
@@ -307,18 +309,17 @@ def vazatar_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> 
     add("prompt position op", "old", rope, 0.0, 4.0 * T * (H + G) * D + 8.0 * T * G * D)
     pairs_n = n_seq * sum(i % m.chunk + 1 for i in range(prompt))
     pairs_o = n_seq * prompt * (prompt + 1) / 2
-    C.qk_norm_rope(u, qn, kn, 1e-5, m.dim, cos, sin, None, None, sb.rows, None, tables, kc, vc, st)
-    add("prompt attention", "new", lambda: C.chunk_attn_prefill(u, kc, vc, sb.tiles, sb.pages, keys, values, tables, m.scale, m.softcap, m.chunk, cat[:, :m.out_dim], st),
+    add("prompt attention", "new", lambda: C.chunk_attn_prefill(uq, kc2, vc2, sb.tiles, sb.pages, keys, values, tables, m.scale, m.softcap, m.chunk, cat[:, :m.out_dim], st),
         2.0 * pairs_n * H * (D + E), 0.0)
     lse, tiles = torch.empty(H, T, device=dev), _tiles([prompt] * n_seq)
     add("prompt attention", "old", lambda: C.attn_varlen_fwd(qkv, a, lse, tiles, H, G, D, 0.1, st), 4.0 * pairs_o * H * D, 0.0)
     n_slots = max(n_seq, B)
     ring, state = torch.zeros(n_slots, sc.conv, sc.inner_p, device=dev, dtype=bf), torch.zeros(n_slots, sc.inner_p, n_st, device=dev)
-    xc, r = R(T, sc.inner_p), torch.randn(T, wx.shape[0], device=dev)
+    xc, code, r = R(T, sc.inner_p), R(T, sc.rank_p), torch.randn(T, 2 * n_st, device=dev)
     add("prompt convolution", "new", lambda: C.conv_silu(su, conv, conv_b, ring, sb.rows, sb.ring_rows[sc.conv], None, xc, st), 0.0, 4.0 * T * sc.inner_p)
-    add("prompt narrow projection", "new", lambda: C.gemm_bf16(xc, wx, r, False, False, None, 1.0, False, st, None), 0.0, 2.0 * T * sc.inner_p + 4.0 * T * wx.shape[0])
-    add("prompt scan", "new", lambda: C.selective_scan(xc, r, su[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state, sb.segs, None, scat[:, :sc.inner_p]), 0.0,
-        6.0 * T * sc.inner_p + 4.0 * T * wx.shape[0])
+    add("prompt narrow projection", "new", lambda: C.gemm_split_store(xc, wx, code, r, st), *gemms((T, wx.shape[0], sc.inner_p)))
+    add("prompt scan", "new", lambda: C.selective_scan(xc, code, r, su[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state, sb.segs, None, scat[:, :sc.inner_p]), 0.0,
+        6.0 * T * sc.inner_p + T * (2.0 * sc.rank_p + 8.0 * n_st))
 
     # ---------------- decode ----------------
     nbd = (ctx + 15) // 16 + 1
@@ -349,11 +350,10 @@ def vazatar_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> 
                                                                dcat[:, :m.out_dim], sp_new, *part, st), 0.0, 2.0 * B * seen * G * (D + E))
     add("decode attention", "old", lambda: C.paged_decode_attn(qb, dk, dv, dtab, lens, ab, H, G, D, 0.1, sp_old, part[0], part[1], st, part[2]), 0.0,
         4.0 * B * ctx * G * D)
-    dxc, dr = R(B, sc.inner_p), torch.randn(B, wx.shape[0], device=dev)
+    dxc, dcode, dr = R(B, sc.inner_p), R(B, sc.rank_p), torch.randn(B, 2 * n_st, device=dev)
     add("decode convolution", "new", lambda: C.conv_silu(dsu, conv, conv_b, ring[:B], None, None, lens, dxc, st), 0.0, 2.0 * B * sc.inner_p * (sc.conv + 2))
-    add("decode narrow projection", "new", lambda: C.gemm_bf16(dxc, wx, dr, False, False, None, 1.0, False, st, None), 0.0,
-        2.0 * (B + wx.shape[0]) * sc.inner_p + 4.0 * B * wx.shape[0])
-    add("decode scan", "new", lambda: C.selective_scan(dxc, dr, dsu[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state[:B], None, lens, dscat[:, :sc.inner_p]), 0.0,
+    add("decode narrow projection", "new", lambda: C.gemm_split_store(dxc, wx, dcode, dr, st), *gemms((B, wx.shape[0], sc.inner_p)))
+    add("decode scan", "new", lambda: C.selective_scan(dxc, dcode, dr, dsu[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state[:B], None, lens, dscat[:, :sc.inner_p]), 0.0,
         8.0 * B * sc.inner_p * n_st + 2.0 * sc.inner_p * sc.rank_p + 4.0 * sc.inner_p * n_st + 6.0 * B * sc.inner_p)
     return cases
 

@@ -287,6 +287,19 @@ def test_residual_gemm(M, N, K, accumulate):
     assert float((xd.double().cpu() - ref).abs().max()) < 2e-5
 
 
+@pytest.mark.parametrize("M,n1,n2,K", [(3, 16, 8, 64), (100, 96, 32, 640), (200, 112, 64, 512), (300, 32, 128, 200)])
+def test_gemm_with_two_kinds_of_output(M, n1, n2, K):
+    C, g = native(), torch.Generator().manual_seed(M)
+    a, w = rnd(g, M, K), rnd(g, n1 + n2, K, std=K ** -0.5)
+    d16, d32 = torch.empty(M, n1 + 8, device="cuda", dtype=torch.bfloat16)[:, :n1], torch.empty(M, n2, device="cuda")
+    st = torch.zeros(1, dtype=torch.int32, device="cuda")
+    C.gemm_split_store(dev(a), dev(w), d16, d32, st)
+    y = a @ w.T
+    assert int(st.item()) == 0
+    close(d16, y[:, :n1], 5e-3)
+    close(d32, y[:, n1:], 1e-5)
+
+
 def test_gemm_32_bit_on_its_way_out():
     C, g = native(), torch.Generator().manual_seed(4)
     a, b, d = torch.randn(70, 130, generator=g), torch.randn(90, 130, generator=g), torch.randn(70, 90, generator=g)
@@ -487,11 +500,16 @@ class ScanCase:
             parts = [[t[at[s]:at[s] + n] for t in data[s]] for s, n in step]
             x, z, code, B, Cm = (torch.cat(t) for t in zip(*parts))
             T = x.shape[0]
-            r = torch.zeros(T, (R + 2 * n_st + 7) // 8 * 8)
-            r[:, :k.R] = code
-            for i in range(k.N):
-                b, c = (R + i, R + k.N + i) if plain else (R + i // q * 2 * q + i % q, R + i // q * 2 * q + q + i % q)
-                r[:, b], r[:, c] = B[:, i], Cm[:, i]
+            if plain:
+                r = torch.zeros(T, (R + 2 * n_st + 7) // 8 * 8)
+                r[:, :R + 2 * k.N] = torch.cat([code, B, Cm], 1)
+                given = (r.cuda(),)
+            else:   # the code by itself, states in quarters: B, then C of each
+                c16, r = torch.zeros(T, R), torch.zeros(T, 4, 2, q)
+                c16[:, :k.R] = code
+                for i in range(k.N):
+                    r[:, i // q, 0, i % q], r[:, i // q, 1, i % q] = B[:, i], Cm[:, i]
+                given = (dev(c16), r.view(T, 2 * n_st).cuda())
             rows, segs, keep, t0 = [], [], [], 0
             for s, n in step:
                 rows += [(s, at[s] + i, t0, 0) for i in range(n)]
@@ -505,7 +523,7 @@ class ScanCase:
             xc, out = torch.empty(T, k.C, device="cuda", dtype=dt), torch.zeros(T, k.C + 8, device="cuda", dtype=dt)[:, :k.C]
             C.conv_silu(u, dev(k.conv.T, dt), dev(k.conv_b, dt), ring, *where, xc, None)
             scan = C.selective_scan_plain if plain else C.selective_scan
-            scan(xc, r.cuda(), u[:, k.C:], wdt, k.R, dev(k.dt_b, torch.float32), A, dev(k.D, torch.float32), state,
+            scan(xc, *given, u[:, k.C:], wdt, k.R, dev(k.dt_b, torch.float32), A, dev(k.D, torch.float32), state,
                  None if decode else torch.tensor(segs, **i32), lens if decode else None, out)
             t0 = 0
             for s, n in step:
