@@ -289,7 +289,7 @@ void selective_scan(const Tensor& xc, const Tensor& code, const Tensor& r, const
   same_type(code, false, "code"); mat(code, "code");
   const int64_t rank_p = (rank + 15) / 16 * 16;
   TORCH_CHECK(4 * agrpo::scan_states_per_lane(a.N) == a.N && agrpo::selective_scan_serves(a.N, a.rank), "selective_scan: states");
-  TORCH_CHECK(code.size(0) >= a.T && code.size(1) == rank_p && r.size(1) == 2 * a.N && wdt.size(1) >= rank_p && a.C % 32 == 0 &&
+  TORCH_CHECK(code.size(0) >= a.T && code.size(1) == rank_p && code.stride(0) == agrpo::scan_code_pitch(a.rank) && r.size(1) == 2 * a.N && r.is_contiguous() && wdt.size(1) >= rank_p && a.C % 32 == 0 &&
               state.stride(0) % 4 == 0 && aligned16(state) && aligned16(a_), "selective_scan: packed layout");
   a.code = code.data_ptr(); a.ldcode = code.stride(0);
   const c10::cuda::CUDAGuard guard(xc.device());
@@ -375,6 +375,7 @@ void bind_hybrid_ops(pybind11::module_& m) {
         py::arg("tickets"), py::arg("status"), NoGil());
   m.def("chunk_decode_serves", &agrpo::chunk_decode_serves);
   m.def("scan_states_per_lane", &agrpo::scan_states_per_lane);
+  m.def("scan_code_pitch", &agrpo::scan_code_pitch);
   m.def("selective_scan_serves", &agrpo::selective_scan_serves);
   m.def("selective_scan_plain", &selective_scan_plain, py::arg("xc"), py::arg("r"), py::arg("z"), py::arg("wdt"), py::arg("rank"), py::arg("dt_b"),
         py::arg("a"), py::arg("d"), py::arg("state"), py::arg("segs"), py::arg("seq_lens"), py::arg("out"), NoGil());

@@ -7,8 +7,8 @@
 // block's rows of W_dt, done by mma.sync in place, so that they never exist in memory (they would be as large as the input in
 // fp32). Read-outs of four tokens are summed over the four lanes at once: three shuffles, after which each lane finishes one.
 //
-// The projection of the input arrives as the step-size code, bf16 [T, rank_p] (rank_p a multiple of 16), and B and C, fp32
-// [T, 8 NS]: for each quarter of the states NS values of B, then NS of C. A in log2 units [C, 4 NS]; state [slots, C, 4 NS].
+// The projection of the input arrives as the step-size code, bf16 rows of rank_p values (a multiple of 16) eight more apart, and B
+// and C, fp32 [T, 8 NS]: for each quarter of the states NS values of B, then NS of C. Both are copied to shared memory as they are. A in log2 units [C, 4 NS]; state [slots, C, 4 NS].
 #include <cuda_bf16.h>
 
 #include "../common/ptx.cuh"
@@ -26,6 +26,7 @@ typedef unsigned long long f32x2;
 
 constexpr int kCh = 32;        // channels per CTA
 constexpr int kScanThreads = 128;
+constexpr int kYPitch = kCh + 4;   // floats per token of the read-outs
 
 __device__ __forceinline__ float ex2(float x) {
   float y;
@@ -70,20 +71,19 @@ __device__ __forceinline__ void softplus_pair(float v0, float v1, float& r0, flo
 
 struct ScanSizes {
   int rank_p, cpitch;     // step-size code: columns, bf16 elements per row in shared memory (also of W_dt's rows)
-  int bc, bpitch;         // B and C: columns, floats per row
+  int bc;                 // B and C: floats per row
 };
-__host__ __device__ inline ScanSizes scan_sizes(int rank, int ns) {
+inline ScanSizes scan_sizes(int rank, int ns) {
   ScanSizes z;
   z.rank_p = (rank + 15) / 16 * 16;
-  z.cpitch = z.rank_p + 8;   // rows of a fragment fall into different banks
+  z.cpitch = scan_code_pitch(rank);
   z.bc = 8 * ns;
-  z.bpitch = z.bc;
   return z;
 }
 // A stage holds tt tokens: code, B and C, x, z (kCh channels each)
-__host__ __device__ inline int scan_stage_bytes(const ScanSizes& z, int tt) { return tt * (z.cpitch * 2 + z.bpitch * 4 + 2 * kCh * 2); }
+__host__ __device__ inline int scan_stage_bytes(const ScanSizes& z, int tt) { return tt * (z.cpitch * 2 + z.bc * 4 + 2 * kCh * 2); }
 inline int scan_smem_bytes(const ScanSizes& z, int tt, int stages) {
-  return stages * scan_stage_bytes(z, tt) + kCh * z.cpitch * 2 + tt * kCh * 8;
+  return stages * scan_stage_bytes(z, tt) + kCh * z.cpitch * 2 + tt * (kCh * 16 + kYPitch * 4);
 }
 template <int TT>
 struct Stage {
@@ -93,7 +93,7 @@ struct Stage {
   bf16* z;
   __device__ __forceinline__ Stage(uint8_t* base, const ScanSizes& s)
       : code(reinterpret_cast<bf16*>(base)), bc(reinterpret_cast<float*>(base + TT * s.cpitch * 2)),
-        x(reinterpret_cast<bf16*>(base + TT * (s.cpitch * 2 + s.bpitch * 4))), z(x + TT * kCh) {}
+        x(reinterpret_cast<bf16*>(base + TT * (s.cpitch * 2 + s.bc * 4))), z(x + TT * kCh) {}
 };
 
 __device__ __forceinline__ void load_wdt(const ScanArgs& p, const ScanSizes& z, int c0, bf16* sw) {
@@ -109,17 +109,14 @@ __device__ __forceinline__ void load_wdt(const ScanArgs& p, const ScanSizes& z, 
 // step size of zero, and must find finite numbers.
 template <int TT>
 __device__ __forceinline__ void load_tile(const ScanArgs& p, const ScanSizes& z, int row0, int n, int c0, const Stage<TT>& st) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const bf16* code = reinterpret_cast<const bf16*>(p.code);
-  for (int t = warp; t < TT; t += 4) {
-    const size_t row = row0 + t;
-    if (t < n) {
-      for (int k = lane * 8; k < z.rank_p; k += 256) cp_async16(st.code + t * z.cpitch + k, code + row * p.ldcode + k);
-      for (int k = lane * 4; k < z.bc; k += 128) cp_async16(st.bc + t * z.bpitch + k, p.r + row * p.ldr + k);
-    } else {
-      for (int k = lane * 8; k < z.rank_p; k += 256) *reinterpret_cast<uint4*>(st.code + t * z.cpitch + k) = make_uint4(0u, 0u, 0u, 0u);
-      for (int k = lane * 4; k < z.bc; k += 128) *reinterpret_cast<uint4*>(st.bc + t * z.bpitch + k) = make_uint4(0u, 0u, 0u, 0u);
-    }
+  const uint8_t* code = reinterpret_cast<const uint8_t*>(p.code) + (size_t)row0 * z.cpitch * 2;
+  const uint8_t* bc = reinterpret_cast<const uint8_t*>(p.r + (size_t)row0 * z.bc);
+  const int n_code = n * z.cpitch / 8, n_bc = n * z.bc / 4;   // rows lie one after the other: flat copies of 16-byte pieces
+  for (int i = threadIdx.x; i < n_code; i += kScanThreads) cp_async16(reinterpret_cast<uint8_t*>(st.code) + i * 16, code + (size_t)i * 16);
+  for (int i = threadIdx.x; i < n_bc; i += kScanThreads) cp_async16(reinterpret_cast<uint8_t*>(st.bc) + i * 16, bc + (size_t)i * 16);
+  if (n < TT) {
+    for (int i = n_code + threadIdx.x; i < TT * z.cpitch / 8; i += kScanThreads) reinterpret_cast<uint4*>(st.code)[i] = make_uint4(0u, 0u, 0u, 0u);
+    for (int i = n_bc + threadIdx.x; i < TT * z.bc / 4; i += kScanThreads) reinterpret_cast<uint4*>(st.bc)[i] = make_uint4(0u, 0u, 0u, 0u);
   }
   for (int i = threadIdx.x; i < n * 4; i += kScanThreads) {
     const int t = i >> 2, k = (i & 3) * 8;
@@ -130,9 +127,9 @@ __device__ __forceinline__ void load_tile(const ScanArgs& p, const ScanSizes& z,
   }
 }
 
-// {dt, dt x} of TT tokens x 32 channels; tokens from n on get zeros, which leave a state as it is. Warp = 8 channels.
+// {dt, dt, dt x, dt x} of TT tokens x 32 channels (each twice, as operands of paired arithmetic); tokens from n on get zeros, which leave a state as it is. Warp = 8 channels.
 template <int TT>
-__device__ __forceinline__ void step_sizes(const ScanSizes& z, const Stage<TT>& st, const bf16* sw, const float (&bias)[2], int n, float2* sdt) {
+__device__ __forceinline__ void step_sizes(const ScanSizes& z, const Stage<TT>& st, const bf16* sw, const float (&bias)[2], int n, float4* sdt) {
   constexpr int M = TT / 16;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, q2 = (lane & 3) * 2;
@@ -157,21 +154,22 @@ __device__ __forceinline__ void step_sizes(const ScanSizes& z, const Stage<TT>& 
 #pragma unroll
     for (int e = 0; e < 4; e += 2) {
       const int t = m * 16 + g + (e >> 1) * 8, c = warp * 8 + q2;
-      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+      float d0 = 0.f, d1 = 0.f;
+      float2 x = make_float2(0.f, 0.f);
       if (t < n) {
-        const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(st.x + t * kCh + c));
-        softplus_pair(acc[m][e] + bias[0], acc[m][e + 1] + bias[1], o.x, o.z);
-        o.y = o.x * x.x;
-        o.w = o.z * x.y;
+        x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(st.x + t * kCh + c));
+        softplus_pair(acc[m][e] + bias[0], acc[m][e + 1] + bias[1], d0, d1);
       }
-      *reinterpret_cast<float4*>(sdt + t * kCh + c) = o;
+      sdt[t * kCh + c] = make_float4(d0, d0, d0 * x.x, d0 * x.x);
+      sdt[t * kCh + c + 1] = make_float4(d1, d1, d1 * x.y, d1 * x.y);
     }
 }
 
 // One token of one channel quarter: S <- exp2(dt A) S + (dt x) B, returns this quarter's part of S . C.
 template <int NS>
-__device__ __forceinline__ float scan_step(const float2 d, const float* bc, const f32x2 (&A)[NS / 2], f32x2 (&S)[NS / 2]) {
-  const f32x2 dt = pack2(d.x, d.x), dx = pack2(d.y, d.y);
+__device__ __forceinline__ float scan_step(const float4* d, const float* bc, const f32x2 (&A)[NS / 2], f32x2 (&S)[NS / 2]) {
+  const ulonglong2 dd = *reinterpret_cast<const ulonglong2*>(d);
+  const f32x2 dt = dd.x, dx = dd.y;
   f32x2 B[NS / 2], C[NS / 2];
   if constexpr (NS >= 4) {
 #pragma unroll
@@ -207,21 +205,20 @@ __device__ __forceinline__ float quad_transpose_sum(const float (&y)[4], int q) 
   return (high ? b : a) + __shfl_xor_sync(0xffffffffu, high ? a : b, 2);
 }
 
-// Finished read-outs of a tile (in sdt[t][c].x) -> skip, gate, store: thread = 8 channels of a token.
+// Finished read-outs of a tile -> skip, gate, store: thread = 8 channels of a token.
 template <int TT>
-__device__ __forceinline__ void store_tile(const ScanArgs& p, const Stage<TT>& st, const float2* sdt, const float* sskip, size_t row0, int n, int c0,
+__device__ __forceinline__ void store_tile(const ScanArgs& p, const Stage<TT>& st, const float* sy, const float* sskip, size_t row0, int n, int c0,
                                            const int* s_pos) {
   for (int i = threadIdx.x; i < n * 4; i += kScanThreads) {
     const int t = i >> 2, k = (i & 3) * 8;
     if (c0 + k >= p.C || (s_pos != nullptr && s_pos[t] < 0)) continue;
-    float x[8], z[8], o[8];
+    float x[8], z[8], d[8], o[8];
     ld8(st.x + t * kCh + k, x);
     ld8(st.z + t * kCh + k, z);
+    ld8(sskip + k, d);
+    ld8(sy + t * kYPitch + k, o);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      const float y = fmaf(sskip[k + e], x[e], sdt[t * kCh + k + e].x);
-      o[e] = y * z[e] * sigmoid_f32(z[e]);
-    }
+    for (int e = 0; e < 8; ++e) o[e] = fmaf(d[e], x[e], o[e]) * z[e] * sigmoid_f32(z[e]);
     st8(reinterpret_cast<bf16*>(p.out) + (row0 + t) * p.ldo + c0 + k, o);
   }
 }
@@ -240,10 +237,11 @@ __device__ __forceinline__ void load_channels(const ScanArgs& p, int c0, float (
 template <int NS, int TT>
 __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const ScanArgs p, const ScanSizes z) {
   extern __shared__ __align__(16) uint8_t ss_smem[];
-  __shared__ float sskip[kCh];
+  __shared__ __align__(16) float sskip[kCh];
   const int stage_bytes = scan_stage_bytes(z, TT);
   bf16* sw = reinterpret_cast<bf16*>(ss_smem + 2 * stage_bytes);
-  float2* sdt = reinterpret_cast<float2*>(sw + kCh * z.cpitch);
+  float4* __restrict__ sdt = reinterpret_cast<float4*>(sw + kCh * z.cpitch);
+  float* __restrict__ sy = reinterpret_cast<float*>(sdt + TT * kCh);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, q = lane & 3;
   const int c0 = blockIdx.x * kCh, cl = warp * 8 + (lane >> 2), c = c0 + cl;
   const bool in = c < p.C;
@@ -273,16 +271,16 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Scan
     const int n = rows_of(j);
     step_sizes<TT>(z, stage, sw, bias, n, sdt);
     __syncwarp();   // a warp computes the step sizes of its own channels
-    const float* bc = stage.bc + q * (2 * NS);
+    const float* __restrict__ bc = stage.bc + q * (2 * NS);
 #pragma unroll 2
     for (int t0 = 0; t0 < TT; t0 += 4) {
       float y[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) y[e] = scan_step<NS>(sdt[(t0 + e) * kCh + cl], bc + (t0 + e) * z.bc, A, S);
-      sdt[(t0 + q) * kCh + cl].x = quad_transpose_sum(y, q);   // all four lanes of the channel have read their step sizes
+      for (int e = 0; e < 4; ++e) y[e] = scan_step<NS>(sdt + (t0 + e) * kCh + cl, bc + (t0 + e) * (8 * NS), A, S);
+      sy[(t0 + q) * kYPitch + cl] = quad_transpose_sum(y, q);
     }
     __syncthreads();
-    store_tile<TT>(p, stage, sdt, sskip, (size_t)seg.x + j * TT, n, c0, nullptr);
+    store_tile<TT>(p, stage, sy, sskip, (size_t)seg.x + j * TT, n, c0, nullptr);
     __syncthreads();
   }
   if (in) {
@@ -298,10 +296,11 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_decode_kernel(con
   constexpr int kAhead = NS <= 4 ? 16 : (NS == 8 ? 8 : 4);   // slots whose states are in registers at a time
   extern __shared__ __align__(16) uint8_t ss_smem[];
   __shared__ int s_pos[kSlots];
-  __shared__ float sskip[kCh];
+  __shared__ __align__(16) float sskip[kCh];
   const Stage<kSlots> stage(ss_smem, z);
   bf16* sw = reinterpret_cast<bf16*>(ss_smem + scan_stage_bytes(z, kSlots));
-  float2* sdt = reinterpret_cast<float2*>(sw + kCh * z.cpitch);
+  float4* __restrict__ sdt = reinterpret_cast<float4*>(sw + kCh * z.cpitch);
+  float* __restrict__ sy = reinterpret_cast<float*>(sdt + kSlots * kCh);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, q = lane & 3;
   const int c0 = blockIdx.x * kCh, cl = warp * 8 + (lane >> 2), c = c0 + cl;
   const bool in = c < p.C;
@@ -343,17 +342,17 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_decode_kernel(con
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = s0 + t0 + e;
-        y[e] = scan_step<NS>(sdt[t * kCh + cl], bc + t * z.bc, A, S[t0 + e]);
+        y[e] = scan_step<NS>(sdt + t * kCh + cl, bc + t * (8 * NS), A, S[t0 + e]);
         if (in && s_pos[t] >= 0) {
 #pragma unroll
           for (int i = 0; i < NS / 2; ++i) *reinterpret_cast<f32x2*>(st + (size_t)t * p.state_pitch + 2 * i) = S[t0 + e][i];
         }
       }
-      sdt[(s0 + t0 + q) * kCh + cl].x = quad_transpose_sum(y, q);
+      sy[(s0 + t0 + q) * kYPitch + cl] = quad_transpose_sum(y, q);
     }
   }
   __syncthreads();
-  store_tile<kSlots>(p, stage, sdt, sskip, (size_t)b0, n, c0, s_pos);
+  store_tile<kSlots>(p, stage, sy, sskip, (size_t)b0, n, c0, s_pos);
 }
 
 template <int NS, int TT>
@@ -369,7 +368,7 @@ bool launch_ns(const ScanArgs& a, cudaStream_t s) {
   const ScanSizes z = scan_sizes(a.rank, NS);
   if (a.segs != nullptr) {
     if (a.n_segs == 0) return true;
-    if (scan_smem_bytes(z, 32, 2) <= 72 * 1024) launch_prompt<NS, 32>(a, z, s);
+    if (scan_smem_bytes(z, 32, 2) <= 74 * 1024) launch_prompt<NS, 32>(a, z, s);
     else if (scan_smem_bytes(z, 16, 2) <= 220 * 1024) launch_prompt<NS, 16>(a, z, s);
     else return false;
     return true;
@@ -385,6 +384,8 @@ bool launch_ns(const ScanArgs& a, cudaStream_t s) {
 }
 
 }  // namespace
+
+int scan_code_pitch(int rank) { return (rank + 15) / 16 * 16 + 8; }   // rows of a fragment fall into different banks
 
 int scan_states_per_lane(int N) { return N <= 8 ? 2 : N <= 16 ? 4 : N <= 32 ? 8 : N <= 64 ? 16 : 0; }
 

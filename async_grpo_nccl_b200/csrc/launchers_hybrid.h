@@ -134,10 +134,11 @@ struct ScanArgs {
   int T, C, N, rank;
 };
 void launch_selective_scan_plain(bool fp32, const ScanArgs& a, cudaStream_t s);
-// bf16, N up to 64, packed: the step-size code by itself (bf16, padded to a multiple of 16 columns), r = for each quarter of the
+// bf16, N up to 64, packed: the step-size code by itself (bf16 rows scan_code_pitch(rank) apart), r = for each quarter of the
 // states n values of B, n of C (n = scan_states_per_lane(N)); a in log2 units; a and the state have 4 n entries per channel, zero
 // beyond N.
 int scan_states_per_lane(int N);   // 0: not served
+int scan_code_pitch(int rank);     // rank rounded up to a multiple of 16, and eight more
 bool selective_scan_serves(int N, int rank);
 bool launch_selective_scan(const ScanArgs& a, cudaStream_t s);   // false (nothing launched): not served
 

@@ -126,7 +126,7 @@ class VazatarDecoder(ListedDecoder):
         scans = [l.mixer for l in ls if not l.attends]
         flat = {"u": max(l.mixer.u_dim for l in ls), "cat": max(l.mixer.out_dim + l.ff_p for l in ls), "xc": max([m.inner_p for m in scans], default=0)}
         buf = {k: torch.empty(T * d, **kw) for k, d in flat.items()}
-        buf["code"] = torch.empty(T * max([m.rank_p for m in scans], default=0), **kw)
+        buf["code"] = torch.empty(T * max([self.C.scan_code_pitch(m.dt_rank) for m in scans], default=0), **kw)
         buf["x"] = torch.empty(T, W, dtype=torch.float32, device=self.dev)
         buf["h"] = torch.empty(T, 2 * W, **kw)
         buf["loop"] = torch.empty(T if self.cfg.loop is not None else 0, 2 * W, **kw)
@@ -233,7 +233,8 @@ class VazatarDecoder(ListedDecoder):
         n, rest = t["wx"].shape[0], (self.w(f"layers.{i}.wdt"), m.dt_rank, t["dt_b"], t["A"], t["D"], state, sb.segs if sb.rows is not None else None,
                                      sb.seq_lens, out)
         if self.packed(i):
-            code, bc = buf["code"][:T * m.rank_p].view(T, m.rank_p), buf["r"][:T * (n - m.rank_p)].view(T, n - m.rank_p)
+            pitch = C.scan_code_pitch(m.dt_rank)
+            code, bc = buf["code"][:T * pitch].view(T, pitch)[:, :m.rank_p], buf["r"][:T * (n - m.rank_p)].view(T, n - m.rank_p)
             C.gemm_split_store(xc, t["wx"], code, bc, self.status)
             C.selective_scan(xc, code, bc, u[:, m.inner_p:], *rest)
         else:

@@ -315,7 +315,7 @@ def vazatar_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> 
     add("prompt attention", "old", lambda: C.attn_varlen_fwd(qkv, a, lse, tiles, H, G, D, 0.1, st), 4.0 * pairs_o * H * D, 0.0)
     n_slots = max(n_seq, B)
     ring, state = torch.zeros(n_slots, sc.conv, sc.inner_p, device=dev, dtype=bf), torch.zeros(n_slots, sc.inner_p, n_st, device=dev)
-    xc, code, r = R(T, sc.inner_p), R(T, sc.rank_p), torch.randn(T, 2 * n_st, device=dev)
+    xc, code, r = R(T, sc.inner_p), R(T, C.scan_code_pitch(sc.dt_rank))[:, :sc.rank_p], torch.randn(T, 2 * n_st, device=dev)
     add("prompt convolution", "new", lambda: C.conv_silu(su, conv, conv_b, ring, sb.rows, sb.ring_rows[sc.conv], None, xc, st), 0.0, 4.0 * T * sc.inner_p)
     add("prompt narrow projection", "new", lambda: C.gemm_split_store(xc, wx, code, r, st), *gemms((T, wx.shape[0], sc.inner_p)))
     add("prompt scan", "new", lambda: C.selective_scan(xc, code, r, su[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state, sb.segs, None, scat[:, :sc.inner_p]), 0.0,
@@ -350,7 +350,7 @@ def vazatar_cases(new: Any, old: Any, T: int, prompt: int, B: int, ctx: int) -> 
                                                                dcat[:, :m.out_dim], sp_new, *part, st), 0.0, 2.0 * B * seen * G * (D + E))
     add("decode attention", "old", lambda: C.paged_decode_attn(qb, dk, dv, dtab, lens, ab, H, G, D, 0.1, sp_old, part[0], part[1], st, part[2]), 0.0,
         4.0 * B * ctx * G * D)
-    dxc, dcode, dr = R(B, sc.inner_p), R(B, sc.rank_p), torch.randn(B, 2 * n_st, device=dev)
+    dxc, dcode, dr = R(B, sc.inner_p), R(B, C.scan_code_pitch(sc.dt_rank))[:, :sc.rank_p], torch.randn(B, 2 * n_st, device=dev)
     add("decode convolution", "new", lambda: C.conv_silu(dsu, conv, conv_b, ring[:B], None, None, lens, dxc, st), 0.0, 2.0 * B * sc.inner_p * (sc.conv + 2))
     add("decode narrow projection", "new", lambda: C.gemm_split_store(dxc, wx, dcode, dr, st), *gemms((B, wx.shape[0], sc.inner_p)))
     add("decode scan", "new", lambda: C.selective_scan(dxc, dcode, dr, dsu[:, sc.inner_p:], wdt, sc.dt_rank, dt_b, A, skip, state[:B], None, lens, dscat[:, :sc.inner_p]), 0.0,

@@ -505,11 +505,11 @@ class ScanCase:
                 r[:, :R + 2 * k.N] = torch.cat([code, B, Cm], 1)
                 given = (r.cuda(),)
             else:   # the code by itself, states in quarters: B, then C of each
-                c16, r = torch.zeros(T, R), torch.zeros(T, 4, 2, q)
+                c16, r = torch.zeros(T, C.scan_code_pitch(k.R)), torch.zeros(T, 4, 2, q)
                 c16[:, :k.R] = code
                 for i in range(k.N):
                     r[:, i // q, 0, i % q], r[:, i // q, 1, i % q] = B[:, i], Cm[:, i]
-                given = (dev(c16), r.view(T, 2 * n_st).cuda())
+                given = (dev(c16)[:, :R], r.view(T, 2 * n_st).cuda())
             rows, segs, keep, t0 = [], [], [], 0
             for s, n in step:
                 rows += [(s, at[s] + i, t0, 0) for i in range(n)]
