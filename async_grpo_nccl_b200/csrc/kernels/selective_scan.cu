@@ -96,12 +96,11 @@ struct Stage {
         x(reinterpret_cast<bf16*>(base + TT * (s.cpitch * 2 + s.bc * 4))), z(x + TT * kCh) {}
 };
 
-__device__ __forceinline__ void load_wdt(const ScanArgs& p, const ScanSizes& z, int c0, bf16* sw) {
+__device__ __forceinline__ void load_wdt(const ScanArgs& p, const ScanSizes& z, int c0, bf16* sw) {  // completes with the first tile
   for (int c = threadIdx.x >> 5; c < kCh; c += 4)
     for (int k = (threadIdx.x & 31) * 8; k < z.rank_p; k += 256) {
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (c0 + c < p.C) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.wdt) + (size_t)(c0 + c) * p.ldw + k);
-      *reinterpret_cast<uint4*>(sw + c * z.cpitch + k) = v;
+      if (c0 + c < p.C) cp_async16(sw + c * z.cpitch + k, reinterpret_cast<const bf16*>(p.wdt) + (size_t)(c0 + c) * p.ldw + k);
+      else *reinterpret_cast<uint4*>(sw + c * z.cpitch + k) = make_uint4(0u, 0u, 0u, 0u);
     }
 }
 
