@@ -164,11 +164,20 @@ __device__ __forceinline__ void step_sizes(const ScanSizes& z, const Stage<TT>& 
     }
 }
 
-// One token of one channel quarter: S <- exp2(dt A) S + (dt x) B, returns this quarter's part of S . C.
+// Decays exp2(dt A) of one token of one channel quarter.
 template <int NS>
-__device__ __forceinline__ float scan_step(const float4* d, const float* bc, const f32x2 (&A)[NS / 2], f32x2 (&S)[NS / 2]) {
-  const ulonglong2 dd = *reinterpret_cast<const ulonglong2*>(d);
-  const f32x2 dt = dd.x, dx = dd.y;
+__device__ __forceinline__ void scan_decays(const f32x2 dt, const f32x2 (&A)[NS / 2], f32x2 (&e)[NS / 2]) {
+#pragma unroll
+  for (int i = 0; i < NS / 2; ++i) {
+    float a, b;
+    unpack2(mul2(dt, A[i]), a, b);
+    e[i] = pack2(ex2(a), ex2(b));
+  }
+}
+
+// The token itself: S <- e S + (dt x) B; returns this quarter's part of S . C.
+template <int NS>
+__device__ __forceinline__ float scan_update(const f32x2 dx, const float* bc, const f32x2 (&e)[NS / 2], f32x2 (&S)[NS / 2]) {
   f32x2 B[NS / 2], C[NS / 2];
   if constexpr (NS >= 4) {
 #pragma unroll
@@ -182,17 +191,23 @@ __device__ __forceinline__ float scan_step(const float4* d, const float* bc, con
     B[0] = v.x;
     C[0] = v.y;
   }
-  f32x2 y = 0;  // bits of {0.f, 0.f}
+  f32x2 y = 0;
 #pragma unroll
   for (int i = 0; i < NS / 2; ++i) {
-    float a, b;
-    unpack2(mul2(dt, A[i]), a, b);
-    S[i] = fma2(pack2(ex2(a), ex2(b)), S[i], mul2(dx, B[i]));
+    S[i] = fma2(e[i], S[i], mul2(dx, B[i]));
     y = i == 0 ? mul2(S[i], C[i]) : fma2(S[i], C[i], y);
   }
   float a, b;
   unpack2(y, a, b);
   return a + b;
+}
+
+template <int NS>
+__device__ __forceinline__ float scan_step(const float4* d, const float* bc, const f32x2 (&A)[NS / 2], f32x2 (&S)[NS / 2]) {
+  const ulonglong2 dd = *reinterpret_cast<const ulonglong2*>(d);
+  f32x2 e[NS / 2];
+  scan_decays<NS>(dd.x, A, e);
+  return scan_update<NS>(dd.y, bc, e, S);
 }
 
 // Sums over the four lanes of a channel for four tokens: lane q gets token q.
@@ -271,12 +286,37 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Scan
     step_sizes<TT>(z, stage, sw, bias, n, sdt);
     __syncwarp();   // a warp computes the step sizes of its own channels
     const float* __restrict__ bc = stage.bc + q * (2 * NS);
-#pragma unroll 2
-    for (int t0 = 0; t0 < TT; t0 += 4) {
-      float y[4];
+    if constexpr (NS <= 8) {
+      // Few warps are resident, so the instruction stream itself must offer parallel work: while a group of four tokens goes
+      // through the recurrence, the next group's decays are computed and the one before is summed and stored.
+      const float4* __restrict__ mine = sdt + cl;
+      f32x2 decay[2][4][NS / 2], dx[2][4];
+      float y[2][4];
+      auto ahead = [&](int t0, int k) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) y[e] = scan_step<NS>(sdt + (t0 + e) * kCh + cl, bc + (t0 + e) * (8 * NS), A, S);
-      sy[(t0 + q) * kYPitch + cl] = quad_transpose_sum(y, q);
+        for (int e = 0; e < 4; ++e) {
+          const ulonglong2 dd = *reinterpret_cast<const ulonglong2*>(mine + (t0 + e) * kCh);
+          dx[k][e] = dd.y;
+          scan_decays<NS>(dd.x, A, decay[k][e]);
+        }
+      };
+      ahead(0, 0);
+#pragma unroll
+      for (int g = 0; g < TT / 4; ++g) {
+        if (g + 1 < TT / 4) ahead(4 * g + 4, (g + 1) & 1);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[g & 1][e] = scan_update<NS>(dx[g & 1][e], bc + (4 * g + e) * (8 * NS), decay[g & 1][e], S);
+        if (g > 0) sy[(4 * g - 4 + q) * kYPitch + cl] = quad_transpose_sum(y[(g + 1) & 1], q);
+      }
+      sy[(TT - 4 + q) * kYPitch + cl] = quad_transpose_sum(y[(TT / 4 - 1) & 1], q);
+    } else {
+#pragma unroll 1
+      for (int t0 = 0; t0 < TT; t0 += 4) {
+        float y[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] = scan_step<NS>(sdt + (t0 + e) * kCh + cl, bc + (t0 + e) * (8 * NS), A, S);
+        sy[(t0 + q) * kYPitch + cl] = quad_transpose_sum(y, q);
+      }
     }
     __syncthreads();
     store_tile<TT>(p, stage, sy, sskip, (size_t)seg.x + j * TT, n, c0, nullptr);
