@@ -43,7 +43,8 @@ class ListedEngine(RolloutEngine):
         self.dtype = self.params.dtype
 
     def _bytes_per_block(self) -> int:
-        return max(1, sum(heads * size for heads, size in self.dec.paged()) * self.block_size * self.params.element_size())
+        n = sum(heads * size for heads, size in self.dec.paged()) * self.block_size * self.params.element_size()
+        return n or 1 << 20  # a design without paged tensors still counts tokens in blocks, which then cost nothing
 
     def _alloc_cache(self) -> None:
         self.cache = [torch.zeros(self.num_blocks, heads, self.block_size, size, dtype=self.dtype, device=self.dev)

@@ -613,6 +613,14 @@ def test_greedy_generation_matches_the_oracle(name, dtype, graph):
     assert checked >= (80 if dtype == "float32" else 5)
 
 
+def test_a_model_without_attention_needs_no_cache():
+    p = U.tokens("scans", 30, seed=33)
+    eng, out = generate("scans", "float32", [p], 10, num_blocks=None)
+    ids, margins = U.oracle_greedy("scans", p, 10)
+    sure = next((i for i, m in enumerate(margins) if m < 2e-3), 10)
+    assert not eng.cache and out[0].output_ids[:sure].tolist() == ids[:sure]
+
+
 def test_samples_of_a_prompt_share_it():
     """n samples start from one prefill: pages are shared, the partial page, the rings and the states are copied."""
     p = U.tokens("odd", 37, seed=31)
